@@ -67,6 +67,16 @@ int32_t ctx_fail(hf2q_ctx* ctx, int32_t code, const char* msg) {
     if (ctx) snprintf(ctx->err, sizeof ctx->err, "%s", msg);
     return code;
 }
+int32_t ctx_cuda_result(hf2q_ctx* ctx, cudaError_t e, const char* what, uint64_t launches) {
+    if (e == cudaSuccess) {
+        ctx->launches += launches;
+        return HF2Q_OK;
+    }
+    snprintf(ctx->err, sizeof ctx->err, "%s: %s", what, cudaGetErrorString(e));
+    return e == cudaErrorMemoryAllocation ? HF2Q_ERR_OUT_OF_MEMORY : e == cudaErrorInvalidValue ? HF2Q_ERR_INVALID_ARGUMENT : HF2Q_ERR_CUDA;
+}
+int ctx_sm_count(const hf2q_ctx* ctx) { return ctx->dev.sm_count; }
+int ctx_device(const hf2q_ctx* ctx) { return ctx->device; }
 }  // namespace hf2q
 
 namespace {

@@ -12,6 +12,9 @@ namespace hf2q {
 // the context's device status word (api.cu), for the translation units that launch kernels outside api.cu
 uint32_t* ctx_status_word(hf2q_ctx* ctx);
 int32_t ctx_fail(hf2q_ctx* ctx, int32_t code, const char* msg);      // sets the context's last-error text, returns code
+int32_t ctx_cuda_result(hf2q_ctx* ctx, cudaError_t e, const char* what, uint64_t launches);   // counts the launches or reports e
+int ctx_sm_count(const hf2q_ctx* ctx);
+int ctx_device(const hf2q_ctx* ctx);
 
 // cudaFuncSetAttribute(MaxDynamicSharedMemorySize) applies to the CURRENT device only, and one
 // process may hold contexts on several GPUs: the opt-in is remembered per device, not per process.

@@ -1,0 +1,457 @@
+// Recurrent mixers with a matrix state per head, token after token in 32-bit arithmetic:
+//
+//   mlstm   exponential input / forget gates with a running maximum (matrix memory of xLSTM)
+//   delta   gated delta rule, one decay per head and key channel
+//
+// Both keep S[key channel][value column] and treat a value column independently, so the state lives in registers:
+// eight lanes share a column (each holds key channels 32 c + 4 l .. + 3), a warp carries four columns, a CTA of four
+// warps sixteen columns of one head.  A token costs no block barrier; sums over the key channels are three shuffles.
+// Tokens are staged in shared memory in batches by asynchronous copies, two batches in flight.  The state in memory
+// is [head][column][key channel, padded to 32] (f32), which makes a lane's channels consecutive.
+#include "seq_common.cuh"
+
+namespace hf2q {
+namespace {
+using namespace seq;
+
+constexpr int SC_WARPS = 4, SC_COLS = 16, SC_TB = 16, SC_THREADS = SC_WARPS * 32;
+
+__device__ __forceinline__ float group8_sum(float v) {
+    v += __shfl_xor_sync(0xffffffffu, v, 1);
+    v += __shfl_xor_sync(0xffffffffu, v, 2);
+    v += __shfl_xor_sync(0xffffffffu, v, 4);
+    return v;
+}
+// rows of `count` floats -> shared memory, asynchronously, 16 bytes at a time where both sides allow it
+__device__ __forceinline__ void stage_rows(float* dst, uint32_t dst_ld, const float* src, size_t src_ld, uint32_t rows, uint32_t count) {
+    if (count % 4 == 0 && src_ld % 4 == 0 && dst_ld % 4 == 0 && (reinterpret_cast<uintptr_t>(src) & 15) == 0) {
+        const uint32_t q = count / 4;
+        for (uint32_t i = threadIdx.x; i < rows * q; i += SC_THREADS)
+            cp_async16(dst + (i / q) * dst_ld + 4 * (i % q), src + (i / q) * src_ld + 4 * (i % q));
+    } else {
+        for (uint32_t i = threadIdx.x; i < rows * count; i += SC_THREADS)
+            cp_async4(dst + (i / count) * dst_ld + i % count, src + (i / count) * src_ld + i % count);
+    }
+}
+
+template <int RQ> struct State {                     // RQ groups of four key channels per lane
+    float4 v[RQ];
+    __device__ __forceinline__ void load(const float* p) {
+#pragma unroll
+        for (int c = 0; c < RQ; ++c) v[c] = *reinterpret_cast<const float4*>(p + 32 * c);
+    }
+    __device__ __forceinline__ void zero() {
+#pragma unroll
+        for (int c = 0; c < RQ; ++c) v[c] = make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    __device__ __forceinline__ void store(float* p) const {
+#pragma unroll
+        for (int c = 0; c < RQ; ++c) *reinterpret_cast<float4*>(p + 32 * c) = v[c];
+    }
+    __device__ __forceinline__ float dot(const float* p) const {
+        float s = 0.f;
+#pragma unroll
+        for (int c = 0; c < RQ; ++c) {
+            const float4 k = *reinterpret_cast<const float4*>(p + 32 * c);
+            s = fmaf(v[c].x, k.x, s); s = fmaf(v[c].y, k.y, s); s = fmaf(v[c].z, k.z, s); s = fmaf(v[c].w, k.w, s);
+        }
+        return s;
+    }
+    __device__ __forceinline__ void scale(const float* p) {
+#pragma unroll
+        for (int c = 0; c < RQ; ++c) {
+            const float4 k = *reinterpret_cast<const float4*>(p + 32 * c);
+            v[c].x *= k.x; v[c].y *= k.y; v[c].z *= k.z; v[c].w *= k.w;
+        }
+    }
+    __device__ __forceinline__ void axpy(const float* p, float a) {
+#pragma unroll
+        for (int c = 0; c < RQ; ++c) {
+            const float4 k = *reinterpret_cast<const float4*>(p + 32 * c);
+            v[c].x = fmaf(k.x, a, v[c].x); v[c].y = fmaf(k.y, a, v[c].y); v[c].z = fmaf(k.z, a, v[c].z); v[c].w = fmaf(k.w, a, v[c].w);
+        }
+    }
+    __device__ __forceinline__ void decay_axpy(float keep, const float* p, float a) {
+#pragma unroll
+        for (int c = 0; c < RQ; ++c) {
+            const float4 k = *reinterpret_cast<const float4*>(p + 32 * c);
+            v[c].x = fmaf(keep, v[c].x, k.x * a); v[c].y = fmaf(keep, v[c].y, k.y * a);
+            v[c].z = fmaf(keep, v[c].z, k.z * a); v[c].w = fmaf(keep, v[c].w, k.w * a);
+        }
+    }
+};
+
+// ---------------------------------------------------------------- mLSTM
+template <int RQ>
+__global__ void __launch_bounds__(SC_THREADS) mlstm_kernel(const __grid_constant__ hf2q_mlstm a, uint32_t m, float* __restrict__ out) {
+    constexpr uint32_t DP = 32 * RQ;
+    extern __shared__ __align__(16) float dsm[];                    // k, q: [2][SC_TB][DP] each
+    float* ks = dsm;
+    float* qs = dsm + 2 * SC_TB * DP;
+    __shared__ __align__(16) float vs[2][SC_TB][SC_COLS];
+    __shared__ float gi[2][SC_TB], gf[2][SC_TB];
+    pdl_trigger();
+    pdl_wait();
+    const uint32_t h = blockIdx.x, slice = blockIdx.y, n_slices = gridDim.y;
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, l8 = lane & 7;
+    const uint32_t col_s = warp * 4 + (lane >> 3), col0 = slice * SC_COLS, col = col0 + col_s;
+    const uint32_t n_cols = min(static_cast<uint32_t>(SC_COLS), a.vdim - col0);
+    const bool live = col < a.vdim;
+    const float q_scale = 1.0f / sqrtf(static_cast<float>(a.dim));
+    // channels past dim stay zero in shared memory, so the padded part of the state stays zero too
+    for (uint32_t i = threadIdx.x; i < 4 * SC_TB * DP; i += SC_THREADS) dsm[i] = 0.f;
+    for (uint32_t i = threadIdx.x; i < 2 * SC_TB * SC_COLS; i += SC_THREADS) (&vs[0][0][0])[i] = 0.f;
+    __syncthreads();
+    auto stage = [&](uint32_t t0, uint32_t b) {
+        const uint32_t n = min(static_cast<uint32_t>(SC_TB), m - t0);
+        const float* row = a.proj + static_cast<size_t>(t0) * a.ld;
+        stage_rows(ks + b * SC_TB * DP, DP, row + a.k_off + h * a.dim, a.ld, n, a.dim);
+        stage_rows(qs + b * SC_TB * DP, DP, row + a.q_off + h * a.dim, a.ld, n, a.dim);
+        stage_rows(vs[b][0], SC_COLS, row + a.v_off + h * a.vdim + col0, a.ld, n, n_cols);
+        if (threadIdx.x < n) {
+            gi[b][threadIdx.x] = row[static_cast<size_t>(threadIdx.x) * a.ld + a.i_off + h];
+            gf[b][threadIdx.x] = row[static_cast<size_t>(threadIdx.x) * a.ld + a.f_off + h];
+            const float x = a.gate_cap * tanhf((gi[b][threadIdx.x] + a.i_bias[h]) / a.gate_cap);
+            const float f = a.gate_cap * tanhf((gf[b][threadIdx.x] + a.f_bias[h]) / a.gate_cap);
+            gi[b][threadIdx.x] = x;
+            gf[b][threadIdx.x] = -softplusf(-f);
+        }
+        cp_async_commit();
+    };
+    State<RQ> S, N;
+    float* sp = a.s + (static_cast<size_t>(h) * a.vdim + (live ? col : 0)) * DP + 4 * l8;
+    float* np = a.n + (static_cast<size_t>(h) * n_slices + slice) * DP + 4 * l8;
+    float* mp = a.mx + static_cast<size_t>(h) * n_slices + slice;
+    if (live) S.load(sp); else S.zero();
+    N.load(np);
+    float mx = *mp;
+    stage(0, 0);
+    for (uint32_t t0 = 0, b = 0; t0 < m; t0 += SC_TB, b ^= 1) {
+        if (t0 + SC_TB < m) { stage(t0 + SC_TB, b ^ 1); cp_async_wait<1>(); }
+        else cp_async_wait<0>();
+        __syncthreads();
+        const uint32_t n = min(static_cast<uint32_t>(SC_TB), m - t0);
+        for (uint32_t j = 0; j < n; ++j) {
+            const float i_t = gi[b][j], f_t = gf[b][j];
+            const float m_new = fmaxf(f_t + mx, i_t);
+            const float keep = expf(f_t + mx - m_new), write = expf(i_t - m_new);
+            mx = m_new;
+            const float* k = ks + (b * SC_TB + j) * DP + 4 * l8;
+            const float* q = qs + (b * SC_TB + j) * DP + 4 * l8;
+            S.decay_axpy(keep, k, write * vs[b][j][col_s]);
+            N.decay_axpy(keep, k, write);
+            const float num = group8_sum(S.dot(q)) * q_scale, den = group8_sum(N.dot(q)) * q_scale;
+            if (l8 == 0 && live)
+                out[static_cast<size_t>(t0 + j) * a.heads * a.vdim + static_cast<size_t>(h) * a.vdim + col] = num / (fmaxf(fabsf(den), expf(-mx)) + 1e-6f);
+        }
+        __syncthreads();
+    }
+    if (live) S.store(sp);
+    if (warp == 0 && lane < 8) N.store(np);
+    if (threadIdx.x == 0) *mp = mx;
+}
+
+// ---------------------------------------------------------------- gated delta rule
+// S <- g S;  u = beta (v - S^T k);  S <- S + k u;  o = S^T q
+template <int RQ>
+__device__ __forceinline__ float delta_token(State<RQ>& S, const float* g, const float* k, const float* q, float v, float beta) {
+    S.scale(g);
+    const float u = beta * (v - group8_sum(S.dot(k)));
+    S.axpy(k, u);
+    return group8_sum(S.dot(q));
+}
+
+template <int RQ>
+__global__ void __launch_bounds__(SC_THREADS) delta_scan_kernel(const __grid_constant__ hf2q_delta a, uint32_t m, const float* __restrict__ qkv,
+                                                                const float* __restrict__ beta, const float* __restrict__ g, float* __restrict__ out) {
+    constexpr uint32_t DP = 32 * RQ;
+    extern __shared__ __align__(16) float dsm[];                    // k, q, g: [2][SC_TB][DP] each
+    float* ks = dsm;
+    float* qs = dsm + 2 * SC_TB * DP;
+    float* gs = dsm + 4 * SC_TB * DP;
+    __shared__ __align__(16) float vs[2][SC_TB][SC_COLS];
+    __shared__ float bs[2][SC_TB];
+    pdl_trigger();
+    pdl_wait();
+    const uint32_t h = blockIdx.x, slice = blockIdx.y, kvh = h / (a.heads / a.kv_heads);
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, l8 = lane & 7;
+    const uint32_t col_s = warp * 4 + (lane >> 3), col0 = slice * SC_COLS, col = col0 + col_s;
+    const uint32_t n_cols = min(static_cast<uint32_t>(SC_COLS), a.vdim - col0);
+    const bool live = col < a.vdim;
+    const uint32_t qk = a.kv_heads * a.dim, ld = 2 * qk + a.heads * a.vdim;
+    for (uint32_t i = threadIdx.x; i < 6 * SC_TB * DP; i += SC_THREADS) dsm[i] = 0.f;
+    for (uint32_t i = threadIdx.x; i < 2 * SC_TB * SC_COLS; i += SC_THREADS) (&vs[0][0][0])[i] = 0.f;
+    __syncthreads();
+    auto stage = [&](uint32_t t0, uint32_t b) {
+        const uint32_t n = min(static_cast<uint32_t>(SC_TB), m - t0);
+        const float* row = qkv + static_cast<size_t>(t0) * ld;
+        stage_rows(qs + b * SC_TB * DP, DP, row + kvh * a.dim, ld, n, a.dim);
+        stage_rows(ks + b * SC_TB * DP, DP, row + qk + kvh * a.dim, ld, n, a.dim);
+        stage_rows(vs[b][0], SC_COLS, row + 2 * qk + h * a.vdim + col0, ld, n, n_cols);
+        stage_rows(gs + b * SC_TB * DP, DP, g + (static_cast<size_t>(t0) * a.heads + h) * a.dim, static_cast<size_t>(a.heads) * a.dim, n, a.dim);
+        if (threadIdx.x < n) bs[b][threadIdx.x] = beta[static_cast<size_t>(t0 + threadIdx.x) * a.heads + h];
+        cp_async_commit();
+    };
+    State<RQ> S;
+    float* sp = a.s + (static_cast<size_t>(h) * a.vdim + (live ? col : 0)) * DP + 4 * l8;
+    if (live) S.load(sp); else S.zero();
+    stage(0, 0);
+    for (uint32_t t0 = 0, b = 0; t0 < m; t0 += SC_TB, b ^= 1) {
+        if (t0 + SC_TB < m) { stage(t0 + SC_TB, b ^ 1); cp_async_wait<1>(); }
+        else cp_async_wait<0>();
+        __syncthreads();
+        const uint32_t n = min(static_cast<uint32_t>(SC_TB), m - t0);
+        for (uint32_t j = 0; j < n; ++j) {
+            const uint32_t o = (b * SC_TB + j) * DP + 4 * l8;
+            const float r = delta_token<RQ>(S, gs + o, ks + o, qs + o, vs[b][j][col_s], bs[b][j]);
+            if (l8 == 0 && live) out[static_cast<size_t>(t0 + j) * a.heads * a.vdim + static_cast<size_t>(h) * a.vdim + col] = r;
+        }
+        __syncthreads();
+    }
+    if (live) S.store(sp);
+}
+
+// convolution + SiLU of channel `ch` (0 .. 2 qk + heads vdim) for one token; before(j): the input j tokens back
+template <typename Before>
+__device__ __forceinline__ float conv_silu(const float* w, uint32_t taps, float now, Before before) {
+    float s = now * w[taps - 1];
+    for (uint32_t j = 1; j < taps; ++j) s = fmaf(before(j), w[taps - 1 - j], s);
+    return siluf(s);
+}
+__device__ __forceinline__ float decay_of(float a_log, float x) { return expf(-expf(a_log) * softplusf(x)); }
+__device__ __forceinline__ float low_rank_dot(const void* w, size_t row, uint32_t ld, const float* x) {
+    const __nv_bfloat16* r = static_cast<const __nv_bfloat16*>(w) + row * ld;
+    float s = 0.f;
+    for (uint32_t c = 0; c < ld; c += 8) {
+        float f[8];
+        load8(r + c, f);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) s = fmaf(f[i], x[c + i], s);
+    }
+    return s;
+}
+
+// One token from the raw projection row: convolution, SiLU, unit norms, decays, gate and the state update.
+template <int RQ>
+__global__ void __launch_bounds__(SC_THREADS) delta_step_kernel(const __grid_constant__ hf2q_delta a, float* __restrict__ out, float* __restrict__ gate) {
+    constexpr uint32_t DP = 32 * RQ;
+    __shared__ __align__(16) float ks[DP], qs[DP], gs[DP], vs[SC_COLS];
+    __shared__ float red[64];
+    extern __shared__ __align__(16) float lr[];                     // a1 [a_rank_ld], g1 [g_rank_ld]
+    pdl_trigger();
+    const uint32_t h = blockIdx.x, slice = blockIdx.y, rep = a.heads / a.kv_heads, kvh = h / rep;
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, l8 = lane & 7;
+    const uint32_t col_s = warp * 4 + (lane >> 3), col0 = slice * SC_COLS, col = col0 + col_s;
+    const uint32_t n_cols = min(static_cast<uint32_t>(SC_COLS), a.vdim - col0);
+    const bool live = col < a.vdim;
+    pdl_wait();
+    State<RQ> S;
+    float* sp = a.s + (static_cast<size_t>(h) * a.vdim + (live ? col : 0)) * DP + 4 * l8;
+    if (live) S.load(sp); else S.zero();
+    const uint32_t pos = *a.pos, qk = a.kv_heads * a.dim;
+    for (uint32_t i = threadIdx.x; i < a.a_rank_ld; i += SC_THREADS) lr[i] = a.proj[a.a1_off + i];
+    for (uint32_t i = threadIdx.x; i < a.g_rank_ld; i += SC_THREADS) lr[a.a_rank_ld + i] = a.proj[a.g1_off + i];
+    // the state ring has one column more than the taps look back, so this token's column is read by nobody
+    auto channel = [&](uint32_t ch, const float* w, float now, bool keep) {
+        float* st = a.conv_state + static_cast<size_t>(ch) * a.taps;
+        const float v = conv_silu(w, a.taps, now, [&](uint32_t j) { return st[(pos + a.taps - j) % a.taps]; });
+        if (keep) st[pos % a.taps] = now;
+        return v;
+    };
+    float ss[2] = {0.f, 0.f};
+    for (uint32_t i = threadIdx.x; i < DP; i += SC_THREADS) {
+        float q = 0.f, k = 0.f;
+        if (i < a.dim) {
+            const uint32_t c = kvh * a.dim + i;
+            const bool keep = slice == 0 && h % rep == 0;
+            q = channel(c, a.q_conv + static_cast<size_t>(c) * a.taps, a.proj[a.q_off + c], keep);
+            k = channel(qk + c, a.k_conv + static_cast<size_t>(c) * a.taps, a.proj[a.k_off + c], keep);
+        }
+        qs[i] = q;
+        ks[i] = k;
+        ss[0] += q * q;
+        ss[1] += k * k;
+    }
+    if (threadIdx.x < SC_COLS) {
+        float v = 0.f;
+        if (threadIdx.x < n_cols) {
+            const uint32_t c = h * a.vdim + col0 + threadIdx.x;
+            v = channel(2 * qk + c, a.v_conv + static_cast<size_t>(c) * a.taps, a.proj[a.v_off + c], true);
+        }
+        vs[threadIdx.x] = v;
+    }
+    block_sum(ss, red);                                             // (its barrier also publishes lr and vs)
+    const float iq = 1.0f / sqrtf(ss[0] + 1e-6f) / sqrtf(static_cast<float>(a.dim)), ik = 1.0f / sqrtf(ss[1] + 1e-6f);
+    for (uint32_t i = threadIdx.x; i < DP; i += SC_THREADS) {
+        qs[i] *= iq;
+        ks[i] *= ik;
+        gs[i] = i < a.dim ? decay_of(a.a_log[h], low_rank_dot(a.a2, static_cast<size_t>(h) * a.dim + i, a.a_rank_ld, lr) + a.dt_bias[h * a.dim + i]) : 0.f;
+    }
+    if (threadIdx.x < n_cols) {
+        const uint32_t c = h * a.vdim + col0 + threadIdx.x;
+        gate[c] = low_rank_dot(a.g2, c, a.g_rank_ld, lr + a.a_rank_ld);
+    }
+    __syncthreads();
+    const float r = delta_token<RQ>(S, gs + 4 * l8, ks + 4 * l8, qs + 4 * l8, vs[col_s], sigmoidf(a.proj[a.b_off + h]));
+    if (live) {
+        S.store(sp);
+        if (l8 == 0) out[h * a.vdim + col] = r;
+    }
+}
+
+// One CTA per token: a warp takes one head of q or k (or a head of v) at a time.
+template <typename LR>
+__global__ void __launch_bounds__(256) delta_prep_kernel(const __grid_constant__ hf2q_delta a, float* __restrict__ qkv, float* __restrict__ beta,
+                                                         LR* __restrict__ a1, LR* __restrict__ g1) {
+    pdl_trigger();
+    pdl_wait();
+    const uint32_t t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const uint32_t pos = *a.pos, qk = a.kv_heads * a.dim;
+    const float* row = a.proj + static_cast<size_t>(t) * a.ld;
+    float* dst = qkv + static_cast<size_t>(t) * (2 * qk + a.heads * a.vdim);
+    auto channel = [&](uint32_t ch, const float* w, uint32_t off) {
+        return conv_silu(w, a.taps, row[off], [&](uint32_t j) {
+            return j <= t ? row[static_cast<ptrdiff_t>(off) - static_cast<ptrdiff_t>(j) * a.ld]
+                          : a.conv_state[static_cast<size_t>(ch) * a.taps + (pos + t + a.taps - j) % a.taps];
+        });
+    };
+    for (uint32_t hd = warp; hd < 2 * a.kv_heads; hd += 8) {
+        const bool is_k = hd >= a.kv_heads;
+        const uint32_t c0 = (is_k ? hd - a.kv_heads : hd) * a.dim;
+        const float* w = is_k ? a.k_conv : a.q_conv;
+        float v[8], s = 0.f;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+            const uint32_t i = lane + 32 * j;
+            v[j] = i < a.dim ? channel((is_k ? qk : 0u) + c0 + i, w + static_cast<size_t>(c0 + i) * a.taps, (is_k ? a.k_off : a.q_off) + c0 + i) : 0.f;
+            s += v[j] * v[j];
+        }
+        float inv = 1.0f / sqrtf(warp_sum(s) + 1e-6f);
+        if (!is_k) inv /= sqrtf(static_cast<float>(a.dim));
+#pragma unroll
+        for (int j = 0; j < 8; ++j)
+            if (lane + 32 * j < a.dim) dst[(is_k ? qk : 0u) + c0 + lane + 32 * j] = v[j] * inv;
+    }
+    for (uint32_t c = threadIdx.x; c < a.heads * a.vdim; c += 256)
+        dst[2 * qk + c] = channel(2 * qk + c, a.v_conv + static_cast<size_t>(c) * a.taps, a.v_off + c);
+    for (uint32_t h = threadIdx.x; h < a.heads; h += 256) beta[static_cast<size_t>(t) * a.heads + h] = sigmoidf(row[a.b_off + h]);
+    for (uint32_t c = threadIdx.x; c < a.a_rank_ld; c += 256) a1[static_cast<size_t>(t) * a.a_rank_ld + c] = from_f32<LR>(row[a.a1_off + c]);
+    for (uint32_t c = threadIdx.x; c < a.g_rank_ld; c += 256) g1[static_cast<size_t>(t) * a.g_rank_ld + c] = from_f32<LR>(row[a.g1_off + c]);
+}
+
+__global__ void __launch_bounds__(256) delta_decay_kernel(const float* __restrict__ a_log, const float* __restrict__ dt_bias, uint32_t dim, uint32_t per_token,
+                                                          uint64_t n, float* __restrict__ g) {
+    pdl_trigger();
+    pdl_wait();
+    const uint64_t stride = static_cast<uint64_t>(gridDim.x) * blockDim.x;
+    for (uint64_t i = static_cast<uint64_t>(blockIdx.x) * blockDim.x + threadIdx.x; i < n; i += stride) {
+        const uint32_t c = static_cast<uint32_t>(i % per_token);
+        g[i] = decay_of(a_log[c / dim], g[i] + dt_bias[c]);
+    }
+}
+
+bool delta_ok(const hf2q_delta* a) {
+    return a && a->proj && a->q_conv && a->k_conv && a->v_conv && a->a_log && a->dt_bias && a->a2 && a->g2 && a->conv_state && a->s && a->pos &&
+           a->heads && a->kv_heads && a->heads % a->kv_heads == 0 && a->dim && a->dim <= 256 && a->vdim && a->taps && a->a_rank_ld % 8 == 0 &&
+           a->g_rank_ld % 8 == 0 && a->a_rank_ld && a->g_rank_ld;
+}
+template <int RQ>
+cudaError_t launch_scan(const hf2q_delta& a, uint32_t m, const float* qkv, const float* beta, const float* g, float* out, cudaStream_t st) {
+    static PerDeviceFlag flag;
+    const size_t smem = 6ull * SC_TB * 32 * RQ * sizeof(float);
+    if (const cudaError_t e = ensure_max_dynamic_smem(delta_scan_kernel<RQ>, static_cast<int>(smem), flag); e != cudaSuccess) return e;
+    return launch_pdl(delta_scan_kernel<RQ>, dim3(a.heads, (a.vdim + SC_COLS - 1) / SC_COLS), dim3(SC_THREADS), smem, st, a, m, qkv, beta, g, out);
+}
+
+template <int RQ>
+cudaError_t launch_mlstm(const hf2q_mlstm& a, uint32_t m, float* out, cudaStream_t st) {
+    static PerDeviceFlag flag;
+    const size_t smem = 4ull * SC_TB * 32 * RQ * sizeof(float);
+    if (const cudaError_t e = ensure_max_dynamic_smem(mlstm_kernel<RQ>, static_cast<int>(smem), flag); e != cudaSuccess) return e;
+    return launch_pdl(mlstm_kernel<RQ>, dim3(a.heads, (a.vdim + SC_COLS - 1) / SC_COLS), dim3(SC_THREADS), smem, st, a, m, out);
+}
+
+#define HF2Q_RQ_CASES(F) F(1) F(2) F(3) F(4) F(5) F(6) F(7) F(8)
+
+}  // namespace
+}  // namespace hf2q
+
+using namespace hf2q;
+using namespace hf2q::seq;
+
+extern "C" {
+
+HF2Q_API int32_t hf2q_cuda_mlstm(hf2q_ctx* ctx, void* stream, const hf2q_mlstm* a, uint32_t m, float* out) {
+    if (!ctx) return HF2Q_ERR_INVALID_ARGUMENT;
+    if (!a || !a->proj || !a->i_bias || !a->f_bias || !a->s || !a->n || !a->mx || !out || a->heads == 0 || a->dim == 0 || a->vdim == 0 || a->dim > 256 ||
+        !(a->gate_cap > 0.f))
+        return ctx_fail(ctx, HF2Q_ERR_INVALID_ARGUMENT, "mlstm: null pointer, or a size outside dim 1..256");
+    if (m == 0) return HF2Q_OK;
+    const cudaStream_t st = static_cast<cudaStream_t>(stream);
+    cudaError_t e = cudaErrorInvalidValue;
+    switch ((a->dim + 31) / 32) {
+#define F(RQ) case RQ: e = launch_mlstm<RQ>(*a, m, out, st); break;
+        HF2Q_RQ_CASES(F)
+#undef F
+        default: break;
+    }
+    return ctx_cuda_result(ctx, e, "mlstm", 1);
+}
+
+HF2Q_API int32_t hf2q_cuda_delta_step(hf2q_ctx* ctx, void* stream, const hf2q_delta* a, float* out, float* gate) {
+    if (!ctx) return HF2Q_ERR_INVALID_ARGUMENT;
+    if (!delta_ok(a) || !out || !gate) return ctx_fail(ctx, HF2Q_ERR_INVALID_ARGUMENT, "delta_step: null pointer or an unsupported size");
+    const dim3 grid(a->heads, (a->vdim + SC_COLS - 1) / SC_COLS);
+    const size_t smem = static_cast<size_t>(a->a_rank_ld + a->g_rank_ld) * 4;
+    if (smem > 32 * 1024) return ctx_fail(ctx, HF2Q_ERR_INVALID_ARGUMENT, "delta_step: rank too large");
+    cudaError_t e = cudaErrorInvalidValue;
+    switch ((a->dim + 31) / 32) {
+#define F(RQ) case RQ: e = launch_pdl(delta_step_kernel<RQ>, grid, dim3(SC_THREADS), smem, static_cast<cudaStream_t>(stream), *a, out, gate); break;
+        HF2Q_RQ_CASES(F)
+#undef F
+        default: break;
+    }
+    return ctx_cuda_result(ctx, e, "delta_step", 1);
+}
+
+HF2Q_API int32_t hf2q_cuda_delta_prep(hf2q_ctx* ctx, void* stream, const hf2q_delta* a, uint32_t m, float* qkv, float* beta, void* a1, void* g1,
+                                      uint32_t lr_dtype) {
+    if (!ctx) return HF2Q_ERR_INVALID_ARGUMENT;
+    if (!delta_ok(a) || !qkv || !beta || !a1 || !g1) return ctx_fail(ctx, HF2Q_ERR_INVALID_ARGUMENT, "delta_prep: null pointer or an unsupported size");
+    if (m == 0) return HF2Q_OK;
+    const cudaStream_t st = static_cast<cudaStream_t>(stream);
+    cudaError_t e = cudaErrorInvalidValue;
+    if (lr_dtype == HF2Q_DT_F32)
+        e = launch_pdl(delta_prep_kernel<float>, dim3(m), dim3(256), 0, st, *a, qkv, beta, static_cast<float*>(a1), static_cast<float*>(g1));
+    else if (lr_dtype == HF2Q_DT_BF16)
+        e = launch_pdl(delta_prep_kernel<__nv_bfloat16>, dim3(m), dim3(256), 0, st, *a, qkv, beta, static_cast<__nv_bfloat16*>(a1), static_cast<__nv_bfloat16*>(g1));
+    return ctx_cuda_result(ctx, e, "delta_prep", 1);
+}
+
+HF2Q_API int32_t hf2q_cuda_delta_decay(hf2q_ctx* ctx, void* stream, const hf2q_delta* a, uint32_t m, float* g) {
+    if (!ctx) return HF2Q_ERR_INVALID_ARGUMENT;
+    if (!delta_ok(a) || !g) return ctx_fail(ctx, HF2Q_ERR_INVALID_ARGUMENT, "delta_decay: null pointer or an unsupported size");
+    if (m == 0) return HF2Q_OK;
+    const uint64_t n = static_cast<uint64_t>(m) * a->heads * a->dim, want = (n + 255) / 256, cap = static_cast<uint64_t>(ctx_sm_count(ctx)) * 16;
+    const cudaError_t e = launch_pdl(delta_decay_kernel, dim3(static_cast<unsigned>(want < cap ? want : cap)), dim3(256), 0, static_cast<cudaStream_t>(stream),
+                                     a->a_log, a->dt_bias, a->dim, a->heads * a->dim, n, g);
+    return ctx_cuda_result(ctx, e, "delta_decay", 1);
+}
+
+HF2Q_API int32_t hf2q_cuda_delta_scan(hf2q_ctx* ctx, void* stream, const hf2q_delta* a, uint32_t m, const float* qkv, const float* beta, const float* g,
+                                      float* out) {
+    if (!ctx) return HF2Q_ERR_INVALID_ARGUMENT;
+    if (!delta_ok(a) || !qkv || !beta || !g || !out) return ctx_fail(ctx, HF2Q_ERR_INVALID_ARGUMENT, "delta_scan: null pointer or an unsupported size");
+    if (m == 0) return HF2Q_OK;
+    const cudaStream_t st = static_cast<cudaStream_t>(stream);
+    cudaError_t e = cudaErrorInvalidValue;
+    switch ((a->dim + 31) / 32) {
+#define F(RQ) case RQ: e = launch_scan<RQ>(*a, m, qkv, beta, g, out, st); break;
+        HF2Q_RQ_CASES(F)
+#undef F
+        default: break;
+    }
+    return ctx_cuda_result(ctx, e, "delta_scan", 1);
+}
+
+}  // extern "C"

@@ -1,0 +1,151 @@
+// Shared device helpers of the bf16-weight sequence-model kernels (dense_bf16.cu, window_attn.cu,
+// scan.cu, seq_ops.cu): element conversion, block reductions, programmatic dependent launch, and the
+// row prologues that both the stand-alone kernels and the fused mat-vec use.
+#pragma once
+#include "common.cuh"
+#include "kernels.h"
+
+namespace hf2q {
+namespace seq {
+
+__device__ __forceinline__ float to_f32(float v) { return v; }
+__device__ __forceinline__ float to_f32(__nv_bfloat16 v) { return __bfloat162float(v); }
+template <typename T> __device__ __forceinline__ T from_f32(float v);
+template <> __device__ __forceinline__ float from_f32<float>(float v) { return v; }
+template <> __device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
+
+__device__ __forceinline__ float bf_lo(uint32_t w) { return __uint_as_float(w << 16); }
+__device__ __forceinline__ float bf_hi(uint32_t w) { return __uint_as_float(w & 0xffff0000u); }
+
+// eight consecutive elements (16-byte aligned for bf16, 32 bytes read as two 16-byte loads for f32)
+__device__ __forceinline__ void load8(const __nv_bfloat16* p, float (&o)[8]) {
+    const uint4 v = *reinterpret_cast<const uint4*>(p);
+    o[0] = bf_lo(v.x); o[1] = bf_hi(v.x); o[2] = bf_lo(v.y); o[3] = bf_hi(v.y);
+    o[4] = bf_lo(v.z); o[5] = bf_hi(v.z); o[6] = bf_lo(v.w); o[7] = bf_hi(v.w);
+}
+__device__ __forceinline__ void load8(const float* p, float (&o)[8]) {
+    const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+    o[0] = a.x; o[1] = a.y; o[2] = a.z; o[3] = a.w; o[4] = b.x; o[5] = b.y; o[6] = b.z; o[7] = b.w;
+}
+
+__device__ __forceinline__ float sigmoidf(float x) { return 1.0f / (1.0f + expf(-x)); }
+__device__ __forceinline__ float softplusf(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+__device__ __forceinline__ float siluf(float x) { return x / (1.0f + expf(-x)); }
+__device__ __forceinline__ float gelu_tanhf(float x) {
+    return 0.5f * x * (1.0f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
+}
+
+__device__ __forceinline__ float warp_sum(float v) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+    return v;
+}
+// Sum of N values over the block; red: N * 32 floats of shared memory.  Ends with every thread holding the
+// sums; the caller may reuse `red` only after another barrier.
+template <int N>
+__device__ __forceinline__ void block_sum(float (&v)[N], float* red) {
+#pragma unroll
+    for (int i = 0; i < N; ++i) v[i] = warp_sum(v[i]);
+    if ((threadIdx.x & 31) == 0)
+#pragma unroll
+        for (int i = 0; i < N; ++i) red[i * 32 + (threadIdx.x >> 5)] = v[i];
+    __syncthreads();
+    const uint32_t nw = blockDim.x >> 5;
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+        float s = 0.f;
+        for (uint32_t w = 0; w < nw; ++w) s += red[i * 32 + w];
+        v[i] = s;
+    }
+}
+
+// Programmatic dependent launch.  Every kernel launched with launch_pdl() calls pdl_wait() before it touches
+// memory that an earlier kernel of the stream writes (or still reads); weights may be touched before.
+__device__ __forceinline__ void pdl_trigger() { asm volatile("griddepcontrol.launch_dependents;" ::: "memory"); }
+__device__ __forceinline__ void pdl_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
+__device__ __forceinline__ void prefetch_l2(const void* p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
+
+template <typename... KArgs, typename... Args>
+inline cudaError_t launch_pdl(void (*kern)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t st, Args... args) {
+    cudaLaunchConfig_t cfg{};
+    cfg.gridDim = grid;
+    cfg.blockDim = block;
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = st;
+    cudaLaunchAttribute attr[1];
+    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[0].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = 1;
+    return cudaLaunchKernelEx(&cfg, kern, static_cast<KArgs>(args)...);
+}
+
+__device__ __forceinline__ void cp_async4(void* dst, const void* src) {
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_async16(void* dst, const void* src) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N> __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+// ---------------------------------------------------------------- row prologues
+// Residual update of row t into xs[0..width) (shared memory):
+//   x + 0.5 (rms(a) a_norm + rms(b) b_norm)  (+ add0)  (+ step)
+// and the reciprocal root mean square of the result.  Rows are `width` floats apart.
+__device__ __forceinline__ float residual_row(const hf2q_pre_norm& p, uint32_t t, float* xs, float* red) {
+    const size_t o = static_cast<size_t>(t) * p.width;
+    const float n = static_cast<float>(p.width);
+    float ia = 0.f, ib = 0.f;
+    if (p.a) {
+        float s[2] = {0.f, 0.f};
+        for (uint32_t i = threadIdx.x; i < p.width; i += blockDim.x) {
+            const float va = p.a[o + i], vb = p.b[o + i];
+            s[0] += va * va;
+            s[1] += vb * vb;
+        }
+        block_sum(s, red);
+        ia = 0.5f / sqrtf(s[0] / n + p.eps);
+        ib = 0.5f / sqrtf(s[1] / n + p.eps);
+        __syncthreads();
+    }
+    float s[1] = {0.f};
+    for (uint32_t i = threadIdx.x; i < p.width; i += blockDim.x) {
+        float v = p.x[o + i];
+        if (p.a) v += p.a[o + i] * ia * p.a_norm[i] + p.b[o + i] * ib * p.b_norm[i];
+        if (p.add0) v += p.add0[o + i];
+        if (p.step) v += p.step[i];
+        xs[i] = v;
+        s[0] += v * v;
+    }
+    block_sum(s, red);
+    const float inv = 1.0f / sqrtf(s[0] / n + p.eps);
+    __syncthreads();
+    return inv;
+}
+
+// One row of gated head outputs into out[0..heads * head_dim): (norm ? o / rms_head(o) * norm : o) * sigmoid(gate);
+// one warp per head.  norm_all: the weight spans all heads, else one head_dim vector is shared.
+template <typename OUT>
+__device__ __forceinline__ void gated_heads_row(const hf2q_gated_heads& g, uint32_t t, OUT* out, uint32_t warp, uint32_t n_warps) {
+    const uint32_t lane = threadIdx.x & 31;
+    const float* o = g.o + static_cast<size_t>(t) * g.ldo;
+    const float* gate = g.gate + static_cast<size_t>(t) * g.ldg;
+    for (uint32_t h = warp; h < g.heads; h += n_warps) {
+        const uint32_t c0 = h * g.head_dim;
+        float inv = 1.0f;
+        if (g.norm) {
+            float s = 0.f;
+            for (uint32_t i = lane; i < g.head_dim; i += 32) { const float v = o[c0 + i]; s += v * v; }
+            inv = 1.0f / sqrtf(warp_sum(s) / static_cast<float>(g.head_dim) + g.eps);
+        }
+        for (uint32_t i = lane; i < g.head_dim; i += 32) {
+            float v = o[c0 + i];
+            if (g.norm) v = v * inv * g.norm[g.norm_all ? c0 + i : i];
+            out[c0 + i] = from_f32<OUT>(v * sigmoidf(gate[c0 + i]));
+        }
+    }
+}
+
+}  // namespace seq
+}  // namespace hf2q

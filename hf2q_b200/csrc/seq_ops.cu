@@ -1,0 +1,162 @@
+// Row-wise steps around the products of a bf16-weight decoder: embedding rows with the hashed bigram table, the
+// residual update + RMS norm + token shift in front of a product, gated head outputs, and the hand-over of the
+// shift / convolution state after a portion of several tokens.
+#include "seq_common.cuh"
+
+namespace hf2q {
+namespace {
+using namespace seq;
+
+__global__ void __launch_bounds__(256) embed_kernel(const __grid_constant__ hf2q_embed e, const uint32_t* __restrict__ ids, uint32_t m,
+                                                    float* __restrict__ x, uint32_t* status) {
+    pdl_trigger();
+    pdl_wait();
+    const uint32_t t = blockIdx.x;
+    const uint32_t id = ids[t], pos = *e.pos + t;
+    const uint32_t before = t ? ids[t - 1] : *e.prev;
+    const uint32_t last = ids[m - 1];
+    __syncthreads();                                       // row 0 reads *prev before it replaces it
+    if (t == 0 && threadIdx.x == 0) *e.prev = last;
+    const bool bad = id >= e.vocab;
+    if (bad && threadIdx.x == 0) atomicOr(status, STATUS_BAD_EXPERT_ID);
+    const __nv_bfloat16* row = static_cast<const __nv_bfloat16*>(e.embed) + static_cast<size_t>(bad ? 0 : id) * e.ld;
+    const __nv_bfloat16* big = nullptr;
+    if (e.bigram) {
+        const uint64_t r = pos == 0 ? e.buckets : (before * e.mul_prev + id * e.mul_cur) % e.buckets;
+        big = static_cast<const __nv_bfloat16*>(e.bigram) + r * e.ld;
+    }
+    for (uint32_t i = threadIdx.x; i < e.width; i += blockDim.x) {
+        float v = bad ? 0.f : to_f32(row[i]);
+        if (big) v += to_f32(big[i]);
+        x[static_cast<size_t>(t) * e.width + i] = v;
+    }
+}
+
+// one CTA per row; with a token shift the row before it is recomputed from the same inputs
+template <typename OUT>
+__global__ void __launch_bounds__(256) pre_norm_kernel(const __grid_constant__ hf2q_pre_norm p, uint32_t m, OUT* __restrict__ out, uint32_t ldo,
+                                                       float* __restrict__ h_last) {
+    extern __shared__ float xs[];                          // width, and another width with a shift
+    __shared__ float red[64];
+    pdl_trigger();
+    pdl_wait();
+    const uint32_t t = blockIdx.x;
+    float inv_b = 0.f;
+    float* xb = xs + p.width;
+    if (p.shift && t > 0) inv_b = residual_row(p, t - 1, xb, red);
+    const float inv = residual_row(p, t, xs, red);
+    const uint32_t pos = p.shift ? *p.pos : 0u;
+    for (uint32_t i = threadIdx.x; i < ldo; i += blockDim.x) {
+        float h = 0.f;
+        if (i < p.width) {
+            const float x = xs[i], w = p.norm[i];
+            if (p.x_out) p.x_out[static_cast<size_t>(t) * p.width + i] = x;
+            h = x * inv * w;
+            if (p.shift) {
+                const float b = t > 0 ? xb[i] * inv_b * w : p.shift_state[static_cast<size_t>((pos + 1) & 1) * p.width + i];
+                if (m == 1) p.shift_state[static_cast<size_t>(pos & 1) * p.width + i] = h;
+                else if (t == m - 1) h_last[i] = h;
+                h += (b - h) * p.shift[i];
+            }
+        }
+        out[static_cast<size_t>(t) * ldo + i] = from_f32<OUT>(h);
+    }
+}
+
+template <typename OUT>
+__global__ void __launch_bounds__(256) gated_heads_kernel(const __grid_constant__ hf2q_gated_heads g, OUT* __restrict__ out, uint32_t ldo) {
+    pdl_trigger();
+    pdl_wait();
+    const uint32_t t = blockIdx.x;
+    OUT* row = out + static_cast<size_t>(t) * ldo;
+    for (uint32_t i = g.heads * g.head_dim + threadIdx.x; i < ldo; i += blockDim.x) row[i] = from_f32<OUT>(0.f);
+    gated_heads_row<OUT>(g, t, row, threadIdx.x >> 5, blockDim.x >> 5);
+}
+
+__global__ void __launch_bounds__(256) state_tail_kernel(const uint32_t* __restrict__ pos_dev, uint32_t m, const float* __restrict__ h_last,
+                                                         float* __restrict__ shift_state, uint32_t width, const __grid_constant__ hf2q_delta d,
+                                                         uint32_t channels) {
+    pdl_trigger();
+    pdl_wait();
+    const uint32_t pos = *pos_dev;
+    const uint32_t i = blockIdx.x * blockDim.x + threadIdx.x;
+    if (shift_state && i < width) shift_state[static_cast<size_t>((pos + m - 1) & 1) * width + i] = h_last[i];
+    if (i < channels) {
+        // inputs of the last taps - 1 positions; those before this portion are in the state already
+        const uint32_t qk = d.kv_heads * d.dim;
+        const uint32_t col = i < qk ? d.q_off + i : i < 2 * qk ? d.k_off + (i - qk) : d.v_off + (i - 2 * qk);
+        const uint32_t keep = d.taps - 1 < m ? d.taps - 1 : m;
+        for (uint32_t j = 0; j < keep; ++j) {
+            const uint32_t t = m - 1 - j;
+            d.conv_state[static_cast<size_t>(i) * d.taps + (pos + t) % d.taps] = d.proj[static_cast<size_t>(t) * d.ld + col];
+        }
+    }
+}
+
+}  // namespace
+}  // namespace hf2q
+
+using namespace hf2q;
+using namespace hf2q::seq;
+
+extern "C" {
+
+HF2Q_API int32_t hf2q_cuda_embed(hf2q_ctx* ctx, void* stream, const hf2q_embed* e, const uint32_t* ids, uint32_t m, float* x) {
+    if (!ctx) return HF2Q_ERR_INVALID_ARGUMENT;
+    if (!e || !e->embed || !e->pos || !e->prev || !ids || !x || e->vocab == 0 || e->width == 0 || e->ld < e->width || (e->bigram && e->buckets == 0))
+        return ctx_fail(ctx, HF2Q_ERR_INVALID_ARGUMENT, "embed: null pointer or empty table");
+    if (m == 0) return HF2Q_OK;
+    const cudaError_t r = launch_pdl(embed_kernel, dim3(m), dim3(256), 0, static_cast<cudaStream_t>(stream), *e, ids, m, x, ctx_status_word(ctx));
+    return ctx_cuda_result(ctx, r, "embed", 1);
+}
+
+HF2Q_API int32_t hf2q_cuda_pre_norm(hf2q_ctx* ctx, void* stream, const hf2q_pre_norm* p, uint32_t m, void* out, uint32_t out_dtype, uint32_t ldo,
+                                    float* h_last) {
+    if (!ctx) return HF2Q_ERR_INVALID_ARGUMENT;
+    if (!p || !p->x || !p->norm || !out || p->width == 0 || ldo < p->width || p->x_out == p->x || (p->a && (!p->b || !p->a_norm || !p->b_norm)) ||
+        (p->shift && (!p->shift_state || !p->pos || (m > 1 && !h_last))))
+        return ctx_fail(ctx, HF2Q_ERR_INVALID_ARGUMENT, "pre_norm: null pointer, or x_out is x");
+    if (m == 0) return HF2Q_OK;
+    const size_t smem = static_cast<size_t>(p->width) * (p->shift ? 8 : 4);
+    if (smem > 200 * 1024) return ctx_fail(ctx, HF2Q_ERR_INVALID_ARGUMENT, "pre_norm: width too large");
+    const cudaStream_t st = static_cast<cudaStream_t>(stream);
+    static PerDeviceFlag f32f, bff;
+    cudaError_t e;
+    if (out_dtype == HF2Q_DT_F32) {
+        e = ensure_max_dynamic_smem(pre_norm_kernel<float>, 200 * 1024, f32f);
+        if (e == cudaSuccess) e = launch_pdl(pre_norm_kernel<float>, dim3(m), dim3(256), smem, st, *p, m, static_cast<float*>(out), ldo, h_last);
+    } else if (out_dtype == HF2Q_DT_BF16) {
+        e = ensure_max_dynamic_smem(pre_norm_kernel<__nv_bfloat16>, 200 * 1024, bff);
+        if (e == cudaSuccess) e = launch_pdl(pre_norm_kernel<__nv_bfloat16>, dim3(m), dim3(256), smem, st, *p, m, static_cast<__nv_bfloat16*>(out), ldo, h_last);
+    } else {
+        e = cudaErrorInvalidValue;
+    }
+    return ctx_cuda_result(ctx, e, "pre_norm", 1);
+}
+
+HF2Q_API int32_t hf2q_cuda_gated_heads(hf2q_ctx* ctx, void* stream, const hf2q_gated_heads* g, uint32_t m, void* out, uint32_t out_dtype, uint32_t ldo) {
+    if (!ctx) return HF2Q_ERR_INVALID_ARGUMENT;
+    if (!g || !g->o || !g->gate || !out || ldo < g->heads * g->head_dim) return ctx_fail(ctx, HF2Q_ERR_INVALID_ARGUMENT, "gated_heads: null pointer or a short row");
+    if (m == 0) return HF2Q_OK;
+    const cudaStream_t st = static_cast<cudaStream_t>(stream);
+    cudaError_t e = cudaErrorInvalidValue;
+    if (out_dtype == HF2Q_DT_F32) e = launch_pdl(gated_heads_kernel<float>, dim3(m), dim3(256), 0, st, *g, static_cast<float*>(out), ldo);
+    else if (out_dtype == HF2Q_DT_BF16) e = launch_pdl(gated_heads_kernel<__nv_bfloat16>, dim3(m), dim3(256), 0, st, *g, static_cast<__nv_bfloat16*>(out), ldo);
+    return ctx_cuda_result(ctx, e, "gated_heads", 1);
+}
+
+HF2Q_API int32_t hf2q_cuda_state_tail(hf2q_ctx* ctx, void* stream, const uint32_t* pos, uint32_t m, const float* h_last, float* shift_state,
+                                      uint32_t width, const hf2q_delta* delta) {
+    if (!ctx) return HF2Q_ERR_INVALID_ARGUMENT;
+    if (!pos || m == 0 || (shift_state && !h_last) || (delta && (!delta->proj || !delta->conv_state || delta->taps == 0)))
+        return ctx_fail(ctx, HF2Q_ERR_INVALID_ARGUMENT, "state_tail: null pointer");
+    const uint32_t channels = delta && delta->taps > 1 ? 2 * delta->kv_heads * delta->dim + delta->heads * delta->vdim : 0;
+    const uint32_t n = shift_state && width > channels ? width : channels;
+    if (n == 0) return HF2Q_OK;
+    const hf2q_delta none{};
+    const cudaError_t e = launch_pdl(state_tail_kernel, dim3((n + 255) / 256), dim3(256), 0, static_cast<cudaStream_t>(stream), pos, m, h_last,
+                                     shift_state, width, delta ? *delta : none, channels);
+    return ctx_cuda_result(ctx, e, "state_tail", 1);
+}
+
+}  // extern "C"

@@ -20,6 +20,7 @@ from __future__ import annotations
 import ctypes as C
 from dataclasses import dataclass
 
+import numpy as np
 import torch
 
 from . import _lib, ops
@@ -90,7 +91,72 @@ class _KvCache(C.Structure):           # hf2q_kv_cache in include/hf2q_cuda.h
                 ("n_kv_heads", C.c_uint32), ("head_dim", C.c_uint32), ("max_seq", C.c_uint32)]
 
 
-class LlamaDecoder:
+class GreedyDecoder:
+    """The greedy generation loop over one captured decode step, and the sequence interface the engine drives.
+
+    A decoder supplies ``decode_step`` (device work only: token ``self.tok`` at ``self.pos`` -> next token, position + 1,
+    ``self.logits``), ``extend`` and the slot calls.  ``loop_state`` lists the tensors a step changes in a way that the
+    next step reads, which the warm-up in front of a capture must put back."""
+
+    _graph = None
+
+    def decode_step(self) -> None:
+        raise NotImplementedError
+
+    def loop_state(self) -> list:
+        return [self.pos, self.tok]
+
+    # ---- sequences: open_slot -> extend / generate -> close_slot
+    def open_slot(self) -> int:
+        raise NotImplementedError
+
+    def close_slot(self, slot: int) -> None:
+        raise NotImplementedError
+
+    def bind(self, slot: int) -> None:
+        """Makes ``slot`` the sequence that decode_step, generate and capture work on."""
+
+    def extend(self, slot: int, ids: torch.Tensor, want) -> torch.Tensor:
+        """Runs the sequence's next tokens; logits [len(want), vocab] (f32) at the wanted places among them."""
+        raise NotImplementedError
+
+    def capture(self) -> None:
+        """Captures one decode step into a CUDA graph (after a few eager steps have warmed every kernel up)."""
+        g = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(g):
+            self.decode_step()
+        self._graph = g
+
+    def ensure_graph(self) -> None:
+        if self._graph is None:
+            saved = [t.clone() for t in self.loop_state()]
+            self.decode_step()                        # warm-up outside the capture; state restored below
+            torch.cuda.synchronize(self.dev)
+            self._restore(saved)
+            self.capture()
+            self._restore(saved)
+
+    def _restore(self, saved) -> None:
+        for t, v in zip(self.loop_state(), saved):
+            t.copy_(v)
+
+    def generate(self, n: int, use_graph: bool = True, collect: bool = True):
+        """Greedy decode of n tokens starting from the current (tok, pos) state; returns the generated ids
+        (``collect=False``: nothing is copied out between the steps and None is returned)."""
+        out = torch.empty(n, dtype=torch.int32, device=self.dev) if collect else None
+        if use_graph:
+            self.ensure_graph()
+        for t in range(n):
+            if use_graph:
+                self._graph.replay()
+            else:
+                self.decode_step()
+            if collect:
+                out[t:t + 1].copy_(self.tok)
+        return out
+
+
+class LlamaDecoder(GreedyDecoder):
     def __init__(self, ctx: ops.GpuContext, cfg: LlamaConfig, weights: ModelWeights, prefill_chunk: int = 2048):
         self.ctx, self.cfg, self.w = ctx, cfg, weights
         self.lib = ctx._lib
@@ -130,10 +196,45 @@ class LlamaDecoder:
         self.att_scratch = torch.zeros(max(need.value, 16), dtype=torch.uint8, device=dev)
         self.prefill_chunk = prefill_chunk
         self._pf = None                 # prefill buffers, allocated on first use
-        self._graph = None
+        self._open, self._length = False, 0
         for lw in weights.layers:
             if not ops.quantized_matmul_swiglu_supported(ctx, 1, lw.gate, torch.float32):
                 raise ops.Hf2qError(_lib.ERR_INVALID_ARGUMENT, "gate/up shape does not fit the fused SwiGLU launch")
+
+    @classmethod
+    def from_gguf(cls, ctx: ops.GpuContext, path, max_seq: int = 32768, prefill_chunk: int = 2048) -> "LlamaDecoder":
+        """Loads a GGUF file with the ``llama`` key prefix and tensor names (block bytes unchanged; an absent
+        output.weight means the tied embedding)."""
+        from .gguf import GgufFile
+        with GgufFile(path) as g:
+            md = lambda k, default=None: g.metadata.get("llama." + k, default)
+            n_q, hidden = int(md("attention.head_count")), int(md("embedding_length"))
+            emb = g.tensors["token_embd.weight"]
+            cfg = LlamaConfig(n_layers=int(md("block_count")), hidden=hidden, n_heads=n_q, n_kv_heads=int(md("attention.head_count_kv", n_q)),
+                              head_dim=int(md("attention.key_length", hidden // n_q)), ffn=int(md("feed_forward_length")), vocab=emb.shape[0],
+                              rms_eps=float(md("attention.layer_norm_rms_epsilon", 1e-5)), rope_theta=float(md("rope.freq_base", 10000.0)), max_seq=max_seq)
+
+            def weight(*names):                        # row ranges of one block format back to back: one tensor
+                ti = [g.tensors[n] for n in names]
+                raw = np.concatenate([g.load_tensor(n) for n in names])
+                return ops.load_quant_weight(ctx, raw, ti[0].ggml_type, sum(t.shape[0] for t in ti), ti[0].shape[1])
+
+            def vec(name):
+                return torch.from_numpy(g.load_tensor(name).view(np.float32).copy()).to(torch.device("cuda", ctx.device))
+
+            layers = []
+            for i in range(cfg.n_layers):
+                p = f"blk.{i}."
+                q, k, v = (p + f"attn_{x}.weight" for x in "qkv")
+                t = [g.tensors[n].ggml_type for n in (q, k, v)]
+                if t[0] != t[1]:
+                    raise ops.Hf2qError(_lib.ERR_UNSUPPORTED_TYPE, f"{p}: attn_q and attn_k have different block formats")
+                fused = t[2] == t[0]
+                layers.append(LayerWeights(vec(p + "attn_norm.weight"), weight(q, k, v) if fused else weight(q, k), None if fused else weight(v),
+                                           weight(p + "attn_output.weight"), vec(p + "ffn_norm.weight"), weight(p + "ffn_gate.weight"),
+                                           weight(p + "ffn_up.weight"), weight(p + "ffn_down.weight")))
+            out = "output.weight" if "output.weight" in g.tensors else "token_embd.weight"
+            return cls(ctx, cfg, ModelWeights(weight("token_embd.weight"), layers, vec("output_norm.weight"), weight(out)), prefill_chunk)
 
     # ---- thin wrappers over the C ABI (current stream) -----------------------------------------
     def _s(self):
@@ -202,33 +303,6 @@ class LlamaDecoder:
         qkv = sum(len(self._qkv_segments(lw)) for lw in self.w.layers)                            # one launch per row range of the fused QKV
         return 1 + per_layer * self.cfg.n_layers + qkv + (2 if self.fused_norm else 3)
 
-    def capture(self) -> None:
-        """Captures one decode step into a CUDA graph (after a few eager steps have warmed every kernel up)."""
-        g = torch.cuda.CUDAGraph()
-        with torch.cuda.graph(g):
-            self.decode_step()
-        self._graph = g
-
-    def generate(self, n: int, use_graph: bool = True, collect: bool = True):
-        """Greedy decode of n tokens starting from the current (tok, pos) state; returns the generated ids
-        (``collect=False``: nothing is copied out between the steps and None is returned)."""
-        out = torch.empty(n, dtype=torch.int32, device=self.dev) if collect else None
-        if use_graph and self._graph is None:
-            saved = (self.pos.clone(), self.tok.clone())
-            self.decode_step()                        # warm-up outside the capture; state restored below
-            torch.cuda.synchronize(self.dev)
-            self.pos.copy_(saved[0]); self.tok.copy_(saved[1])
-            self.capture()
-            self.pos.copy_(saved[0]); self.tok.copy_(saved[1])
-        for t in range(n):
-            if use_graph:
-                self._graph.replay()
-            else:
-                self.decode_step()
-            if collect:
-                out[t:t + 1].copy_(self.tok)
-        return out
-
     # ---- prefill: m tokens per chunk through the GEMM path ---------------------------------------
     def _prefill_buffers(self, m):
         if self._pf is None or self._pf["m"] < m:
@@ -240,20 +314,51 @@ class LlamaDecoder:
                         "u": torch.empty((m, c.ffn), **f32)}
         return self._pf
 
-    def prefill(self, ids: torch.Tensor) -> None:
-        """Runs the prompt (int32 ids on the device) from position 0, fills the KV cache, and leaves
-        (tok, pos) = (greedy next token, len(ids)) for ``generate``; self.logits holds the last logits."""
+    # ---- the engine's sequence interface: one sequence at a time --------------------------------
+    n_slots = 1
+
+    def open_slot(self) -> int:
+        if self._open:
+            raise RuntimeError("no free sequence slot")
+        self._open, self._length = True, 0
+        return 0
+
+    def close_slot(self, slot: int) -> None:
+        self._open = False
+
+    def extend(self, slot: int, ids: torch.Tensor, want) -> torch.Tensor:
+        out = torch.empty((len(want), self.cfg.vocab), dtype=torch.float32, device=self.dev)
+        self.prefill(ids, start=self._length, want=list(want), want_out=out)
+        self._length += int(ids.numel())
+        return out
+
+    def _want_logits(self, x, delta, p0, m, start, want, out) -> None:
+        rows = [(j, start + w - p0) for j, w in enumerate(want) if 0 <= start + w - p0 < m]
+        if not rows:
+            return
+        idx = torch.tensor([r for _, r in rows], device=self.dev)
+        xs, n = x.index_select(0, idx), len(rows)
+        xn = torch.empty_like(xs)
+        self._rms(xs, None if delta is None else delta.index_select(0, idx), self.w.out_norm, xn, n)
+        logits = torch.empty((n, self.cfg.vocab), dtype=torch.float32, device=self.dev)
+        ops.quantized_matmul_ggml(self.ctx, xn, self.w.output, logits, self.w.output.matmul_params(n))
+        out[rows[0][0]:rows[0][0] + n].copy_(logits)
+
+    def prefill(self, ids: torch.Tensor, start: int = 0, want=(), want_out=None) -> None:
+        """Runs tokens (int32 ids on the device) from position ``start``, fills the KV cache, and leaves
+        (tok, pos) = (greedy next token, start + len(ids)) for ``generate``; self.logits holds the last logits.
+        ``want``: ascending places among the tokens whose logits go to the rows of ``want_out``."""
         c, ctx, lib = self.cfg, self.ctx, self.lib
-        T = int(ids.numel())
-        if T == 0 or T >= c.max_seq:
-            raise ops.Hf2qError(_lib.ERR_INVALID_ARGUMENT, f"prompt length {T} must be in 1..max_seq-1")
+        T = start + int(ids.numel())
+        if T == start or T >= c.max_seq:
+            raise ops.Hf2qError(_lib.ERR_INVALID_ARGUMENT, f"sequence length {T} must be in 1..max_seq-1 and grow")
         ids = ids.to(self.dev, torch.int32).contiguous()
-        for p0 in range(0, T, self.prefill_chunk):
+        for p0 in range(start, T, self.prefill_chunk):
             m = min(self.prefill_chunk, T - p0)
-            b = self._prefill_buffers(min(self.prefill_chunk, T))
+            b = self._prefill_buffers(min(self.prefill_chunk, T - start))
             x, xn, qkv, att, o, g, u = (b[k][:m] for k in ("x", "xn", "qkv", "att", "o", "g", "u"))
             self.pos.fill_(p0)
-            self._get_rows(ids[p0:p0 + m], m, x)
+            self._get_rows(ids[p0 - start:p0 - start + m], m, x)
             delta = None
             for i, lw in enumerate(self.w.layers):
                 self._rms(x, delta, lw.attn_norm, xn, m)                                   # x += previous layer's FFN output (unfused form)
@@ -282,6 +387,7 @@ class LlamaDecoder:
                     ops.quantized_matmul_ggml(ctx, g, lw.down, o, lw.down.matmul_params(m))
                     delta = o
             self._pf_delta = delta
+            self._want_logits(x, delta, p0, m, start, want, want_out)
             if p0 + m == T:
                 # only the last token's logits are needed: x_last += delta_last, final norm, output head
                 self.x.copy_(x[m - 1:m])

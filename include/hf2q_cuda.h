@@ -643,6 +643,145 @@ HF2Q_API int32_t hf2q_cuda_argmax(hf2q_ctx* ctx, void* stream, const float* logi
 /* residual_add: x[i] += delta[i]. */
 HF2Q_API int32_t hf2q_cuda_add(hf2q_ctx* ctx, void* stream, float* x, const float* delta, uint64_t n);
 
+/* ---- decoder designs with bf16 weights: products, recurrent mixers, windowed attention ------------------ *
+ * Weights are row-major bf16 [n][k], k a multiple of 8 (pad with zero columns), 16-byte aligned.  Activations are
+ * f32, or bf16 in front of the tensor-core product.  x f32 and no tensor-core use = every step in 32-bit. */
+enum { HF2Q_EPI_NONE = 0, HF2Q_EPI_GELU = 1, HF2Q_EPI_ADD = 2, HF2Q_EPI_SOFTCAP = 3 };
+
+/* y[m][n] = epilogue(x[m][k] . w^T), rows of x / y are ldx / ldy elements apart.  m <= 8: mat-vec kernel (fp32
+ * arithmetic); more rows: tcgen05 for bf16 x, a CUDA-core fp32 product for f32 x.  ADD: + residual (layout of y, may
+ * be y); GELU: tanh form; SOFTCAP: cap * tanh(y / cap).  y_dtype f32 or bf16. */
+HF2Q_API int32_t hf2q_cuda_dense_matmul(hf2q_ctx* ctx, void* stream, const void* x, uint32_t x_dtype, uint32_t ldx,
+                                        const void* w, void* y, uint32_t y_dtype, uint32_t ldy, uint32_t m, uint32_t n,
+                                        uint32_t k, uint32_t epilogue, const float* residual, float cap);
+
+/* What stands in front of a layer's product.  Residual update: x + (rms(a) a_norm + rms(b) b_norm) / 2 if a != NULL,
+ * + add0 if not NULL, + step (one row) if not NULL; stored to x_out if not NULL (must not alias x).  Then
+ * h = x / rms(x) * norm, and with shift != NULL the token shift h + (h_before - h) * shift.  shift_state f32
+ * [2][width]: the un-shifted h of position p in row p & 1 (zeros before the first token). */
+typedef struct hf2q_pre_norm {
+    const float *x, *a, *b, *a_norm, *b_norm, *add0, *step;
+    float* x_out;
+    const float *norm, *shift;
+    float* shift_state;
+    const uint32_t* pos;     /* device: position of row 0 */
+    float eps;
+    uint32_t width;
+} hf2q_pre_norm;
+/* out[m][ldo] (f32 or bf16; columns width .. ldo zeroed).  m > 1: the un-shifted h of the last row goes to h_last and
+ * hf2q_cuda_state_tail moves it into shift_state; m == 1 updates shift_state itself. */
+HF2Q_API int32_t hf2q_cuda_pre_norm(hf2q_ctx* ctx, void* stream, const hf2q_pre_norm* p, uint32_t m, void* out,
+                                    uint32_t out_dtype, uint32_t ldo, float* h_last);
+
+/* (norm ? o / rms over the head * norm : o) * sigmoid(gate), per head; norm_all: the weight has heads * head_dim
+ * elements, else head_dim shared by the heads. */
+typedef struct hf2q_gated_heads {
+    const float *o, *gate, *norm;
+    uint32_t ldo, ldg, heads, head_dim, norm_all;
+    float eps;
+} hf2q_gated_heads;
+HF2Q_API int32_t hf2q_cuda_gated_heads(hf2q_ctx* ctx, void* stream, const hf2q_gated_heads* g, uint32_t m, void* out,
+                                       uint32_t out_dtype, uint32_t ldo);
+
+/* One-row products with their prologue and epilogue in the same launch (f32 arithmetic); up to two segments with
+ * the same kind of prologue run side by side. */
+enum { HF2Q_PRO_NONE = 0, HF2Q_PRO_NORM = 1, HF2Q_PRO_GATED = 2 };
+typedef struct hf2q_matvec {
+    const void* w;
+    float* y;
+    const float* residual;
+    const float* x;          /* PRO_NONE */
+    hf2q_pre_norm pre;       /* PRO_NORM */
+    hf2q_gated_heads gated;  /* PRO_GATED */
+    uint32_t n, k, epilogue;
+    float cap;
+} hf2q_matvec;
+HF2Q_API int32_t hf2q_cuda_dense_matvec(hf2q_ctx* ctx, void* stream, uint32_t prologue, const hf2q_matvec* segs,
+                                        uint32_t n_segs);
+
+/* x[t,:] = embed[ids[t],:] (+ bigram[(before * mul_prev + ids[t] * mul_cur) mod buckets,:]; the first token of a sequence takes row
+ * `buckets`).  prev: the token in front of ids[0]; left holding ids[m - 1].  embed / bigram bf16, bigram may be NULL. */
+typedef struct hf2q_embed {
+    const void *embed, *bigram;
+    uint32_t vocab, width, ld, buckets;   /* ld: elements between rows of both tables */
+    uint64_t mul_prev, mul_cur;
+    const uint32_t* pos;
+    uint32_t* prev;
+} hf2q_embed;
+HF2Q_API int32_t hf2q_cuda_embed(hf2q_ctx* ctx, void* stream, const hf2q_embed* e, const uint32_t* ids, uint32_t m, float* x);
+
+/* Sliding-window attention over a ring cache: position p lives in slot p % capacity.  Query head h reads KV head
+ * h / (heads / kv_heads); key j is visible to i when 0 <= i - j < window.  score = (q . k) * scale
+ * - r1[h] ln(1 + r2[h] (i - j)) (r1 NULL: no distance term); q and k are first divided by their root mean square and
+ * multiplied with q_norm / k_norm (NULL: taken as they are).  qkv rows are ld floats apart, at the three offsets. */
+typedef struct hf2q_window_attn {
+    const float* qkv;
+    uint32_t ld, q_off, k_off, v_off;
+    const float *q_norm, *k_norm, *r1, *r2;
+    void *k_cache, *v_cache;              /* [kv_heads][capacity][dim or vdim, padded to 8], f32 or bf16 (cache_dtype) */
+    uint32_t heads, kv_heads, dim, vdim, window, capacity, cache_dtype;
+    float scale, eps;
+    const uint32_t* pos;
+} hf2q_window_attn;
+HF2Q_API int32_t hf2q_cuda_window_attn_scratch_bytes(hf2q_ctx* ctx, const hf2q_window_attn* a, uint64_t* out);
+/* One token: append and attend in one launch.  out f32 [heads * vdim]; scratch zeroed once when allocated. */
+HF2Q_API int32_t hf2q_cuda_window_attn_decode(hf2q_ctx* ctx, void* stream, const hf2q_window_attn* a, float* out,
+                                              void* scratch, uint64_t scratch_bytes);
+/* m tokens (window - 1 + m <= capacity): normalised queries to q_out ([m][heads][dim padded to 8], cache_dtype), keys
+ * and values to the cache. */
+HF2Q_API int32_t hf2q_cuda_window_attn_append(hf2q_ctx* ctx, void* stream, const hf2q_window_attn* a, uint32_t m, void* q_out);
+/* ... then attention times sigmoid(gate) (gate NULL: plain) -> out [m][ldo], f32 or bf16. */
+HF2Q_API int32_t hf2q_cuda_window_attn_prefill(hf2q_ctx* ctx, void* stream, const hf2q_window_attn* a, uint32_t m,
+                                               const void* q, const float* gate, uint32_t ldg, void* out,
+                                               uint32_t out_dtype, uint32_t ldo);
+
+/* Matrix memory with exponential input / forget gates and a running maximum (mLSTM), m tokens from the carried state.
+ * Rows of proj (ld apart) hold q, k [heads][dim], v [heads][vdim] and the raw gates i, f [heads] at their offsets; q is
+ * scaled by dim^-1/2, the gates are capped: i = cap tanh((i + i_bias) / cap), f = logsigmoid(cap tanh((f + f_bias) / cap)).
+ * State, f32: s [heads][vdim][dim padded to 32], n [heads][slices][same], mx [heads][slices], slices = ceil(vdim / 16).
+ * out f32 [m][heads * vdim]. */
+typedef struct hf2q_mlstm {
+    const float* proj;
+    uint32_t ld, q_off, k_off, v_off, i_off, f_off;
+    const float *i_bias, *f_bias;
+    float *s, *n, *mx;
+    uint32_t heads, dim, vdim;
+    float gate_cap;
+} hf2q_mlstm;
+HF2Q_API int32_t hf2q_cuda_mlstm(hf2q_ctx* ctx, void* stream, const hf2q_mlstm* a, uint32_t m, float* out);
+
+/* Gated delta rule with one decay per head and key channel.  Rows of proj hold q, k [kv_heads][dim], v [heads][vdim],
+ * beta logits b [heads] and the low-rank activations a1, g1 [rank] at their offsets.  q, k, v pass a causal depth-wise
+ * convolution (weights f32 [channels][taps]) and SiLU; q, k become unit vectors per head, q times dim^-1/2.
+ * conv_state f32 [2 kv_heads dim + heads vdim][taps]: the input of position p in column p % taps.
+ * decay = exp(-exp(a_log[h]) softplus(a2 . a1 + dt_bias)); gate = g2 . g1 (the sigmoid is hf2q_cuda_gated_heads').
+ * State f32 s [heads][vdim][dim padded to 32]. */
+typedef struct hf2q_delta {
+    const float* proj;
+    uint32_t ld, q_off, k_off, v_off, b_off, a1_off, g1_off;
+    const float *q_conv, *k_conv, *v_conv, *a_log, *dt_bias;
+    const void *a2, *g2;                  /* bf16 [heads * dim][rank_ld], [heads * vdim][rank_ld] */
+    float *conv_state, *s;
+    uint32_t heads, kv_heads, dim, vdim, taps, a_rank_ld, g_rank_ld;
+    const uint32_t* pos;
+} hf2q_delta;
+/* One token, everything in one launch: out, gate f32 [heads * vdim]. */
+HF2Q_API int32_t hf2q_cuda_delta_step(hf2q_ctx* ctx, void* stream, const hf2q_delta* a, float* out, float* gate);
+/* m tokens: convolution, SiLU and unit norms -> qkv f32 [m][2 kv_heads dim + heads vdim] (q, k, v), sigmoid(b) -> beta
+ * [m][heads], the low-rank activations -> a1, g1 [m][rank_ld] (lr_dtype). */
+HF2Q_API int32_t hf2q_cuda_delta_prep(hf2q_ctx* ctx, void* stream, const hf2q_delta* a, uint32_t m, float* qkv, float* beta,
+                                      void* a1, void* g1, uint32_t lr_dtype);
+/* decay logits (a2 . a1, f32 [m][heads * dim]) -> decays, in place. */
+HF2Q_API int32_t hf2q_cuda_delta_decay(hf2q_ctx* ctx, void* stream, const hf2q_delta* a, uint32_t m, float* g);
+/* the recurrence over m tokens; out f32 [m][heads * vdim]. */
+HF2Q_API int32_t hf2q_cuda_delta_scan(hf2q_ctx* ctx, void* stream, const hf2q_delta* a, uint32_t m, const float* qkv,
+                                      const float* beta, const float* g, float* out);
+
+/* After a portion of m > 1 tokens: h_last -> shift_state row (pos + m - 1) & 1 (shift_state NULL: none), and the last
+ * convolution inputs -> delta->conv_state (delta NULL: none). */
+HF2Q_API int32_t hf2q_cuda_state_tail(hf2q_ctx* ctx, void* stream, const uint32_t* pos, uint32_t m, const float* h_last,
+                                      float* shift_state, uint32_t width, const hf2q_delta* delta);
+
 /* ---- introspection ------------------------------------------------------------------------ */
 
 /* Number of kernels this library has launched through `ctx` since creation (the reference keeps
