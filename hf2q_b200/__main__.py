@@ -31,7 +31,7 @@ def trace(args) -> int:
     """Reads one JSON object a line: {"step": n, "entries": [{"id", "tokens", "want"}], "end": [ids]}; writes the wanted
     logits of a step to OUT/<step>.f32 (little-endian f32) and answers "done <step>"."""
     from .engine import Engine, Entry
-    ctx, model = _model(args, args.max_tokens, 1)
+    ctx, model = _model(args, args.max_tokens, 4)
     engine, out = Engine(model), Path(args.out)
     for line in sys.stdin:
         if not line.strip():

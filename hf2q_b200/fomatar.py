@@ -76,7 +76,7 @@ class FomatarConfig:
 
     @property
     def bigram(self):
-        return self.raw.get("embedding", {}).get("bigram")
+        return (self.raw.get("embedding") or {}).get("bigram")
 
     def runs(self) -> list[Run]:
         n, lp = len(self.layers), self.loop

@@ -30,7 +30,7 @@ def gelu_tanh(x):
 def embedding(cfg, w, tokens):
     """Token rows plus the row of (previous token, token) in the hashed bigram table."""
     x = w["embed"][tokens]
-    bg = cfg.get("embedding", {}).get("bigram")
+    bg = (cfg.get("embedding") or {}).get("bigram")
     if bg:
         rows = [bg["buckets"]]
         for a, b in zip(tokens[:-1], tokens[1:]):
