@@ -698,6 +698,236 @@ def bench_decode(hq, oracle, torch, ctx, dev, args) -> dict:
             "host_seconds_building_weights": round(t_build, 1), "eager_launches_seen": int(ctx.launch_count - l0), "clocks": clocks}
 
 
+FOMATAR_SIZES = {        # width, heads, KV heads, memory heads, feed-forward, window
+    "2048": (2048, 16, 4, 8, 6144, 2048),
+    "4096": (4096, 32, 8, 16, 14336, 4096),
+}
+
+
+def fomatar_config(size: str, layers: int, vocab: int) -> dict:
+    """Layers of a real model's proportions, mixers alternating: windowed attention beside an mLSTM memory, gated delta rule."""
+    w, h, g, rh, ff, window = FOMATAR_SIZES[size]
+    par = {"type": "parallel", "mlp": {"kind": "dense", "ff": ff},
+           "mixer": {"left": {"heads": h, "kv_heads": g, "dim": 128, "vdim": 128, "mask": {"size": window}, "scale": 128 ** -0.5},
+                     "right": {"heads": rh, "dim": 128, "vdim": 128, "gate_cap": 15.0}}}
+    dlt = {"type": "channel_delta", "mlp": {"kind": "dense", "ff": ff}, "mixer": {"heads": h, "kv_heads": h // 2, "dim": 128, "vdim": 128, "conv": 4}}
+    return {"architecture": "Fomatar", "width": w, "vocab": vocab, "norm": {"eps": 1e-5}, "logit_softcap": 30.0,
+            "embedding": {"bigram": {"buckets": 65521, "mul_prev": 1000003, "mul_cur": 8191}}, "layers": [par if i % 2 == 0 else dlt for i in range(layers)],
+            "loop": None}
+
+
+def fomatar_tensors(torch, cfg, rank=128):
+    """get(name) drawing each tensor when it is asked for (bf16 N(0, 1/sqrt(k)); norms one; gates and decays moderate)."""
+    w, shapes = cfg["width"], {"embed": (cfg["vocab"], cfg["width"]), "bigram": (cfg["embedding"]["bigram"]["buckets"] + 1, cfg["width"]),
+                               "head": (cfg["vocab"], cfg["width"]), "final.norm": (cfg["width"],)}
+    for i, e in enumerate(cfg["layers"]):
+        p, m = f"l{i}.mix.", e["mixer"]
+        for n in ("norm1", "norm2", "shift"):
+            shapes[f"l{i}.{n}"] = (w,)
+        shapes |= {f"l{i}.mlp.up": (e["mlp"]["ff"], w), f"l{i}.mlp.down": (w, e["mlp"]["ff"])}
+        if e["type"] == "parallel":
+            L, R = m["left"], m["right"]
+            a, b, c, d, r = L["heads"] * L["dim"], L["kv_heads"] * L["dim"], L["kv_heads"] * L["vdim"], L["heads"] * L["vdim"], R["heads"]
+            shapes |= {p + "left.q": (a, w), p + "left.k": (b, w), p + "left.v": (c, w), p + "left.g": (d, w), p + "left.o": (w, d), p + "left.out": (w,),
+                       p + "left.q.norm": (L["dim"],), p + "left.k.norm": (L["dim"],), p + "left.r1": (L["heads"],), p + "left.r2": (L["heads"],),
+                       p + "right.q": (r * R["dim"], w), p + "right.k": (r * R["dim"], w), p + "right.v": (r * R["vdim"], w), p + "right.g": (r * R["vdim"], w),
+                       p + "right.o": (w, r * R["vdim"]), p + "right.out": (w,), p + "right.norm": (r * R["vdim"],), p + "right.i": (r, w),
+                       p + "right.f": (r, w), p + "right.i.b": (r,), p + "right.f.b": (r,)}
+        else:
+            H, G, d, dv, K = m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["conv"]
+            shapes |= {p + "q": (G * d, w), p + "k": (G * d, w), p + "v": (H * dv, w), p + "q.conv": (G * d, K), p + "k.conv": (G * d, K),
+                       p + "v.conv": (H * dv, K), p + "b": (H, w), p + "A_log": (H,), p + "dt_bias": (H * d,), p + "a1": (rank, w), p + "a2": (H * d, rank),
+                       p + "g1": (rank, w), p + "g2": (H * dv, rank), p + "norm": (dv,), p + "o": (w, H * dv)}
+    g = torch.Generator(device="cuda").manual_seed(0)
+
+    def get(name):
+        s = shapes[name]
+        leaf = name.rsplit(".", 1)[-1]
+        if len(s) == 1:
+            t = torch.full(s, 1.0 if leaf in ("norm", "norm1", "norm2", "out") else -2.0 if leaf in ("A_log", "dt_bias") else 0.3)
+        else:
+            t = torch.randn(s, generator=g, device="cuda") * (1.0 if leaf in ("embed", "bigram") else s[-1] ** -0.5)
+        return t.to(torch.bfloat16).cpu()
+    return get
+
+
+class _CallLog:
+    """Records the C-ABI calls of a decoder step so that one kind of kernel can be timed alone, over all its layers."""
+
+    def __init__(self, sop):
+        self.sop, self.calls = sop, []
+
+    def __enter__(self):
+        self._orig = self.sop._call
+
+        def call(name, *a):
+            self.calls.append((name, a))
+            self._orig(name, *a)
+        self.sop._call = call
+        return self
+
+    def __exit__(self, *exc):
+        self.sop._call = self._orig
+
+    def time(self, torch, name, reps=20):
+        calls = [a for n, a in self.calls if n == name]
+        if not calls:
+            return None, []
+
+        def run():
+            for a in calls:
+                self._orig(name, *a)
+        return _timed(torch, _graph_of(torch, run).replay, reps), calls
+
+
+def bench_fomatar(hq, oracle, torch, ctx, dev, args) -> dict:
+    """The Fomatar design beside the quantized Llama decoder at equal width, heads, head size, feed-forward and depth:
+    prefill and decode throughput, and every kernel alone against its roofline.  Random weights, four layers (0.9 to
+    2.4 GB of them: larger than L2), 8192-token prompts in portions of 2048."""
+    from hf2q_b200 import decoder as D
+    from hf2q_b200.fomatar import FomatarConfig, FomatarDecoder
+    hbm, kind = measured_hbm_peak()
+    _, burst, _ = measured_tensor_peaks()
+    layers, vocab, n_prompt, n_new, chunk = 4, 32768, (args.tokens or 8192), 100, 2048
+    sampler = ClockSampler(ctx.device)
+    sampler.start()
+    l0, sizes = ctx.launch_count, {}
+
+    def timed_once(fn):
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        e0.record()
+        fn()
+        e1.record()
+        torch.cuda.synchronize()
+        return e0.elapsed_time(e1) * 1e-3
+
+    def throughput(model):
+        ids = torch.randint(0, vocab, (n_prompt,), dtype=torch.int32, device=dev, generator=torch.Generator(device=dev).manual_seed(0))
+        best = 1e9
+        for _ in range(4):
+            slot = model.open_slot()
+            model.bind(slot)
+            best = min(best, timed_once(lambda: model.extend(slot, ids, [])))
+            model.close_slot(slot)
+        slot = model.open_slot()
+        model.extend(slot, ids, [])
+        model.bind(slot)
+        model.generate(8, collect=False)
+        dt = timed_once(lambda: model.generate(n_new, collect=False))
+        ctx.check_status()
+        assert bool(torch.isfinite(model.logits).all())
+        return {"prefill_tok_s": round(n_prompt / best), "decode_tok_s": round(n_new / dt, 1), "decode_us_per_token": round(1e6 * dt / n_new, 1)}, slot
+
+    for size, (w, h, g, rh, ff, window) in FOMATAR_SIZES.items():
+        cfg = fomatar_config(size, layers, vocab)
+        model = FomatarDecoder(ctx, FomatarConfig(cfg), fomatar_tensors(torch, cfg), max_seq=n_prompt + 1024, prefill_chunk=chunk)
+        ours, slot = throughput(model)
+        per_token = model.decode_bytes_per_token()
+        ours["decode_frac_of_hbm_roofline"] = round(per_token / (ours["decode_us_per_token"] * 1e-6) / 1e9 / hbm, 3)
+        kernels = {}
+        # one decode step, kind by kind
+        with _CallLog(model.sop) as log:
+            model.decode_step()
+        n_par = layers // 2
+        st = 2 * 4 * 128 * 128
+        work = {"dense_matvec": sum(r.nbytes for l in model.layers for r in (l.mixer.proj, l.up, l.down)) + model.head.nbytes +
+                sum(l.mixer.lo.nbytes + l.mixer.ro.nbytes if l.mixer.combines else l.mixer.o.nbytes for l in model.layers),
+                "window_attn_decode": n_par * window * g * 256 * 2, "mlstm": n_par * rh * st,
+                "delta_step": n_par * (h * st + model.layers[1].mixer.a2.nbytes + model.layers[1].mixer.g2.nbytes)}
+        for name, nbytes in work.items():
+            dt, calls = log.time(torch, name)
+            kernels["decode " + name] = {"us": round(1e6 * dt / len(calls), 2), "GB/s": round(nbytes / dt / 1e9), "frac": round(nbytes / dt / 1e9 / hbm, 3)}
+        # one portion deep in a prompt
+        ids = torch.randint(0, vocab, (chunk,), dtype=torch.int32, device=dev)
+        model.pos.fill_(n_prompt - chunk)
+        with _CallLog(model.sop) as log:
+            model._portion(ids, chunk)
+        seen = sum(min(window, n_prompt - chunk + i + 1) for i in range(chunk))
+        flop = {"dense_matmul": 2 * chunk * sum(r.n * r.k for l in model.layers for r in (l.mixer.proj, l.up, l.down)) + 2 * chunk * sum(
+                    l.mixer.lo.n * l.mixer.lo.k + l.mixer.ro.n * l.mixer.ro.k if l.mixer.combines else
+                    l.mixer.o.n * l.mixer.o.k + l.mixer.a2.n * l.mixer.a2.k + l.mixer.g2.n * l.mixer.g2.k for l in model.layers),
+                "window_attn_prefill": n_par * seen * h * 2 * 256}
+        for name, fl in flop.items():
+            dt, calls = log.time(torch, name, 10)
+            kernels["prefill " + name] = {"us": round(1e6 * dt / len(calls), 1), "TFLOP/s": round(fl / dt / 1e12, 1), "frac": round(fl / dt / 1e12 / burst, 3)}
+        # the recurrences: bytes of their operands, each read or written once
+        io = {"mlstm": n_par * chunk * rh * 128 * 4 * 4, "delta_scan": n_par * chunk * (h // 2 * 2 + h * 3) * 128 * 4,
+              "delta_prep": n_par * chunk * (h // 2 * 2 + h) * 128 * 8, "delta_decay": n_par * chunk * h * 128 * 8, "gated_heads": chunk * 10 * 128 * n_par * (rh + h),
+              "pre_norm": chunk * w * 4 * (n_par * (1 + 0.5 + 4 + 0.5) + n_par * (1 + 0.5 + 1 + 0.5)), "window_attn_append": n_par * chunk * (h + 2 * g) * 128 * 6}
+        for name, nbytes in io.items():
+            dt, calls = log.time(torch, name, 10)
+            kernels["prefill " + name] = {"us": round(1e6 * dt / len(calls), 1), "GB/s": round(nbytes / dt / 1e9), "frac": round(nbytes / dt / 1e9 / hbm, 3)}
+        model.close_slot(slot)
+        del model, log
+        torch.cuda.empty_cache()
+
+        lc = D.LlamaConfig(n_layers=layers, hidden=w, n_heads=h, n_kv_heads=g, head_dim=128, ffn=ff, vocab=vocab, max_seq=n_prompt + 1024)
+        llama = D.LlamaDecoder(ctx, lc, build_llama_weights(hq, oracle, torch, ctx, dev, lc), prefill_chunk=chunk)
+        theirs, slot = throughput(llama)
+        theirs["decode_frac_of_hbm_roofline"] = round((llama.weight_bytes_per_token() + llama.kv_bytes_per_position() * n_prompt) /
+                                                      (theirs["decode_us_per_token"] * 1e-6) / 1e9 / hbm, 3)
+        like = {}
+        qkv = torch.randn((chunk, (h + 2 * g) * 128), device=dev)
+        att = torch.empty((chunk, h * 128), device=dev)
+        llama.pos.fill_(n_prompt - chunk)
+        import ctypes as C
+
+        def all_attn():
+            for kv in llama.kv:
+                ctx._check(ctx._lib.hf2q_cuda_attn_prefill(ctx._h, ctx._stream(), qkv.data_ptr(), chunk, h, C.byref(kv), n_prompt - chunk, att.data_ptr(), 0))
+        dt = _timed(torch, _graph_of(torch, all_attn).replay, 5) / layers
+        fl = sum(n_prompt - chunk + i + 1 for i in range(chunk)) * h * 2 * 256
+        like["prefill attention"] = {"us": round(1e6 * dt, 1), "TFLOP/s": round(fl / dt / 1e12, 1), "frac": round(fl / dt / 1e12 / burst, 3)}
+        row = torch.randn((1, (h + 2 * g) * 128), device=dev)
+
+        def all_dec():
+            for kv in llama.kv:
+                ctx._check(ctx._lib.hf2q_cuda_attn_decode_fused(ctx._h, ctx._stream(), row.data_ptr(), h, 5e5, C.byref(kv), llama.pos.data_ptr(), llama.att.data_ptr(),
+                                                                hq.ops.DT_F32, llama.att_scratch.data_ptr(), llama.att_scratch.numel()))
+        llama.pos.fill_(window - 1)                                   # as many cached positions as our window holds
+        dt = _timed(torch, _graph_of(torch, all_dec).replay, 20) / layers
+        nb = 2 * g * window * 132
+        like["decode attention"] = {"us": round(1e6 * dt, 2), "GB/s": round(nb / dt / 1e9), "frac": round(nb / dt / 1e9 / hbm, 3)}
+        x = torch.randn((chunk, w), device=dev)
+        xb, hid = x.to(torch.bfloat16), torch.randn((chunk, ff), device=dev).to(torch.bfloat16)
+        yf, yw = torch.empty((chunk, ff), device=dev), torch.empty((chunk, w), device=dev)
+        x1, y1, z1, h1 = x[:1].contiguous(), torch.empty((1, ff), device=dev), torch.empty((1, w), device=dev), torch.randn((1, ff), device=dev)
+        ws = torch.empty(chunk * ff * 2 + 4096, dtype=torch.uint8, device=dev)
+
+        def products():
+            for lw in llama.w.layers:
+                for wt in (lw.gate, lw.up):
+                    hq.quantized_matmul_ggml(ctx, xb, wt, yf, wt.matmul_params(chunk), ws)
+                hq.quantized_matmul_ggml(ctx, hid, lw.down, yw, lw.down.matmul_params(chunk), ws)
+        dt = _timed(torch, _graph_of(torch, products).replay, 5)
+        fl = layers * 3 * 2 * chunk * w * ff
+        like["prefill products"] = {"us": round(1e6 * dt / (3 * layers), 1), "TFLOP/s": round(fl / dt / 1e12, 1), "frac": round(fl / dt / 1e12 / burst, 3)}
+
+        def vecs():
+            for lw in llama.w.layers:
+                for wt in (lw.gate, lw.up):
+                    hq.quantized_matmul_ggml(ctx, x1, wt, y1, wt.matmul_params(1))
+                hq.quantized_matmul_ggml(ctx, h1, lw.down, z1, lw.down.matmul_params(1))
+        dt = _timed(torch, _graph_of(torch, vecs).replay, 20)
+        nb = sum(t.nbytes for lw in llama.w.layers for t in (lw.gate, lw.up, lw.down))
+        like["decode products"] = {"us": round(1e6 * dt / (3 * layers), 2), "GB/s": round(nb / dt / 1e9), "frac": round(nb / dt / 1e9 / hbm, 3)}
+        nw = torch.ones(w, device=dev)
+        dt = _timed(torch, _graph_of(torch, lambda: [llama._rms(x, yw, nw, torch.empty_like(x), chunk) for _ in range(4)]).replay, 10) / 4
+        like["prefill rms_norm"] = {"us": round(1e6 * dt, 1), "GB/s": round(chunk * w * 16 / dt / 1e9), "frac": round(chunk * w * 16 / dt / 1e9 / hbm, 3)}
+        llama.close_slot(slot)
+        sizes[size] = {"fomatar": ours, "llama": theirs, "fomatar_kernels": kernels, "llama_like_kernels": like}
+        del llama
+        torch.cuda.empty_cache()
+    big = sizes["4096"]["fomatar"]
+    return {"metric": "Fomatar decode tok/s", "value": big["decode_tok_s"], "unit": "tok/s", "higher_is_better": True, "dtype": "bf16 weights and operands, f32 accumulate and state",
+            "config": {"workload": f"{layers} layers (two windowed attention + mLSTM, two gated delta), widths {', '.join(FOMATAR_SIZES)}, vocab {vocab}; prefill of {n_prompt} tokens in "
+                                   f"portions of {chunk}, then {n_new} greedy tokens from one CUDA graph; beside the Q4_K_M Llama decoder at equal width, heads, feed-forward and depth",
+                       "timing": "CUDA events; kernels alone from a CUDA graph of their calls over all layers (weights larger than L2)"},
+            "sizes": sizes, "roofline": {"hbm_gbs": hbm, "bf16_tflops_burst": burst, "peak_source": f"of {kind}"},
+            "gpu_launches": int(ctx.launch_count - l0), "clocks": sampler.stop()}
+
+
 def run_secondary(args) -> None:
     """One of the other workloads alone on one GPU: one JSON line."""
     import torch
@@ -717,6 +947,8 @@ def run_secondary(args) -> None:
         line = bench_config1(hq, oracle, torch, ctx, dev, args)
     elif args.workload == "decode":
         line = bench_decode(hq, oracle, torch, ctx, dev, args)
+    elif args.workload == "fomatar":
+        line = bench_fomatar(hq, oracle, torch, ctx, dev, args)
     elif args.workload == "attention":
         line = bench_attention(hq, oracle, torch, ctx, dev, args)
     else:
@@ -742,9 +974,10 @@ def main() -> None:
     ap.add_argument("--no-strong", action="store_true", help="several GPUs: skip the strong-scaling leg")
     ap.add_argument("--no-graph", action="store_true", help="issue launches eagerly instead of replaying a CUDA graph")
     ap.add_argument("--qtype", default="", help="matvec: one ggml type number (2, 8, 12, 13, 14) instead of all five")
-    ap.add_argument("--workload", default="gemv", choices=["gemv", "gemm", "moe", "matvec", "config1", "decode", "attention"],
+    ap.add_argument("--workload", default="gemv", choices=["gemv", "gemm", "moe", "matvec", "config1", "decode", "attention", "fomatar"],
                     help="gemv: the headline Q6_K decode sweep (default, carries the others as `secondary`); gemm: Q4_K_M prefill "
-                         "GEMM sweep; moe: Qwen3-style A3B expert layer (Q5_K mul_mat_id); matvec: all block formats; config1: Q4_K 4096^2 f32")
+                         "GEMM sweep; moe: Qwen3-style A3B expert layer (Q5_K mul_mat_id); matvec: all block formats; config1: Q4_K 4096^2 f32; "
+                         "fomatar: the bf16 design with recurrent mixers beside the quantized decoder at equal size")
     ap.add_argument("--tokens", type=int, default=0, help="gemm/moe: one token count instead of the sweep")
     args = ap.parse_args()
     if args.warmup < 3:

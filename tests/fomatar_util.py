@@ -104,7 +104,20 @@ def oracle_logits(cfg, w, ids):
     return F.forward(cfg, as_f64(w), ids)
 
 
-def error(got, want):
-    """Root mean square difference over the vocabulary, largest position, in units of the logits' own spread."""
+def errors(got, want):
+    """Root mean square difference over the vocabulary at every position, in units of the logits' own spread."""
     got = got.detach().cpu().double().numpy() if isinstance(got, torch.Tensor) else got
-    return float((np.sqrt(((got - want) ** 2).mean(-1)) / want.std()).max())
+    return np.sqrt(((got - want) ** 2).mean(-1)) / want.std()
+
+
+def error(got, want):
+    return float(errors(got, want).max())
+
+
+def close(got, want, dtype):
+    """f32: every position to rounding.  bf16: product operands carry 8 bits, and an mLSTM quotient whose denominator is
+    near its floor magnifies that at single positions, so those have room while nineteen of twenty have little."""
+    e = errors(got, want)
+    if dtype == torch.float32:
+        return e.max() < 1e-4
+    return np.quantile(e, 0.95) < 6e-2 and e.max() < 0.3

@@ -19,8 +19,7 @@ from tests import fomatar_util as U
 
 pytestmark = pytest.mark.gpu
 ROOT = Path(__file__).resolve().parent.parent
-# f32: rounding only; bf16: operands of every product carry 8 bits, three to eight layers deep
-TOL = {torch.float32: 1e-4, torch.bfloat16: 6e-2}
+TOL = {torch.float32: 1e-4}
 LEN = {"a": 190, "b": 120, "c": 330}
 
 
@@ -65,7 +64,7 @@ def test_prompt_portions_and_single_tokens(gpu_ctx, name, dtype):
     ids, want = want_of(name, LEN[name])
     n = len(ids)
     for cuts in ([n], [1] * n, cuts_of(n, [3, 64, 2, 2, 7, 1]), cuts_of(n, [2]), [n - 5] + [1] * 5):
-        assert U.error(run(m, ids, cuts), want) < TOL[dtype], cuts[:6]
+        assert U.close(run(m, ids, cuts), want, dtype), cuts[:6]
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
@@ -79,7 +78,7 @@ def test_every_layer_run(gpu_ctx, dtype):
     F.forward(cfg, U.as_f64(w), ids, want)
     assert len(got) == len(want) == len(m.runs)
     for r, (a, b) in enumerate(zip(got, want)):
-        assert U.error(a, b) < TOL[dtype], r
+        assert U.close(a, b, dtype), r
 
 
 def test_internal_chunks_do_not_show(gpu_ctx):
@@ -147,7 +146,7 @@ def test_interleaved_sequences_and_reused_slots(gpu_ctx, dtype):
             if waiting:
                 live.append(waiting.pop(0))
     for i, (_, want) in seqs.items():
-        assert U.error(torch.cat(rows[i]), want) < TOL[dtype], i
+        assert U.close(torch.cat(rows[i]), want, dtype), i
     # in a reused slot a sequence gives the very bits it gives alone
     fresh, _, _ = load(gpu_ctx, "a", dtype)
     ids = seqs["s"][0]
@@ -240,10 +239,10 @@ def test_trace_runner_replays_portions(folder, tmp_path, dtype):
         c = len(s["entries"][0]["tokens"])
         if s["entries"][0]["want"]:
             got = np.fromfile(tmp_path / f"{s['step']}.f32", "<f4").reshape(c, -1)
-            assert U.error(got.astype(np.float64), want[at:at + c]) < TOL[getattr(torch, dtype)]
+            assert U.close(got.astype(np.float64), want[at:at + c], getattr(torch, dtype))
         at += c
     got = np.fromfile(tmp_path / f"{len(steps) - 1}.f32", "<f4")[None]
-    assert U.error(got.astype(np.float64), want[8:9]) < TOL[getattr(torch, dtype)]
+    assert U.close(got.astype(np.float64), want[8:9], getattr(torch, dtype))
 
 
 def test_llama_through_the_same_registry_and_engine(gpu_ctx, tmp_path):
