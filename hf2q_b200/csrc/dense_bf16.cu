@@ -73,26 +73,45 @@ struct MatvecSegs {
     uint32_t blocks0;        // CTAs of segment 0
 };
 
-template <int PRO, int RW>
-__global__ void __launch_bounds__(MV_THREADS) dense_matvec_kernel(const __grid_constant__ MatvecSegs p) {
-    extern __shared__ __align__(16) float xs[];
+// One-row product.  A CTA owns a contiguous range of weight rows, cut into chunks of MV_CHUNK elements; its warps take
+// the chunks in turn, each through a private ring of bulk copies that starts filling before the wait for the previous
+// kernel (weights never change).  Chunk sums of a block of rows meet in shared memory and are added in chunk order.
+constexpr int MR_WARPS = 16, MR_THREADS = MR_WARPS * 32, MV_CHUNK = 1024, MR_STAGES = 3, MR_PART = 2048;
+constexpr uint32_t MR_RING = MR_WARPS * MR_STAGES * MV_CHUNK * 2;
+
+template <int PRO>
+__global__ void __launch_bounds__(MR_THREADS) dense_matvec_kernel(const __grid_constant__ MatvecSegs p, uint32_t* status) {
+    extern __shared__ __align__(128) uint8_t mv_smem[];                 // ring, then x [k] f32
     __shared__ float red[64];
+    __shared__ float part[2][MR_PART];
+    __shared__ uint64_t bars[MR_WARPS][MR_STAGES];
     pdl_trigger();
     const bool second = blockIdx.x >= p.blocks0;
     const hf2q_matvec& s = p.s[second];
-    const uint32_t blk = blockIdx.x - (second ? p.blocks0 : 0u);
-    const __nv_bfloat16* w = static_cast<const __nv_bfloat16*>(s.w);
+    const uint32_t blk = blockIdx.x - (second ? p.blocks0 : 0u), n_blk = second ? gridDim.x - p.blocks0 : p.blocks0;
     const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const uint32_t cta_row0 = blk * MV_WARPS * RW;
-    // the CTA's weight rows are one contiguous range: bring the head of it towards L2 before the wait
-    {
-        const char* b = reinterpret_cast<const char*>(w + static_cast<size_t>(cta_row0) * s.k);
-        const size_t bytes = static_cast<size_t>(min(static_cast<uint32_t>(MV_WARPS * RW), s.n - cta_row0)) * s.k * 2;
-        for (size_t o = threadIdx.x * 128ull; o < bytes; o += MV_THREADS * 128ull) prefetch_l2(b + o);
+    __nv_bfloat16* ring = reinterpret_cast<__nv_bfloat16*>(mv_smem) + static_cast<size_t>(warp) * MR_STAGES * MV_CHUNK;
+    float* xs = reinterpret_cast<float*>(mv_smem + MR_RING);
+    // rows [row0, row1) of this CTA, spread evenly
+    const uint32_t row0 = static_cast<uint32_t>(static_cast<uint64_t>(s.n) * blk / n_blk), row1 = static_cast<uint32_t>(static_cast<uint64_t>(s.n) * (blk + 1) / n_blk);
+    const uint32_t per_row = (s.k + MV_CHUNK - 1) / MV_CHUNK, n_chunks = (row1 - row0) * per_row;
+    const __nv_bfloat16* w = static_cast<const __nv_bfloat16*>(s.w) + static_cast<size_t>(row0) * s.k;
+    auto issue = [&](uint32_t i) {                                      // this warp's chunk number i
+        const uint32_t c = i * MR_WARPS + warp;
+        if (c >= n_chunks) return;
+        const uint32_t k0 = (c % per_row) * MV_CHUNK, bytes = min(static_cast<uint32_t>(MV_CHUNK), s.k - k0) * 2;
+        uint64_t* bar = &bars[warp][i % MR_STAGES];
+        mbar_arrive_expect_tx(bar, bytes);
+        bulk_g2s(ring + (i % MR_STAGES) * MV_CHUNK, w + static_cast<size_t>(c / per_row) * s.k + k0, bytes, bar);
+    };
+    if (lane == 0) {
+        for (int i = 0; i < MR_STAGES; ++i) mbar_init(&bars[warp][i], 1);
+        mbar_fence_init();
+        for (int i = 0; i < MR_STAGES; ++i) issue(i);
     }
     pdl_wait();
     if constexpr (PRO == HF2Q_PRO_NONE) {
-        for (uint32_t i = threadIdx.x; i < s.k; i += MV_THREADS) xs[i] = s.x[i];
+        for (uint32_t i = threadIdx.x; i < s.k; i += MR_THREADS) xs[i] = s.x[i];
     } else if constexpr (PRO == HF2Q_PRO_NORM) {
         const hf2q_pre_norm& q = s.pre;
         const float inv = residual_row(q, 0, xs, red);
@@ -100,7 +119,7 @@ __global__ void __launch_bounds__(MV_THREADS) dense_matvec_kernel(const __grid_c
         const uint32_t pos = q.shift ? *q.pos : 0u;
         const float* before = q.shift_state + static_cast<size_t>((pos + 1) & 1) * q.width;
         float* now = q.shift_state + static_cast<size_t>(pos & 1) * q.width;
-        for (uint32_t i = threadIdx.x; i < s.k; i += MV_THREADS) {
+        for (uint32_t i = threadIdx.x; i < s.k; i += MR_THREADS) {
             float h = 0.f;
             if (i < q.width) {
                 const float x = xs[i];
@@ -114,24 +133,48 @@ __global__ void __launch_bounds__(MV_THREADS) dense_matvec_kernel(const __grid_c
             xs[i] = h;
         }
     } else {
-        for (uint32_t i = s.gated.heads * s.gated.head_dim + threadIdx.x; i < s.k; i += MV_THREADS) xs[i] = 0.f;
-        gated_heads_row<float>(s.gated, 0, xs, warp, MV_WARPS);
+        for (uint32_t i = s.gated.heads * s.gated.head_dim + threadIdx.x; i < s.k; i += MR_THREADS) xs[i] = 0.f;
+        gated_heads_row<float>(s.gated, 0, xs, warp, MR_WARPS);
     }
     __syncthreads();
-    const uint32_t row0 = cta_row0 + warp * RW;
-    if (row0 >= s.n) return;
-    float acc[RW][1];
+    const uint32_t block_rows = max(1u, MR_PART / per_row);
+    bool ok = true;
+    uint32_t i = 0;                                                     // this warp's chunk counter
+    for (uint32_t r0 = 0, pb = 0; r0 < row1 - row0; r0 += block_rows, pb ^= 1) {
+        const uint32_t rows = min(block_rows, row1 - row0 - r0), c_end = (r0 + rows) * per_row;
+        for (uint32_t c = i * MR_WARPS + warp; c < c_end; ++i, c += MR_WARPS) {
+            const uint32_t st = i % MR_STAGES, kc = c % per_row, k0 = kc * MV_CHUNK, len = min(static_cast<uint32_t>(MV_CHUNK), s.k - k0);
+            if (ok) ok = mbar_wait_bounded(&bars[warp][st], (i / MR_STAGES) & 1, status);
+            ok = __all_sync(0xffffffffu, ok);
+            float acc = 0.f;
+            if (ok) {
+                const uint4* wv = reinterpret_cast<const uint4*>(ring + st * MV_CHUNK);
+                const float* xv = xs + k0;
 #pragma unroll
-    for (int r = 0; r < RW; ++r) acc[r][0] = 0.f;
-    matvec_rows<RW, 1>(w, row0, s.n, s.k, xs, acc);
-    if (lane == 0) {
-#pragma unroll
-        for (int r = 0; r < RW; ++r)
-            if (row0 + r < s.n) {
-                float v = epilogue_value(acc[r][0], s.epilogue, s.cap);
-                if (s.epilogue == HF2Q_EPI_ADD) v += s.residual[row0 + r];
-                s.y[row0 + r] = v;
+                for (int u = 0; u < MV_CHUNK / 256; ++u) {
+                    const uint32_t e = lane + 32 * u;
+                    if (8 * e < len) {
+                        const uint4 v = wv[e];
+                        const float4 a = *reinterpret_cast<const float4*>(xv + 8 * e), b = *reinterpret_cast<const float4*>(xv + 8 * e + 4);
+                        acc = fmaf(bf_lo(v.x), a.x, acc); acc = fmaf(bf_hi(v.x), a.y, acc); acc = fmaf(bf_lo(v.y), a.z, acc); acc = fmaf(bf_hi(v.y), a.w, acc);
+                        acc = fmaf(bf_lo(v.z), b.x, acc); acc = fmaf(bf_hi(v.z), b.y, acc); acc = fmaf(bf_lo(v.w), b.z, acc); acc = fmaf(bf_hi(v.w), b.w, acc);
+                    }
+                }
             }
+            __syncwarp();                                               // every lane has read the stage
+            if (lane == 0 && ok) issue(i + MR_STAGES);
+            acc = warp_sum(acc);
+            if (lane == 0) part[pb][c - r0 * per_row] = acc;
+        }
+        __syncthreads();                                                // (the other half of `part` is free: its readers passed this barrier)
+        for (uint32_t r = threadIdx.x; r < rows; r += MR_THREADS) {
+            float v = 0.f;
+            for (uint32_t kc = 0; kc < per_row; ++kc) v += part[pb][r * per_row + kc];
+            const uint32_t row = row0 + r0 + r;
+            v = epilogue_value(v, s.epilogue, s.cap);
+            if (s.epilogue == HF2Q_EPI_ADD) v += s.residual[row];
+            s.y[row] = v;
+        }
     }
 }
 
@@ -462,11 +505,12 @@ cudaError_t dense_any(const DenseArgs& a, int sms, uint32_t* status, cudaStream_
     return launch_pdl(dense_gemm_f32_kernel<X, Y>, dim3((a.n + FT - 1) / FT, (a.m + FT - 1) / FT), dim3(256), 0, st, a);
 }
 
-template <int PRO, int RW>
-cudaError_t launch_fused(const MatvecSegs& p, uint32_t blocks, size_t smem, cudaStream_t st) {
+constexpr uint32_t MR_MAX_SMEM = 208 * 1024;
+template <int PRO>
+cudaError_t launch_fused(const MatvecSegs& p, uint32_t blocks, size_t smem, uint32_t* status, cudaStream_t st) {
     static PerDeviceFlag flag;
-    if (const cudaError_t e = ensure_max_dynamic_smem(dense_matvec_kernel<PRO, RW>, MV_SMEM, flag); e != cudaSuccess) return e;
-    return launch_pdl(dense_matvec_kernel<PRO, RW>, dim3(blocks), dim3(MV_THREADS), smem, st, p);
+    if (const cudaError_t e = ensure_max_dynamic_smem(dense_matvec_kernel<PRO>, MR_MAX_SMEM, flag); e != cudaSuccess) return e;
+    return launch_pdl(dense_matvec_kernel<PRO>, dim3(blocks), dim3(MR_THREADS), smem, st, p, status);
 }
 
 }  // namespace
@@ -503,35 +547,33 @@ HF2Q_API int32_t hf2q_cuda_dense_matvec(hf2q_ctx* ctx, void* stream, uint32_t pr
     if (!ctx) return HF2Q_ERR_INVALID_ARGUMENT;
     if (!segs || n_segs == 0 || n_segs > 2 || prologue > HF2Q_PRO_GATED) return ctx_fail(ctx, HF2Q_ERR_INVALID_ARGUMENT, "dense_matvec: bad segments");
     MatvecSegs p{};
-    uint32_t blocks = 0, rows = 0, kmax = 0;
+    uint32_t kmax = 0;
+    uint64_t chunks[2] = {0, 0};
     for (uint32_t i = 0; i < n_segs; ++i) {
         const hf2q_matvec& s = segs[i];
-        if (!s.w || !s.y || s.n == 0 || s.k == 0 || s.k % 8 || reinterpret_cast<uintptr_t>(s.w) % 16 || s.k * 4ull > MV_SMEM ||
+        if (!s.w || !s.y || s.n == 0 || s.k == 0 || s.k % 8 || reinterpret_cast<uintptr_t>(s.w) % 16 || MR_RING + s.k * 4ull > MR_MAX_SMEM ||
             (prologue == HF2Q_PRO_NONE && !s.x) ||
-            (prologue == HF2Q_PRO_NORM && (!s.pre.x || !s.pre.norm || s.pre.width > s.k || (s.pre.shift && (!s.pre.shift_state || !s.pre.pos)))) ||
+            (prologue == HF2Q_PRO_NORM && (!s.pre.x || !s.pre.norm || s.pre.width > s.k || !pre_norm_aligned(s.pre) || (s.pre.a && (!s.pre.b || !s.pre.a_norm || !s.pre.b_norm)) || (s.pre.shift && (!s.pre.shift_state || !s.pre.pos)))) ||
             (prologue == HF2Q_PRO_GATED && (!s.gated.o || !s.gated.gate || s.gated.heads * s.gated.head_dim > s.k)) ||
             (s.epilogue == HF2Q_EPI_ADD && !s.residual))
             return ctx_fail(ctx, HF2Q_ERR_INVALID_ARGUMENT, "dense_matvec: bad segment");
         p.s[i] = s;
-        rows += s.n;
+        chunks[i] = static_cast<uint64_t>(s.n) * ((s.k + MV_CHUNK - 1) / MV_CHUNK);
         kmax = s.k > kmax ? s.k : kmax;
     }
-    // two rows per warp once that still leaves several CTAs per SM
-    const uint32_t rw = rows >= static_cast<uint32_t>(ctx_sm_count(ctx)) * MV_WARPS * 4 ? 2 : 1;
-    for (uint32_t i = 0; i < n_segs; ++i) {
-        blocks += (segs[i].n + MV_WARPS * rw - 1) / (MV_WARPS * rw);
-        if (i == 0) p.blocks0 = blocks;
-    }
+    // one CTA per SM, shared by the segments in proportion to their chunks; no more CTAs than rows
+    const uint64_t total = chunks[0] + chunks[1], sms = static_cast<uint64_t>(ctx_sm_count(ctx));
+    auto ctas = [&](uint32_t i, uint64_t want) { return static_cast<uint32_t>(want < 1 ? 1 : want > segs[i].n ? segs[i].n : want); };
+    uint32_t blocks = p.blocks0 = ctas(0, n_segs == 1 ? sms : (sms * chunks[0] + total / 2) / total);
+    if (n_segs == 2) blocks += ctas(1, sms > p.blocks0 ? sms - p.blocks0 : 1);
     const cudaStream_t st = static_cast<cudaStream_t>(stream);
-    const size_t smem = static_cast<size_t>(kmax) * 4;
+    const size_t smem = MR_RING + static_cast<size_t>(kmax) * 4;
+    uint32_t* status = ctx_status_word(ctx);
     cudaError_t e;
-    switch (prologue * 2 + (rw - 1)) {
-        case 0: e = launch_fused<HF2Q_PRO_NONE, 1>(p, blocks, smem, st); break;
-        case 1: e = launch_fused<HF2Q_PRO_NONE, 2>(p, blocks, smem, st); break;
-        case 2: e = launch_fused<HF2Q_PRO_NORM, 1>(p, blocks, smem, st); break;
-        case 3: e = launch_fused<HF2Q_PRO_NORM, 2>(p, blocks, smem, st); break;
-        case 4: e = launch_fused<HF2Q_PRO_GATED, 1>(p, blocks, smem, st); break;
-        default: e = launch_fused<HF2Q_PRO_GATED, 2>(p, blocks, smem, st); break;
+    switch (prologue) {
+        case HF2Q_PRO_NONE: e = launch_fused<HF2Q_PRO_NONE>(p, blocks, smem, status, st); break;
+        case HF2Q_PRO_NORM: e = launch_fused<HF2Q_PRO_NORM>(p, blocks, smem, status, st); break;
+        default: e = launch_fused<HF2Q_PRO_GATED>(p, blocks, smem, status, st); break;
     }
     return ctx_cuda_result(ctx, e, "dense_matvec", 1);
 }

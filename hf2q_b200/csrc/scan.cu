@@ -8,6 +8,8 @@
 // warps sixteen columns of one head.  A token costs no block barrier; sums over the key channels are three shuffles.
 // Tokens are staged in shared memory in batches by asynchronous copies, two batches in flight.  The state in memory
 // is [head][column][key channel, padded to 32] (f32), which makes a lane's channels consecutive.
+#include <math_constants.h>
+
 #include "seq_common.cuh"
 
 namespace hf2q {
@@ -34,50 +36,52 @@ __device__ __forceinline__ void stage_rows(float* dst, uint32_t dst_ld, const fl
     }
 }
 
-template <int RQ> struct State {                     // RQ groups of four key channels per lane
-    float4 v[RQ];
+// two f32 values in a 64-bit register; one instruction works on both (IEEE arithmetic on each half)
+typedef unsigned long long f2;
+__device__ __forceinline__ f2 f2_mul(f2 a, f2 b) { f2 d; asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b)); return d; }
+__device__ __forceinline__ f2 f2_fma(f2 a, f2 b, f2 c) { f2 d; asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c)); return d; }
+__device__ __forceinline__ f2 f2_add(f2 a, f2 b) { f2 d; asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b)); return d; }
+__device__ __forceinline__ f2 f2_both(float a) { f2 d; asm("mov.b64 %0, {%1, %1};" : "=l"(d) : "f"(a)); return d; }
+__device__ __forceinline__ float f2_sum(f2 a) { float x, y; asm("mov.b64 {%0, %1}, %2;" : "=f"(x), "=f"(y) : "l"(a)); return x + y; }
+
+template <int RQ> struct Vec {                       // a lane's RQ groups of four key channels
+    f2 v[2 * RQ];
     __device__ __forceinline__ void load(const float* p) {
 #pragma unroll
-        for (int c = 0; c < RQ; ++c) v[c] = *reinterpret_cast<const float4*>(p + 32 * c);
+        for (int c = 0; c < RQ; ++c) {
+            const ulonglong2 q = *reinterpret_cast<const ulonglong2*>(p + 32 * c);
+            v[2 * c] = q.x;
+            v[2 * c + 1] = q.y;
+        }
     }
     __device__ __forceinline__ void zero() {
 #pragma unroll
-        for (int c = 0; c < RQ; ++c) v[c] = make_float4(0.f, 0.f, 0.f, 0.f);
+        for (int c = 0; c < 2 * RQ; ++c) v[c] = 0ull;
     }
     __device__ __forceinline__ void store(float* p) const {
 #pragma unroll
-        for (int c = 0; c < RQ; ++c) *reinterpret_cast<float4*>(p + 32 * c) = v[c];
+        for (int c = 0; c < RQ; ++c) *reinterpret_cast<ulonglong2*>(p + 32 * c) = make_ulonglong2(v[2 * c], v[2 * c + 1]);
     }
-    __device__ __forceinline__ float dot(const float* p) const {
-        float s = 0.f;
+    // sum over this lane's channels, in four interleaved partial sums (two pairs)
+    __device__ __forceinline__ float dot(const Vec& k) const {
+        f2 a = f2_mul(v[0], k.v[0]), b = f2_mul(v[1], k.v[1]);
 #pragma unroll
-        for (int c = 0; c < RQ; ++c) {
-            const float4 k = *reinterpret_cast<const float4*>(p + 32 * c);
-            s = fmaf(v[c].x, k.x, s); s = fmaf(v[c].y, k.y, s); s = fmaf(v[c].z, k.z, s); s = fmaf(v[c].w, k.w, s);
-        }
-        return s;
+        for (int c = 1; c < RQ; ++c) { a = f2_fma(v[2 * c], k.v[2 * c], a); b = f2_fma(v[2 * c + 1], k.v[2 * c + 1], b); }
+        return f2_sum(f2_add(a, b));
     }
-    __device__ __forceinline__ void scale(const float* p) {
+    __device__ __forceinline__ void scale(const Vec& k) {
 #pragma unroll
-        for (int c = 0; c < RQ; ++c) {
-            const float4 k = *reinterpret_cast<const float4*>(p + 32 * c);
-            v[c].x *= k.x; v[c].y *= k.y; v[c].z *= k.z; v[c].w *= k.w;
-        }
+        for (int c = 0; c < 2 * RQ; ++c) v[c] = f2_mul(v[c], k.v[c]);
     }
-    __device__ __forceinline__ void axpy(const float* p, float a) {
+    __device__ __forceinline__ void axpy(const Vec& k, float a) {
+        const f2 aa = f2_both(a);
 #pragma unroll
-        for (int c = 0; c < RQ; ++c) {
-            const float4 k = *reinterpret_cast<const float4*>(p + 32 * c);
-            v[c].x = fmaf(k.x, a, v[c].x); v[c].y = fmaf(k.y, a, v[c].y); v[c].z = fmaf(k.z, a, v[c].z); v[c].w = fmaf(k.w, a, v[c].w);
-        }
+        for (int c = 0; c < 2 * RQ; ++c) v[c] = f2_fma(k.v[c], aa, v[c]);
     }
-    __device__ __forceinline__ void decay_axpy(float keep, const float* p, float a) {
+    __device__ __forceinline__ void decay_axpy(float keep, const Vec& k, float a) {
+        const f2 kk = f2_both(keep), aa = f2_both(a);
 #pragma unroll
-        for (int c = 0; c < RQ; ++c) {
-            const float4 k = *reinterpret_cast<const float4*>(p + 32 * c);
-            v[c].x = fmaf(keep, v[c].x, k.x * a); v[c].y = fmaf(keep, v[c].y, k.y * a);
-            v[c].z = fmaf(keep, v[c].z, k.z * a); v[c].w = fmaf(keep, v[c].w, k.w * a);
-        }
+        for (int c = 0; c < 2 * RQ; ++c) v[c] = f2_fma(kk, v[c], f2_mul(k.v[c], aa));
     }
 };
 
@@ -89,7 +93,7 @@ __global__ void __launch_bounds__(SC_THREADS) mlstm_kernel(const __grid_constant
     float* ks = dsm;
     float* qs = dsm + 2 * SC_TB * DP;
     __shared__ __align__(16) float vs[2][SC_TB][SC_COLS];
-    __shared__ float gi[2][SC_TB], gf[2][SC_TB];
+    __shared__ float gk[2][SC_TB], gw[2][SC_TB], ge[2][SC_TB];     // keep, write, exp(-maximum)
     pdl_trigger();
     pdl_wait();
     const uint32_t h = blockIdx.x, slice = blockIdx.y, n_slices = gridDim.y;
@@ -98,6 +102,8 @@ __global__ void __launch_bounds__(SC_THREADS) mlstm_kernel(const __grid_constant
     const uint32_t n_cols = min(static_cast<uint32_t>(SC_COLS), a.vdim - col0);
     const bool live = col < a.vdim;
     const float q_scale = 1.0f / sqrtf(static_cast<float>(a.dim));
+    float* mp = a.mx + static_cast<size_t>(h) * n_slices + slice;
+    float mx = *mp;                                          // carried by the last warp
     // channels past dim stay zero in shared memory, so the padded part of the state stays zero too
     for (uint32_t i = threadIdx.x; i < 4 * SC_TB * DP; i += SC_THREADS) dsm[i] = 0.f;
     for (uint32_t i = threadIdx.x; i < 2 * SC_TB * SC_COLS; i += SC_THREADS) (&vs[0][0][0])[i] = 0.f;
@@ -108,53 +114,67 @@ __global__ void __launch_bounds__(SC_THREADS) mlstm_kernel(const __grid_constant
         stage_rows(ks + b * SC_TB * DP, DP, row + a.k_off + h * a.dim, a.ld, n, a.dim);
         stage_rows(qs + b * SC_TB * DP, DP, row + a.q_off + h * a.dim, a.ld, n, a.dim);
         stage_rows(vs[b][0], SC_COLS, row + a.v_off + h * a.vdim + col0, a.ld, n, n_cols);
-        if (threadIdx.x < n) {
-            gi[b][threadIdx.x] = row[static_cast<size_t>(threadIdx.x) * a.ld + a.i_off + h];
-            gf[b][threadIdx.x] = row[static_cast<size_t>(threadIdx.x) * a.ld + a.f_off + h];
-            const float x = a.gate_cap * tanhf((gi[b][threadIdx.x] + a.i_bias[h]) / a.gate_cap);
-            const float f = a.gate_cap * tanhf((gf[b][threadIdx.x] + a.f_bias[h]) / a.gate_cap);
-            gi[b][threadIdx.x] = x;
-            gf[b][threadIdx.x] = -softplusf(-f);
+        // gate factors of the batch, by the last warp (lane = token): the running maximum is a max-plus scan over the
+        // pairs (f, i), m_t = max(m + f_1 + .. + f_t, max_s (i_s + f_(s+1) + .. + f_t))
+        if (warp == SC_WARPS - 1) {
+            float f = 0.f, x = -CUDART_INF_F;
+            if (lane < n) {
+                const float* g = row + static_cast<size_t>(lane) * a.ld + h;
+                x = a.gate_cap * tanhf((g[a.i_off] + a.i_bias[h]) / a.gate_cap);
+                f = -softplusf(-a.gate_cap * tanhf((g[a.f_off] + a.f_bias[h]) / a.gate_cap));
+            }
+            const float f_own = f, x_own = x;
+#pragma unroll
+            for (int d = 1; d < SC_TB; d *= 2) {
+                const float fo = __shfl_up_sync(0xffffffffu, f, d), xo = __shfl_up_sync(0xffffffffu, x, d);
+                if (lane >= d) { x = fmaxf(xo + f, x); f += fo; }
+            }
+            const float m_t = fmaxf(mx + f, x);
+            float before = __shfl_up_sync(0xffffffffu, m_t, 1);
+            if (lane == 0) before = mx;
+            if (lane < n) {
+                gk[b][lane] = expf(f_own + before - m_t);
+                gw[b][lane] = expf(x_own - m_t);
+                ge[b][lane] = expf(-m_t);
+            }
+            mx = __shfl_sync(0xffffffffu, m_t, n - 1);
         }
         cp_async_commit();
     };
-    State<RQ> S, N;
+    Vec<RQ> S, N;
     float* sp = a.s + (static_cast<size_t>(h) * a.vdim + (live ? col : 0)) * DP + 4 * l8;
     float* np = a.n + (static_cast<size_t>(h) * n_slices + slice) * DP + 4 * l8;
-    float* mp = a.mx + static_cast<size_t>(h) * n_slices + slice;
     if (live) S.load(sp); else S.zero();
     N.load(np);
-    float mx = *mp;
     stage(0, 0);
     for (uint32_t t0 = 0, b = 0; t0 < m; t0 += SC_TB, b ^= 1) {
         if (t0 + SC_TB < m) { stage(t0 + SC_TB, b ^ 1); cp_async_wait<1>(); }
         else cp_async_wait<0>();
         __syncthreads();
         const uint32_t n = min(static_cast<uint32_t>(SC_TB), m - t0);
+#pragma unroll 4
         for (uint32_t j = 0; j < n; ++j) {
-            const float i_t = gi[b][j], f_t = gf[b][j];
-            const float m_new = fmaxf(f_t + mx, i_t);
-            const float keep = expf(f_t + mx - m_new), write = expf(i_t - m_new);
-            mx = m_new;
-            const float* k = ks + (b * SC_TB + j) * DP + 4 * l8;
-            const float* q = qs + (b * SC_TB + j) * DP + 4 * l8;
+            Vec<RQ> k, q;
+            k.load(ks + (b * SC_TB + j) * DP + 4 * l8);
+            q.load(qs + (b * SC_TB + j) * DP + 4 * l8);
+            const float keep = gk[b][j], write = gw[b][j];
             S.decay_axpy(keep, k, write * vs[b][j][col_s]);
             N.decay_axpy(keep, k, write);
             const float num = group8_sum(S.dot(q)) * q_scale, den = group8_sum(N.dot(q)) * q_scale;
             if (l8 == 0 && live)
-                out[static_cast<size_t>(t0 + j) * a.heads * a.vdim + static_cast<size_t>(h) * a.vdim + col] = num / (fmaxf(fabsf(den), expf(-mx)) + 1e-6f);
+                out[static_cast<size_t>(t0 + j) * a.heads * a.vdim + static_cast<size_t>(h) * a.vdim + col] = num / (fmaxf(fabsf(den), ge[b][j]) + 1e-6f);
         }
         __syncthreads();
     }
     if (live) S.store(sp);
     if (warp == 0 && lane < 8) N.store(np);
-    if (threadIdx.x == 0) *mp = mx;
+    if (warp == SC_WARPS - 1 && lane == 0) *mp = mx;
 }
 
 // ---------------------------------------------------------------- gated delta rule
 // S <- g S;  u = beta (v - S^T k);  S <- S + k u;  o = S^T q
 template <int RQ>
-__device__ __forceinline__ float delta_token(State<RQ>& S, const float* g, const float* k, const float* q, float v, float beta) {
+__device__ __forceinline__ float delta_token(Vec<RQ>& S, const Vec<RQ>& g, const Vec<RQ>& k, const Vec<RQ>& q, float v, float beta) {
     S.scale(g);
     const float u = beta * (v - group8_sum(S.dot(k)));
     S.axpy(k, u);
@@ -192,7 +212,7 @@ __global__ void __launch_bounds__(SC_THREADS) delta_scan_kernel(const __grid_con
         if (threadIdx.x < n) bs[b][threadIdx.x] = beta[static_cast<size_t>(t0 + threadIdx.x) * a.heads + h];
         cp_async_commit();
     };
-    State<RQ> S;
+    Vec<RQ> S;
     float* sp = a.s + (static_cast<size_t>(h) * a.vdim + (live ? col : 0)) * DP + 4 * l8;
     if (live) S.load(sp); else S.zero();
     stage(0, 0);
@@ -201,9 +221,14 @@ __global__ void __launch_bounds__(SC_THREADS) delta_scan_kernel(const __grid_con
         else cp_async_wait<0>();
         __syncthreads();
         const uint32_t n = min(static_cast<uint32_t>(SC_TB), m - t0);
+#pragma unroll 4
         for (uint32_t j = 0; j < n; ++j) {
             const uint32_t o = (b * SC_TB + j) * DP + 4 * l8;
-            const float r = delta_token<RQ>(S, gs + o, ks + o, qs + o, vs[b][j][col_s], bs[b][j]);
+            Vec<RQ> dg, k, q;
+            dg.load(gs + o);
+            k.load(ks + o);
+            q.load(qs + o);
+            const float r = delta_token<RQ>(S, dg, k, q, vs[b][j][col_s], bs[b][j]);
             if (l8 == 0 && live) out[static_cast<size_t>(t0 + j) * a.heads * a.vdim + static_cast<size_t>(h) * a.vdim + col] = r;
         }
         __syncthreads();
@@ -244,8 +269,10 @@ __global__ void __launch_bounds__(SC_THREADS) delta_step_kernel(const __grid_con
     const uint32_t col_s = warp * 4 + (lane >> 3), col0 = slice * SC_COLS, col = col0 + col_s;
     const uint32_t n_cols = min(static_cast<uint32_t>(SC_COLS), a.vdim - col0);
     const bool live = col < a.vdim;
+    for (uint32_t i = threadIdx.x; i < a.dim; i += SC_THREADS)       // weights: towards L2 before the wait
+        for (uint32_t c = 0; c < a.a_rank_ld; c += 64) prefetch_l2(static_cast<const __nv_bfloat16*>(a.a2) + (static_cast<size_t>(h) * a.dim + i) * a.a_rank_ld + c);
     pdl_wait();
-    State<RQ> S;
+    Vec<RQ> S;
     float* sp = a.s + (static_cast<size_t>(h) * a.vdim + (live ? col : 0)) * DP + 4 * l8;
     if (live) S.load(sp); else S.zero();
     const uint32_t pos = *a.pos, qk = a.kv_heads * a.dim;
@@ -292,7 +319,11 @@ __global__ void __launch_bounds__(SC_THREADS) delta_step_kernel(const __grid_con
         gate[c] = low_rank_dot(a.g2, c, a.g_rank_ld, lr + a.a_rank_ld);
     }
     __syncthreads();
-    const float r = delta_token<RQ>(S, gs + 4 * l8, ks + 4 * l8, qs + 4 * l8, vs[col_s], sigmoidf(a.proj[a.b_off + h]));
+    Vec<RQ> dg, k, q;
+    dg.load(gs + 4 * l8);
+    k.load(ks + 4 * l8);
+    q.load(qs + 4 * l8);
+    const float r = delta_token<RQ>(S, dg, k, q, vs[col_s], sigmoidf(a.proj[a.b_off + h]));
     if (live) {
         S.store(sp);
         if (l8 == 0) out[h * a.vdim + col] = r;

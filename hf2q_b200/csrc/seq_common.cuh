@@ -90,16 +90,33 @@ __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commi
 template <int N> __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
 // ---------------------------------------------------------------- row prologues
+// rows whose width is a multiple of four are read in 16-byte groups
+inline bool pre_norm_aligned(const hf2q_pre_norm& p) {
+    if (p.width % 4) return true;
+    const void* all[] = {p.x, p.a, p.b, p.a_norm, p.b_norm, p.add0, p.step};
+    for (const void* q : all)
+        if (reinterpret_cast<uintptr_t>(q) % 16) return false;
+    return true;
+}
+
 // Residual update of row t into xs[0..width) (shared memory):
 //   x + 0.5 (rms(a) a_norm + rms(b) b_norm)  (+ add0)  (+ step)
 // and the reciprocal root mean square of the result.  Rows are `width` floats apart.
 __device__ __forceinline__ float residual_row(const hf2q_pre_norm& p, uint32_t t, float* xs, float* red) {
     const size_t o = static_cast<size_t>(t) * p.width;
     const float n = static_cast<float>(p.width);
+    const bool quads = p.width % 4 == 0;                   // rows of whole 16-byte groups
+    const uint32_t nq = quads ? p.width / 4 : 0;
+    auto q4 = [](const float* b, uint32_t i) { return *reinterpret_cast<const float4*>(b + 4 * i); };
     float ia = 0.f, ib = 0.f;
     if (p.a) {
         float s[2] = {0.f, 0.f};
-        for (uint32_t i = threadIdx.x; i < p.width; i += blockDim.x) {
+        for (uint32_t i = threadIdx.x; i < nq; i += blockDim.x) {
+            const float4 va = q4(p.a + o, i), vb = q4(p.b + o, i);
+            s[0] += va.x * va.x + va.y * va.y + va.z * va.z + va.w * va.w;
+            s[1] += vb.x * vb.x + vb.y * vb.y + vb.z * vb.z + vb.w * vb.w;
+        }
+        for (uint32_t i = 4 * nq + threadIdx.x; i < p.width; i += blockDim.x) {
             const float va = p.a[o + i], vb = p.b[o + i];
             s[0] += va * va;
             s[1] += vb * vb;
@@ -110,7 +127,19 @@ __device__ __forceinline__ float residual_row(const hf2q_pre_norm& p, uint32_t t
         __syncthreads();
     }
     float s[1] = {0.f};
-    for (uint32_t i = threadIdx.x; i < p.width; i += blockDim.x) {
+    for (uint32_t i = threadIdx.x; i < nq; i += blockDim.x) {
+        float4 v = q4(p.x + o, i);
+        if (p.a) {
+            const float4 a = q4(p.a + o, i), an = q4(p.a_norm, i), b = q4(p.b + o, i), bn = q4(p.b_norm, i);
+            v.x += a.x * ia * an.x + b.x * ib * bn.x; v.y += a.y * ia * an.y + b.y * ib * bn.y;
+            v.z += a.z * ia * an.z + b.z * ib * bn.z; v.w += a.w * ia * an.w + b.w * ib * bn.w;
+        }
+        if (p.add0) { const float4 a = q4(p.add0 + o, i); v.x += a.x; v.y += a.y; v.z += a.z; v.w += a.w; }
+        if (p.step) { const float4 a = q4(p.step, i); v.x += a.x; v.y += a.y; v.z += a.z; v.w += a.w; }
+        *reinterpret_cast<float4*>(xs + 4 * i) = v;
+        s[0] += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+    }
+    for (uint32_t i = 4 * nq + threadIdx.x; i < p.width; i += blockDim.x) {
         float v = p.x[o + i];
         if (p.a) v += p.a[o + i] * ia * p.a_norm[i] + p.b[o + i] * ib * p.b_norm[i];
         if (p.add0) v += p.add0[o + i];

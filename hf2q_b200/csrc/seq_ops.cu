@@ -32,34 +32,44 @@ __global__ void __launch_bounds__(256) embed_kernel(const __grid_constant__ hf2q
     }
 }
 
-// one CTA per row; with a token shift the row before it is recomputed from the same inputs
+// `run` consecutive rows per CTA; a token shift needs the row before the first as well, recomputed from the same inputs
 template <typename OUT>
-__global__ void __launch_bounds__(256) pre_norm_kernel(const __grid_constant__ hf2q_pre_norm p, uint32_t m, OUT* __restrict__ out, uint32_t ldo,
+__global__ void __launch_bounds__(256) pre_norm_kernel(const __grid_constant__ hf2q_pre_norm p, uint32_t m, uint32_t run, OUT* __restrict__ out, uint32_t ldo,
                                                        float* __restrict__ h_last) {
-    extern __shared__ float xs[];                          // width, and another width with a shift
+    extern __shared__ __align__(16) float xs[];            // width, and another width with a shift: the h of the row before
     __shared__ float red[64];
     pdl_trigger();
     pdl_wait();
-    const uint32_t t = blockIdx.x;
-    float inv_b = 0.f;
-    float* xb = xs + p.width;
-    if (p.shift && t > 0) inv_b = residual_row(p, t - 1, xb, red);
-    const float inv = residual_row(p, t, xs, red);
+    const uint32_t t0 = blockIdx.x * run, t1 = min(t0 + run, m);
     const uint32_t pos = p.shift ? *p.pos : 0u;
-    for (uint32_t i = threadIdx.x; i < ldo; i += blockDim.x) {
-        float h = 0.f;
-        if (i < p.width) {
-            const float x = xs[i], w = p.norm[i];
-            if (p.x_out) p.x_out[static_cast<size_t>(t) * p.width + i] = x;
-            h = x * inv * w;
-            if (p.shift) {
-                const float b = t > 0 ? xb[i] * inv_b * w : p.shift_state[static_cast<size_t>((pos + 1) & 1) * p.width + i];
-                if (m == 1) p.shift_state[static_cast<size_t>(pos & 1) * p.width + i] = h;
-                else if (t == m - 1) h_last[i] = h;
-                h += (b - h) * p.shift[i];
-            }
+    float* before = xs + p.width;                          // an element is read and written by one thread only
+    if (p.shift) {
+        if (t0 > 0) {
+            const float inv = residual_row(p, t0 - 1, before, red);
+            for (uint32_t i = threadIdx.x; i < p.width; i += blockDim.x) before[i] *= inv * p.norm[i];
+        } else {
+            for (uint32_t i = threadIdx.x; i < p.width; i += blockDim.x) before[i] = p.shift_state[static_cast<size_t>((pos + 1) & 1) * p.width + i];
         }
-        out[static_cast<size_t>(t) * ldo + i] = from_f32<OUT>(h);
+    }
+    for (uint32_t t = t0; t < t1; ++t) {
+        const float inv = residual_row(p, t, xs, red);
+        for (uint32_t i = threadIdx.x; i < ldo; i += blockDim.x) {
+            float h = 0.f;
+            if (i < p.width) {
+                const float x = xs[i];
+                if (p.x_out) p.x_out[static_cast<size_t>(t) * p.width + i] = x;
+                h = x * inv * p.norm[i];
+                if (p.shift) {
+                    const float b = before[i];
+                    before[i] = h;
+                    if (m == 1) p.shift_state[static_cast<size_t>(pos & 1) * p.width + i] = h;
+                    else if (t == m - 1) h_last[i] = h;
+                    h += (b - h) * p.shift[i];
+                }
+            }
+            out[static_cast<size_t>(t) * ldo + i] = from_f32<OUT>(h);
+        }
+        __syncthreads();                                   // xs is read across threads before the next row replaces it
     }
 }
 
@@ -114,20 +124,23 @@ HF2Q_API int32_t hf2q_cuda_pre_norm(hf2q_ctx* ctx, void* stream, const hf2q_pre_
                                     float* h_last) {
     if (!ctx) return HF2Q_ERR_INVALID_ARGUMENT;
     if (!p || !p->x || !p->norm || !out || p->width == 0 || ldo < p->width || p->x_out == p->x || (p->a && (!p->b || !p->a_norm || !p->b_norm)) ||
-        (p->shift && (!p->shift_state || !p->pos || (m > 1 && !h_last))))
-        return ctx_fail(ctx, HF2Q_ERR_INVALID_ARGUMENT, "pre_norm: null pointer, or x_out is x");
+        (p->shift && (!p->shift_state || !p->pos || (m > 1 && !h_last))) || !pre_norm_aligned(*p))
+        return ctx_fail(ctx, HF2Q_ERR_INVALID_ARGUMENT, "pre_norm: null or unaligned pointer, or x_out is x");
     if (m == 0) return HF2Q_OK;
     const size_t smem = static_cast<size_t>(p->width) * (p->shift ? 8 : 4);
     if (smem > 200 * 1024) return ctx_fail(ctx, HF2Q_ERR_INVALID_ARGUMENT, "pre_norm: width too large");
     const cudaStream_t st = static_cast<cudaStream_t>(stream);
     static PerDeviceFlag f32f, bff;
+    // long portions: a few rows per CTA while every SM keeps several CTAs
+    const uint32_t run = p->shift && m >= 4u * 4u * static_cast<uint32_t>(ctx_sm_count(ctx)) ? 8 : p->shift && m >= 512 ? 4 : 1;
+    const dim3 grid((m + run - 1) / run);
     cudaError_t e;
     if (out_dtype == HF2Q_DT_F32) {
         e = ensure_max_dynamic_smem(pre_norm_kernel<float>, 200 * 1024, f32f);
-        if (e == cudaSuccess) e = launch_pdl(pre_norm_kernel<float>, dim3(m), dim3(256), smem, st, *p, m, static_cast<float*>(out), ldo, h_last);
+        if (e == cudaSuccess) e = launch_pdl(pre_norm_kernel<float>, grid, dim3(256), smem, st, *p, m, run, static_cast<float*>(out), ldo, h_last);
     } else if (out_dtype == HF2Q_DT_BF16) {
         e = ensure_max_dynamic_smem(pre_norm_kernel<__nv_bfloat16>, 200 * 1024, bff);
-        if (e == cudaSuccess) e = launch_pdl(pre_norm_kernel<__nv_bfloat16>, dim3(m), dim3(256), smem, st, *p, m, static_cast<__nv_bfloat16*>(out), ldo, h_last);
+        if (e == cudaSuccess) e = launch_pdl(pre_norm_kernel<__nv_bfloat16>, grid, dim3(256), smem, st, *p, m, run, static_cast<__nv_bfloat16*>(out), ldo, h_last);
     } else {
         e = cudaErrorInvalidValue;
     }

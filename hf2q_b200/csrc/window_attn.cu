@@ -2,8 +2,8 @@
 // per-head RMS norm of q and k and an optional logarithmic distance term taken off the scores.
 //
 //   append    prefill: normalised queries to a buffer, normalised keys and values to the cache
-//   prefill   bf16 cache: tiles of 64 queries x 64 keys on the tensor cores (f32 scores, softmax and accumulators; the
-//             probabilities enter the value product as a bf16 pair hi + lo); f32 cache: one warp per query in f32
+//   prefill   bf16 cache: tiles of 64 queries x 64 keys on the tensor cores (f32 scores, softmax and accumulators, bf16
+//             product operands); f32 cache: one warp per query in f32
 //   decode    one launch: norm, append, window split over CTAs, merge by the CTA that arrives last
 #include <math_constants.h>
 
@@ -96,7 +96,7 @@ struct WarpAttn {
         for (int g = 0; g < GR; ++g) s[g] = 0.f;
         if (live) {
             const T* kr = kc + static_cast<size_t>(p % a.capacity) * dp;
-#pragma unroll 4
+#pragma unroll 8
             for (uint32_t c = 0; c < dp; c += 8) {
                 float k[8];
                 load8(kr + c, k);
@@ -122,7 +122,7 @@ struct WarpAttn {
         }
         __syncwarp();
         const uint32_t cnt = min(32u, hi - p0);
-#pragma unroll 4
+#pragma unroll 8
         for (uint32_t i = 0; i < cnt; ++i) {
             const T* vr = vc + static_cast<size_t>((p0 + i) % a.capacity) * dvp;
 #pragma unroll
@@ -418,22 +418,16 @@ __global__ void __launch_bounds__(WP_WARPS * 32) window_prefill_mma_kernel(const
                 }
 #pragma unroll
             for (int k = 0; k < WP_K / 16; ++k) {
-                uint32_t hi[4], lo[4];
+                uint32_t pa[4];
 #pragma unroll
-                for (int i = 0; i < 4; ++i) {
-                    const float x = s[2 * k + (i >> 1)][2 * (i & 1)], y = s[2 * k + (i >> 1)][2 * (i & 1) + 1];
-                    hi[i] = pack_bf16(x, y);
-                    lo[i] = pack_bf16(x - bf_lo(hi[i]), y - bf_hi(hi[i]));
-                }
+                for (int i = 0; i < 4; ++i) pa[i] = pack_bf16(s[2 * k + (i >> 1)][2 * (i & 1)], s[2 * k + (i >> 1)][2 * (i & 1) + 1]);
 #pragma unroll
                 for (int n2 = 0; n2 < DM / 16; ++n2) {
                     if (n2 < static_cast<int>(nv)) {
                         uint32_t f[4];
                         ldmatrix4_trans(f, vs + ((16 * k + ((lane >> 3) & 1) * 8 + (lane & 7)) * PITCH + 16 * n2 + (lane >> 4) * 8) * 2);
-                        mma_bf16(o[2 * n2], hi, f[0], f[1]);
-                        mma_bf16(o[2 * n2], lo, f[0], f[1]);
-                        mma_bf16(o[2 * n2 + 1], hi, f[2], f[3]);
-                        mma_bf16(o[2 * n2 + 1], lo, f[2], f[3]);
+                        mma_bf16(o[2 * n2], pa, f[0], f[1]);
+                        mma_bf16(o[2 * n2 + 1], pa, f[2], f[3]);
                     }
                 }
             }

@@ -107,7 +107,21 @@ def test_pre_norm_and_token_shift(sop, width, m):
             p.shift_state, p.x_out = state2.data_ptr(), xo2.data_ptr()
             sop.matvec(S.PRO_NORM, S.struct(S.Matvec, w=w.w, y=y, pre=p, n=w.n, k=w.k))
             assert rel(y, want @ w.w[:, :width].cpu().double().numpy().T) < 1e-5
-            assert torch.equal(state2, state) and torch.equal(xo2, x_out)
+            assert torch.allclose(state2, state, rtol=1e-5, atol=1e-6) and torch.allclose(xo2, x_out, rtol=1e-5, atol=1e-6)
+
+
+@pytest.mark.parametrize("m", [600, 2501])
+def test_pre_norm_of_long_portions(sop, m):
+    """Several rows per CTA: the row in front of a CTA's first one is recomputed."""
+    rng = np.random.default_rng(m)
+    w = 68
+    x, norm, mu, step = rng.standard_normal((m, w)), rng.standard_normal(w), rng.random(w), rng.standard_normal(w)
+    h = F.rms(x + step, 1e-5) * norm
+    xg, ng, mg, sg, state, last, pos = f32(x), f32(norm), f32(mu), f32(step), torch.zeros(2, w, device=DEV), torch.zeros(1, w, device=DEV), dev_pos(0)
+    out, x_out = torch.zeros(m, 72, device=DEV), torch.zeros(m, w, device=DEV)
+    p = S.struct(S.PreNorm, x=xg, step=sg, x_out=x_out, norm=ng, shift=mg, shift_state=state, pos=pos, eps=1e-5, width=w)
+    sop.pre_norm(p, m, out, last)
+    assert rel(out[:, :w], F.token_shift(h, mu)) < 2e-6 and rel(last, h[-1:]) < 1e-6 and rel(x_out, x + step) < 1e-6
 
 
 @pytest.mark.parametrize("norm_all", [0, 1])
