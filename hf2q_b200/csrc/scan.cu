@@ -24,15 +24,16 @@ __device__ __forceinline__ float group8_sum(float v) {
     v += __shfl_xor_sync(0xffffffffu, v, 4);
     return v;
 }
-// rows of `count` floats -> shared memory, asynchronously, 16 bytes at a time where both sides allow it
+// rows of `count` floats -> shared memory, asynchronously, 16 bytes at a time where both sides allow it; a warp takes
+// whole rows
 __device__ __forceinline__ void stage_rows(float* dst, uint32_t dst_ld, const float* src, size_t src_ld, uint32_t rows, uint32_t count) {
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     if (count % 4 == 0 && src_ld % 4 == 0 && dst_ld % 4 == 0 && (reinterpret_cast<uintptr_t>(src) & 15) == 0) {
-        const uint32_t q = count / 4;
-        for (uint32_t i = threadIdx.x; i < rows * q; i += SC_THREADS)
-            cp_async16(dst + (i / q) * dst_ld + 4 * (i % q), src + (i / q) * src_ld + 4 * (i % q));
+        for (uint32_t r = warp; r < rows; r += SC_WARPS)
+            for (uint32_t c = 4 * lane; c < count; c += 128) cp_async16(dst + r * dst_ld + c, src + r * src_ld + c);
     } else {
-        for (uint32_t i = threadIdx.x; i < rows * count; i += SC_THREADS)
-            cp_async4(dst + (i / count) * dst_ld + i % count, src + (i / count) * src_ld + i % count);
+        for (uint32_t r = warp; r < rows; r += SC_WARPS)
+            for (uint32_t c = lane; c < count; c += 32) cp_async4(dst + r * dst_ld + c, src + r * src_ld + c);
     }
 }
 
@@ -152,17 +153,36 @@ __global__ void __launch_bounds__(SC_THREADS) mlstm_kernel(const __grid_constant
         else cp_async_wait<0>();
         __syncthreads();
         const uint32_t n = min(static_cast<uint32_t>(SC_TB), m - t0);
-#pragma unroll 4
-        for (uint32_t j = 0; j < n; ++j) {
+        auto token = [&](uint32_t j, float& num, float& den) {
             Vec<RQ> k, q;
             k.load(ks + (b * SC_TB + j) * DP + 4 * l8);
             q.load(qs + (b * SC_TB + j) * DP + 4 * l8);
             const float keep = gk[b][j], write = gw[b][j];
             S.decay_axpy(keep, k, write * vs[b][j][col_s]);
             N.decay_axpy(keep, k, write);
-            const float num = group8_sum(S.dot(q)) * q_scale, den = group8_sum(N.dot(q)) * q_scale;
-            if (l8 == 0 && live)
-                out[static_cast<size_t>(t0 + j) * a.heads * a.vdim + static_cast<size_t>(h) * a.vdim + col] = num / (fmaxf(fabsf(den), ge[b][j]) + 1e-6f);
+            num = group8_sum(S.dot(q));
+            den = group8_sum(N.dot(q));
+        };
+        auto finish = [&](uint32_t j, float num, float den) {
+            if (live)
+                out[static_cast<size_t>(t0 + j) * a.heads * a.vdim + static_cast<size_t>(h) * a.vdim + col] = num * q_scale / (fmaxf(fabsf(den * q_scale), ge[b][j]) + 1e-6f);
+        };
+        uint32_t j0 = 0;
+        for (; j0 + 8 <= n; j0 += 8) {                       // eight tokens without a branch; lane i of a group finishes token i
+            float num = 0.f, den = 0.f;
+#pragma unroll
+            for (uint32_t u = 0; u < 8; ++u) {
+                float x, y;
+                token(j0 + u, x, y);
+                num = l8 == u ? x : num;
+                den = l8 == u ? y : den;
+            }
+            finish(j0 + l8, num, den);
+        }
+        for (; j0 < n; ++j0) {
+            float x, y;
+            token(j0, x, y);
+            if (l8 == 0) finish(j0, x, y);
         }
         __syncthreads();
     }
@@ -221,15 +241,29 @@ __global__ void __launch_bounds__(SC_THREADS) delta_scan_kernel(const __grid_con
         else cp_async_wait<0>();
         __syncthreads();
         const uint32_t n = min(static_cast<uint32_t>(SC_TB), m - t0);
-#pragma unroll 4
-        for (uint32_t j = 0; j < n; ++j) {
+        auto token = [&](uint32_t j) {
             const uint32_t o = (b * SC_TB + j) * DP + 4 * l8;
             Vec<RQ> dg, k, q;
             dg.load(gs + o);
             k.load(ks + o);
             q.load(qs + o);
-            const float r = delta_token<RQ>(S, dg, k, q, vs[b][j][col_s], bs[b][j]);
-            if (l8 == 0 && live) out[static_cast<size_t>(t0 + j) * a.heads * a.vdim + static_cast<size_t>(h) * a.vdim + col] = r;
+            return delta_token<RQ>(S, dg, k, q, vs[b][j][col_s], bs[b][j]);
+        };
+        float* dst = out + static_cast<size_t>(t0) * a.heads * a.vdim + static_cast<size_t>(h) * a.vdim + col;
+        const size_t row_o = static_cast<size_t>(a.heads) * a.vdim;
+        uint32_t j0 = 0;
+        for (; j0 + 8 <= n; j0 += 8) {                       // eight tokens without a branch; lane i of a group stores token i
+            float r = 0.f;
+#pragma unroll
+            for (uint32_t u = 0; u < 8; ++u) {
+                const float x = token(j0 + u);
+                r = l8 == u ? x : r;
+            }
+            if (live) dst[(j0 + l8) * row_o] = r;
+        }
+        for (; j0 < n; ++j0) {
+            const float r = token(j0);
+            if (l8 == 0 && live) dst[j0 * row_o] = r;
         }
         __syncthreads();
     }

@@ -160,8 +160,30 @@ __device__ __forceinline__ void gated_heads_row(const hf2q_gated_heads& g, uint3
     const uint32_t lane = threadIdx.x & 31;
     const float* o = g.o + static_cast<size_t>(t) * g.ldo;
     const float* gate = g.gate + static_cast<size_t>(t) * g.ldg;
+    // whole 16-byte groups and at most one per lane: a head stays in registers
+    const bool quads = g.head_dim % 4 == 0 && g.head_dim <= 128 &&
+                       ((reinterpret_cast<uintptr_t>(o) | reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(g.norm)) & 15) == 0;
     for (uint32_t h = warp; h < g.heads; h += n_warps) {
         const uint32_t c0 = h * g.head_dim;
+        if (quads) {
+            const uint32_t i = 4 * lane;
+            const bool has = i < g.head_dim;
+            const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+            const float4 v = has ? *reinterpret_cast<const float4*>(o + c0 + i) : zero, x = has ? *reinterpret_cast<const float4*>(gate + c0 + i) : zero;
+            float4 w = make_float4(1.f, 1.f, 1.f, 1.f);
+            if (g.norm) {
+                const float inv = 1.0f / sqrtf(warp_sum(v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w) / static_cast<float>(g.head_dim) + g.eps);
+                if (has) w = *reinterpret_cast<const float4*>(g.norm + (g.norm_all ? c0 + i : i));
+                w = make_float4(w.x * inv, w.y * inv, w.z * inv, w.w * inv);
+            }
+            if (has) {
+                out[c0 + i] = from_f32<OUT>(v.x * w.x * sigmoidf(x.x));
+                out[c0 + i + 1] = from_f32<OUT>(v.y * w.y * sigmoidf(x.y));
+                out[c0 + i + 2] = from_f32<OUT>(v.z * w.z * sigmoidf(x.z));
+                out[c0 + i + 3] = from_f32<OUT>(v.w * w.w * sigmoidf(x.w));
+            }
+            continue;
+        }
         float inv = 1.0f;
         if (g.norm) {
             float s = 0.f;

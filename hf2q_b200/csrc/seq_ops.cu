@@ -34,7 +34,7 @@ __global__ void __launch_bounds__(256) embed_kernel(const __grid_constant__ hf2q
 
 // `run` consecutive rows per CTA; a token shift needs the row before the first as well, recomputed from the same inputs
 template <typename OUT>
-__global__ void __launch_bounds__(256) pre_norm_kernel(const __grid_constant__ hf2q_pre_norm p, uint32_t m, uint32_t run, OUT* __restrict__ out, uint32_t ldo,
+__global__ void __launch_bounds__(512) pre_norm_kernel(const __grid_constant__ hf2q_pre_norm p, uint32_t m, uint32_t run, OUT* __restrict__ out, uint32_t ldo,
                                                        float* __restrict__ h_last) {
     extern __shared__ __align__(16) float xs[];            // width, and another width with a shift: the h of the row before
     __shared__ float red[64];
@@ -51,8 +51,35 @@ __global__ void __launch_bounds__(256) pre_norm_kernel(const __grid_constant__ h
             for (uint32_t i = threadIdx.x; i < p.width; i += blockDim.x) before[i] = p.shift_state[static_cast<size_t>((pos + 1) & 1) * p.width + i];
         }
     }
+    const bool quads = p.width % 4 == 0 && ldo == p.width &&
+                       ((reinterpret_cast<uintptr_t>(p.norm) | reinterpret_cast<uintptr_t>(p.shift) | reinterpret_cast<uintptr_t>(p.x_out) |
+                         reinterpret_cast<uintptr_t>(p.shift_state) | reinterpret_cast<uintptr_t>(h_last) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+    if (quads) __syncthreads();                            // `before` changes hands: groups of four per thread from here on
     for (uint32_t t = t0; t < t1; ++t) {
         const float inv = residual_row(p, t, xs, red);
+        if (quads) {
+            for (uint32_t i = threadIdx.x; i < p.width / 4; i += blockDim.x) {
+                const float4 x = reinterpret_cast<const float4*>(xs)[i], w = reinterpret_cast<const float4*>(p.norm)[i];
+                if (p.x_out) reinterpret_cast<float4*>(p.x_out + static_cast<size_t>(t) * p.width)[i] = x;
+                float4 h = make_float4(x.x * inv * w.x, x.y * inv * w.y, x.z * inv * w.z, x.w * inv * w.w);
+                if (p.shift) {
+                    const float4 b = reinterpret_cast<const float4*>(before)[i], mu = reinterpret_cast<const float4*>(p.shift)[i];
+                    reinterpret_cast<float4*>(before)[i] = h;
+                    if (m == 1) reinterpret_cast<float4*>(p.shift_state + static_cast<size_t>(pos & 1) * p.width)[i] = h;
+                    else if (t == m - 1) reinterpret_cast<float4*>(h_last)[i] = h;
+                    h = make_float4(h.x + (b.x - h.x) * mu.x, h.y + (b.y - h.y) * mu.y, h.z + (b.z - h.z) * mu.z, h.w + (b.w - h.w) * mu.w);
+                }
+                OUT* dst = out + static_cast<size_t>(t) * ldo + 4 * i;
+                if constexpr (sizeof(OUT) == 4) {
+                    *reinterpret_cast<float4*>(dst) = h;
+                } else {
+                    const __nv_bfloat162 lo = __floats2bfloat162_rn(h.x, h.y), hi = __floats2bfloat162_rn(h.z, h.w);
+                    *reinterpret_cast<uint2*>(dst) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+                }
+            }
+            __syncthreads();
+            continue;
+        }
         for (uint32_t i = threadIdx.x; i < ldo; i += blockDim.x) {
             float h = 0.f;
             if (i < p.width) {
@@ -133,14 +160,14 @@ HF2Q_API int32_t hf2q_cuda_pre_norm(hf2q_ctx* ctx, void* stream, const hf2q_pre_
     static PerDeviceFlag f32f, bff;
     // long portions: a few rows per CTA while every SM keeps several CTAs
     const uint32_t run = p->shift && m >= 4u * 4u * static_cast<uint32_t>(ctx_sm_count(ctx)) ? 8 : p->shift && m >= 512 ? 4 : 1;
-    const dim3 grid((m + run - 1) / run);
+    const dim3 grid((m + run - 1) / run), block(p->width >= 2048 ? 512 : 256);
     cudaError_t e;
     if (out_dtype == HF2Q_DT_F32) {
         e = ensure_max_dynamic_smem(pre_norm_kernel<float>, 200 * 1024, f32f);
-        if (e == cudaSuccess) e = launch_pdl(pre_norm_kernel<float>, grid, dim3(256), smem, st, *p, m, run, static_cast<float*>(out), ldo, h_last);
+        if (e == cudaSuccess) e = launch_pdl(pre_norm_kernel<float>, grid, block, smem, st, *p, m, run, static_cast<float*>(out), ldo, h_last);
     } else if (out_dtype == HF2Q_DT_BF16) {
         e = ensure_max_dynamic_smem(pre_norm_kernel<__nv_bfloat16>, 200 * 1024, bff);
-        if (e == cudaSuccess) e = launch_pdl(pre_norm_kernel<__nv_bfloat16>, grid, dim3(256), smem, st, *p, m, run, static_cast<__nv_bfloat16*>(out), ldo, h_last);
+        if (e == cudaSuccess) e = launch_pdl(pre_norm_kernel<__nv_bfloat16>, grid, block, smem, st, *p, m, run, static_cast<__nv_bfloat16*>(out), ldo, h_last);
     } else {
         e = cudaErrorInvalidValue;
     }

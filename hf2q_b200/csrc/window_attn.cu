@@ -96,7 +96,7 @@ struct WarpAttn {
         for (int g = 0; g < GR; ++g) s[g] = 0.f;
         if (live) {
             const T* kr = kc + static_cast<size_t>(p % a.capacity) * dp;
-#pragma unroll 8
+#pragma unroll 4
             for (uint32_t c = 0; c < dp; c += 8) {
                 float k[8];
                 load8(kr + c, k);
@@ -122,7 +122,7 @@ struct WarpAttn {
         }
         __syncwarp();
         const uint32_t cnt = min(32u, hi - p0);
-#pragma unroll 8
+#pragma unroll 4
         for (uint32_t i = 0; i < cnt; ++i) {
             const T* vr = vc + static_cast<size_t>((p0 + i) % a.capacity) * dvp;
 #pragma unroll
