@@ -50,13 +50,9 @@ __device__ __forceinline__ void block_sum(float (&v)[N], float* red) {
 #pragma unroll
         for (int i = 0; i < N; ++i) red[i * 32 + (threadIdx.x >> 5)] = v[i];
     __syncthreads();
-    const uint32_t nw = blockDim.x >> 5;
+    const uint32_t lane = threadIdx.x & 31, nw = blockDim.x >> 5;
 #pragma unroll
-    for (int i = 0; i < N; ++i) {
-        float s = 0.f;
-        for (uint32_t w = 0; w < nw; ++w) s += red[i * 32 + w];
-        v[i] = s;
-    }
+    for (int i = 0; i < N; ++i) v[i] = warp_sum(lane < nw ? red[i * 32 + lane] : 0.f);
 }
 
 // Programmatic dependent launch.  Every kernel launched with launch_pdl() calls pdl_wait() before it touches
