@@ -24,6 +24,19 @@ __device__ __forceinline__ float group8_sum(float v) {
     v += __shfl_xor_sync(0xffffffffu, v, 4);
     return v;
 }
+// Sums of eight values over the eight lanes of a group, transposed: lane l ends with the sum of v[l] (seven shuffles).
+__device__ __forceinline__ float group8_transpose_sum(float (&v)[8], uint32_t l8) {
+#pragma unroll
+    for (int w = 4; w > 0; w >>= 1) {
+        const bool up = l8 & w;
+#pragma unroll
+        for (int i = 0; i < w; ++i) {
+            const float other = __shfl_xor_sync(0xffffffffu, up ? v[i] : v[i + w], w);
+            v[i] = (up ? v[i + w] : v[i]) + other;
+        }
+    }
+    return v[0];
+}
 // rows of `count` floats -> shared memory, asynchronously, 16 bytes at a time where both sides allow it; a warp takes
 // whole rows
 __device__ __forceinline__ void stage_rows(float* dst, uint32_t dst_ld, const float* src, size_t src_ld, uint32_t rows, uint32_t count) {
@@ -153,15 +166,22 @@ __global__ void __launch_bounds__(SC_THREADS) mlstm_kernel(const __grid_constant
         else cp_async_wait<0>();
         __syncthreads();
         const uint32_t n = min(static_cast<uint32_t>(SC_TB), m - t0);
-        auto token = [&](uint32_t j, float& num, float& den) {
-            Vec<RQ> k, q;
-            k.load(ks + (b * SC_TB + j) * DP + 4 * l8);
-            q.load(qs + (b * SC_TB + j) * DP + 4 * l8);
-            const float keep = gk[b][j], write = gw[b][j];
-            S.decay_axpy(keep, k, write * vs[b][j][col_s]);
-            N.decay_axpy(keep, k, write);
-            num = group8_sum(S.dot(q));
-            den = group8_sum(N.dot(q));
+        // a token's operands are read one token ahead of their use
+        struct Operands { Vec<RQ> k, q; float keep, write, v; };
+        auto fetch = [&](uint32_t j) {
+            Operands t;
+            t.k.load(ks + (b * SC_TB + j) * DP + 4 * l8);
+            t.q.load(qs + (b * SC_TB + j) * DP + 4 * l8);
+            t.keep = gk[b][j];
+            t.write = gw[b][j];
+            t.v = vs[b][j][col_s];
+            return t;
+        };
+        auto token = [&](const Operands& t, float& num, float& den) {      // this lane's part of both sums
+            S.decay_axpy(t.keep, t.k, t.write * t.v);
+            N.decay_axpy(t.keep, t.k, t.write);
+            num = S.dot(t.q);
+            den = N.dot(t.q);
         };
         auto finish = [&](uint32_t j, float num, float den) {
             if (live)
@@ -169,19 +189,22 @@ __global__ void __launch_bounds__(SC_THREADS) mlstm_kernel(const __grid_constant
         };
         uint32_t j0 = 0;
         for (; j0 + 8 <= n; j0 += 8) {                       // eight tokens without a branch; lane i of a group finishes token i
-            float num = 0.f, den = 0.f;
+            float num[8], den[8];
+            Operands t = fetch(j0);
 #pragma unroll
             for (uint32_t u = 0; u < 8; ++u) {
-                float x, y;
-                token(j0 + u, x, y);
-                num = l8 == u ? x : num;
-                den = l8 == u ? y : den;
+                const Operands next = fetch(j0 + (u < 7 ? u + 1 : 7));
+                token(t, num[u], den[u]);
+                t = next;
             }
-            finish(j0 + l8, num, den);
+            const float x = group8_transpose_sum(num, l8), y = group8_transpose_sum(den, l8);
+            finish(j0 + l8, x, y);
         }
         for (; j0 < n; ++j0) {
             float x, y;
-            token(j0, x, y);
+            token(fetch(j0), x, y);
+            x = group8_sum(x);
+            y = group8_sum(y);
             if (l8 == 0) finish(j0, x, y);
         }
         __syncthreads();
@@ -194,11 +217,16 @@ __global__ void __launch_bounds__(SC_THREADS) mlstm_kernel(const __grid_constant
 // ---------------------------------------------------------------- gated delta rule
 // S <- g S;  u = beta (v - S^T k);  S <- S + k u;  o = S^T q
 template <int RQ>
-__device__ __forceinline__ float delta_token(Vec<RQ>& S, const Vec<RQ>& g, const Vec<RQ>& k, const Vec<RQ>& q, float v, float beta) {
-    S.scale(g);
-    const float u = beta * (v - group8_sum(S.dot(k)));
-    S.axpy(k, u);
-    return group8_sum(S.dot(q));
+struct DeltaOperands {
+    Vec<RQ> g, k, q;
+    float v, beta;
+};
+template <int RQ>
+__device__ __forceinline__ float delta_token(Vec<RQ>& S, const DeltaOperands<RQ>& t) {          // this lane's part of o
+    S.scale(t.g);
+    const float u = t.beta * (t.v - group8_sum(S.dot(t.k)));
+    S.axpy(t.k, u);
+    return S.dot(t.q);
 }
 
 template <int RQ>
@@ -241,28 +269,33 @@ __global__ void __launch_bounds__(SC_THREADS) delta_scan_kernel(const __grid_con
         else cp_async_wait<0>();
         __syncthreads();
         const uint32_t n = min(static_cast<uint32_t>(SC_TB), m - t0);
-        auto token = [&](uint32_t j) {
+        auto fetch = [&](uint32_t j) {                       // read one token ahead of their use
             const uint32_t o = (b * SC_TB + j) * DP + 4 * l8;
-            Vec<RQ> dg, k, q;
-            dg.load(gs + o);
-            k.load(ks + o);
-            q.load(qs + o);
-            return delta_token<RQ>(S, dg, k, q, vs[b][j][col_s], bs[b][j]);
+            DeltaOperands<RQ> t;
+            t.g.load(gs + o);
+            t.k.load(ks + o);
+            t.q.load(qs + o);
+            t.v = vs[b][j][col_s];
+            t.beta = bs[b][j];
+            return t;
         };
         float* dst = out + static_cast<size_t>(t0) * a.heads * a.vdim + static_cast<size_t>(h) * a.vdim + col;
         const size_t row_o = static_cast<size_t>(a.heads) * a.vdim;
         uint32_t j0 = 0;
         for (; j0 + 8 <= n; j0 += 8) {                       // eight tokens without a branch; lane i of a group stores token i
-            float r = 0.f;
+            float r[8];
+            DeltaOperands<RQ> t = fetch(j0);
 #pragma unroll
             for (uint32_t u = 0; u < 8; ++u) {
-                const float x = token(j0 + u);
-                r = l8 == u ? x : r;
+                const DeltaOperands<RQ> next = fetch(j0 + (u < 7 ? u + 1 : 7));
+                r[u] = delta_token<RQ>(S, t);
+                t = next;
             }
-            if (live) dst[(j0 + l8) * row_o] = r;
+            const float x = group8_transpose_sum(r, l8);
+            if (live) dst[(j0 + l8) * row_o] = x;
         }
         for (; j0 < n; ++j0) {
-            const float r = token(j0);
+            const float r = group8_sum(delta_token<RQ>(S, fetch(j0)));
             if (l8 == 0 && live) dst[j0 * row_o] = r;
         }
         __syncthreads();
@@ -353,11 +386,13 @@ __global__ void __launch_bounds__(SC_THREADS) delta_step_kernel(const __grid_con
         gate[c] = low_rank_dot(a.g2, c, a.g_rank_ld, lr + a.a_rank_ld);
     }
     __syncthreads();
-    Vec<RQ> dg, k, q;
-    dg.load(gs + 4 * l8);
-    k.load(ks + 4 * l8);
-    q.load(qs + 4 * l8);
-    const float r = delta_token<RQ>(S, dg, k, q, vs[col_s], sigmoidf(a.proj[a.b_off + h]));
+    DeltaOperands<RQ> t;
+    t.g.load(gs + 4 * l8);
+    t.k.load(ks + 4 * l8);
+    t.q.load(qs + 4 * l8);
+    t.v = vs[col_s];
+    t.beta = sigmoidf(a.proj[a.b_off + h]);
+    const float r = group8_sum(delta_token<RQ>(S, t));
     if (live) {
         S.store(sp);
         if (l8 == 0) out[h * a.vdim + col] = r;
