@@ -4,8 +4,8 @@
 //   delta   gated delta rule, one decay per head and key channel
 //
 // Both keep S[key channel][value column] and treat a value column independently, so the state lives in registers:
-// eight lanes share a column (each holds key channels 32 c + 4 l .. + 3), a warp carries four columns, a CTA of four
-// warps sixteen columns of one head.  A token costs no block barrier; sums over the key channels are three shuffles.
+// sixteen lanes share a column (each holds key channels 32 c + 2 l and + 1), a warp carries two columns, a CTA of eight
+// warps sixteen columns of one head: the token chain is latency-bound, so many short warps beat few long ones.  A token costs no block barrier; sums over the key channels are four shuffles.
 // Tokens are staged in shared memory in batches by asynchronous copies, two batches in flight.  The state in memory
 // is [head][column][key channel, padded to 32] (f32), which makes a lane's channels consecutive.
 #include <math_constants.h>
@@ -16,19 +16,20 @@ namespace hf2q {
 namespace {
 using namespace seq;
 
-constexpr int SC_WARPS = 4, SC_COLS = 16, SC_TB = 16, SC_THREADS = SC_WARPS * 32;
+constexpr int SC_WARPS = 8, SC_COLS = 16, SC_TB = 16, SC_THREADS = SC_WARPS * 32;
 
-__device__ __forceinline__ float group8_sum(float v) {
+__device__ __forceinline__ float group_sum(float v) {
     v += __shfl_xor_sync(0xffffffffu, v, 1);
     v += __shfl_xor_sync(0xffffffffu, v, 2);
     v += __shfl_xor_sync(0xffffffffu, v, 4);
+    v += __shfl_xor_sync(0xffffffffu, v, 8);
     return v;
 }
-// Sums of eight values over the eight lanes of a group, transposed: lane l ends with the sum of v[l] (seven shuffles).
-__device__ __forceinline__ float group8_transpose_sum(float (&v)[8], uint32_t l8) {
+// Sums of sixteen values over the sixteen lanes of a group, transposed: lane l ends with the sum of v[l] (15 shuffles).
+__device__ __forceinline__ float group_transpose_sum(float (&v)[16], uint32_t l) {
 #pragma unroll
-    for (int w = 4; w > 0; w >>= 1) {
-        const bool up = l8 & w;
+    for (int w = 8; w > 0; w >>= 1) {
+        const bool up = l & w;
 #pragma unroll
         for (int i = 0; i < w; ++i) {
             const float other = __shfl_xor_sync(0xffffffffu, up ? v[i] : v[i + w], w);
@@ -58,44 +59,40 @@ __device__ __forceinline__ f2 f2_add(f2 a, f2 b) { f2 d; asm("add.rn.f32x2 %0, %
 __device__ __forceinline__ f2 f2_both(float a) { f2 d; asm("mov.b64 %0, {%1, %1};" : "=l"(d) : "f"(a)); return d; }
 __device__ __forceinline__ float f2_sum(f2 a) { float x, y; asm("mov.b64 {%0, %1}, %2;" : "=f"(x), "=f"(y) : "l"(a)); return x + y; }
 
-template <int RQ> struct Vec {                       // a lane's RQ groups of four key channels
-    f2 v[2 * RQ];
+template <int RQ> struct Vec {                       // a lane's RQ pairs of key channels
+    f2 v[RQ];
     __device__ __forceinline__ void load(const float* p) {
 #pragma unroll
-        for (int c = 0; c < RQ; ++c) {
-            const ulonglong2 q = *reinterpret_cast<const ulonglong2*>(p + 32 * c);
-            v[2 * c] = q.x;
-            v[2 * c + 1] = q.y;
-        }
+        for (int c = 0; c < RQ; ++c) v[c] = *reinterpret_cast<const f2*>(p + 32 * c);
     }
     __device__ __forceinline__ void zero() {
 #pragma unroll
-        for (int c = 0; c < 2 * RQ; ++c) v[c] = 0ull;
+        for (int c = 0; c < RQ; ++c) v[c] = 0ull;
     }
     __device__ __forceinline__ void store(float* p) const {
 #pragma unroll
-        for (int c = 0; c < RQ; ++c) *reinterpret_cast<ulonglong2*>(p + 32 * c) = make_ulonglong2(v[2 * c], v[2 * c + 1]);
+        for (int c = 0; c < RQ; ++c) *reinterpret_cast<f2*>(p + 32 * c) = v[c];
     }
-    // sum over this lane's channels, in four interleaved partial sums (two pairs)
+    // sum over this lane's channels, in two interleaved pairs of partial sums
     __device__ __forceinline__ float dot(const Vec& k) const {
-        f2 a = f2_mul(v[0], k.v[0]), b = f2_mul(v[1], k.v[1]);
+        f2 s[2] = {f2_mul(v[0], k.v[0]), 0ull};
 #pragma unroll
-        for (int c = 1; c < RQ; ++c) { a = f2_fma(v[2 * c], k.v[2 * c], a); b = f2_fma(v[2 * c + 1], k.v[2 * c + 1], b); }
-        return f2_sum(f2_add(a, b));
+        for (int c = 1; c < RQ; ++c) s[c & 1] = f2_fma(v[c], k.v[c], s[c & 1]);
+        return f2_sum(RQ > 1 ? f2_add(s[0], s[1]) : s[0]);
     }
     __device__ __forceinline__ void scale(const Vec& k) {
 #pragma unroll
-        for (int c = 0; c < 2 * RQ; ++c) v[c] = f2_mul(v[c], k.v[c]);
+        for (int c = 0; c < RQ; ++c) v[c] = f2_mul(v[c], k.v[c]);
     }
     __device__ __forceinline__ void axpy(const Vec& k, float a) {
         const f2 aa = f2_both(a);
 #pragma unroll
-        for (int c = 0; c < 2 * RQ; ++c) v[c] = f2_fma(k.v[c], aa, v[c]);
+        for (int c = 0; c < RQ; ++c) v[c] = f2_fma(k.v[c], aa, v[c]);
     }
     __device__ __forceinline__ void decay_axpy(float keep, const Vec& k, float a) {
         const f2 kk = f2_both(keep), aa = f2_both(a);
 #pragma unroll
-        for (int c = 0; c < 2 * RQ; ++c) v[c] = f2_fma(kk, v[c], f2_mul(k.v[c], aa));
+        for (int c = 0; c < RQ; ++c) v[c] = f2_fma(kk, v[c], f2_mul(k.v[c], aa));
     }
 };
 
@@ -111,8 +108,8 @@ __global__ void __launch_bounds__(SC_THREADS) mlstm_kernel(const __grid_constant
     pdl_trigger();
     pdl_wait();
     const uint32_t h = blockIdx.x, slice = blockIdx.y, n_slices = gridDim.y;
-    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, l8 = lane & 7;
-    const uint32_t col_s = warp * 4 + (lane >> 3), col0 = slice * SC_COLS, col = col0 + col_s;
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, lg = lane & 15;
+    const uint32_t col_s = warp * 2 + (lane >> 4), col0 = slice * SC_COLS, col = col0 + col_s;
     const uint32_t n_cols = min(static_cast<uint32_t>(SC_COLS), a.vdim - col0);
     const bool live = col < a.vdim;
     const float q_scale = 1.0f / sqrtf(static_cast<float>(a.dim));
@@ -156,8 +153,8 @@ __global__ void __launch_bounds__(SC_THREADS) mlstm_kernel(const __grid_constant
         cp_async_commit();
     };
     Vec<RQ> S, N;
-    float* sp = a.s + (static_cast<size_t>(h) * a.vdim + (live ? col : 0)) * DP + 4 * l8;
-    float* np = a.n + (static_cast<size_t>(h) * n_slices + slice) * DP + 4 * l8;
+    float* sp = a.s + (static_cast<size_t>(h) * a.vdim + (live ? col : 0)) * DP + 2 * lg;
+    float* np = a.n + (static_cast<size_t>(h) * n_slices + slice) * DP + 2 * lg;
     if (live) S.load(sp); else S.zero();
     N.load(np);
     stage(0, 0);
@@ -170,8 +167,8 @@ __global__ void __launch_bounds__(SC_THREADS) mlstm_kernel(const __grid_constant
         struct Operands { Vec<RQ> k, q; float keep, write, v; };
         auto fetch = [&](uint32_t j) {
             Operands t;
-            t.k.load(ks + (b * SC_TB + j) * DP + 4 * l8);
-            t.q.load(qs + (b * SC_TB + j) * DP + 4 * l8);
+            t.k.load(ks + (b * SC_TB + j) * DP + 2 * lg);
+            t.q.load(qs + (b * SC_TB + j) * DP + 2 * lg);
             t.keep = gk[b][j];
             t.write = gw[b][j];
             t.v = vs[b][j][col_s];
@@ -188,29 +185,29 @@ __global__ void __launch_bounds__(SC_THREADS) mlstm_kernel(const __grid_constant
                 out[static_cast<size_t>(t0 + j) * a.heads * a.vdim + static_cast<size_t>(h) * a.vdim + col] = num * q_scale / (fmaxf(fabsf(den * q_scale), ge[b][j]) + 1e-6f);
         };
         uint32_t j0 = 0;
-        for (; j0 + 8 <= n; j0 += 8) {                       // eight tokens without a branch; lane i of a group finishes token i
-            float num[8], den[8];
+        for (; j0 + 16 <= n; j0 += 16) {                     // sixteen tokens without a branch; lane i of a group finishes token i
+            float num[16], den[16];
             Operands t = fetch(j0);
 #pragma unroll
-            for (uint32_t u = 0; u < 8; ++u) {
-                const Operands next = fetch(j0 + (u < 7 ? u + 1 : 7));
+            for (uint32_t u = 0; u < 16; ++u) {
+                const Operands next = fetch(j0 + (u < 15 ? u + 1 : 15));
                 token(t, num[u], den[u]);
                 t = next;
             }
-            const float x = group8_transpose_sum(num, l8), y = group8_transpose_sum(den, l8);
-            finish(j0 + l8, x, y);
+            const float x = group_transpose_sum(num, lg), y = group_transpose_sum(den, lg);
+            finish(j0 + lg, x, y);
         }
         for (; j0 < n; ++j0) {
             float x, y;
             token(fetch(j0), x, y);
-            x = group8_sum(x);
-            y = group8_sum(y);
-            if (l8 == 0) finish(j0, x, y);
+            x = group_sum(x);
+            y = group_sum(y);
+            if (lg == 0) finish(j0, x, y);
         }
         __syncthreads();
     }
     if (live) S.store(sp);
-    if (warp == 0 && lane < 8) N.store(np);
+    if (warp == 0 && lane < 16) N.store(np);
     if (warp == SC_WARPS - 1 && lane == 0) *mp = mx;
 }
 
@@ -224,7 +221,7 @@ struct DeltaOperands {
 template <int RQ>
 __device__ __forceinline__ float delta_token(Vec<RQ>& S, const DeltaOperands<RQ>& t) {          // this lane's part of o
     S.scale(t.g);
-    const float u = t.beta * (t.v - group8_sum(S.dot(t.k)));
+    const float u = t.beta * (t.v - group_sum(S.dot(t.k)));
     S.axpy(t.k, u);
     return S.dot(t.q);
 }
@@ -242,8 +239,8 @@ __global__ void __launch_bounds__(SC_THREADS) delta_scan_kernel(const __grid_con
     pdl_trigger();
     pdl_wait();
     const uint32_t h = blockIdx.x, slice = blockIdx.y, kvh = h / (a.heads / a.kv_heads);
-    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, l8 = lane & 7;
-    const uint32_t col_s = warp * 4 + (lane >> 3), col0 = slice * SC_COLS, col = col0 + col_s;
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, lg = lane & 15;
+    const uint32_t col_s = warp * 2 + (lane >> 4), col0 = slice * SC_COLS, col = col0 + col_s;
     const uint32_t n_cols = min(static_cast<uint32_t>(SC_COLS), a.vdim - col0);
     const bool live = col < a.vdim;
     const uint32_t qk = a.kv_heads * a.dim, ld = 2 * qk + a.heads * a.vdim;
@@ -261,7 +258,7 @@ __global__ void __launch_bounds__(SC_THREADS) delta_scan_kernel(const __grid_con
         cp_async_commit();
     };
     Vec<RQ> S;
-    float* sp = a.s + (static_cast<size_t>(h) * a.vdim + (live ? col : 0)) * DP + 4 * l8;
+    float* sp = a.s + (static_cast<size_t>(h) * a.vdim + (live ? col : 0)) * DP + 2 * lg;
     if (live) S.load(sp); else S.zero();
     stage(0, 0);
     for (uint32_t t0 = 0, b = 0; t0 < m; t0 += SC_TB, b ^= 1) {
@@ -270,7 +267,7 @@ __global__ void __launch_bounds__(SC_THREADS) delta_scan_kernel(const __grid_con
         __syncthreads();
         const uint32_t n = min(static_cast<uint32_t>(SC_TB), m - t0);
         auto fetch = [&](uint32_t j) {                       // read one token ahead of their use
-            const uint32_t o = (b * SC_TB + j) * DP + 4 * l8;
+            const uint32_t o = (b * SC_TB + j) * DP + 2 * lg;
             DeltaOperands<RQ> t;
             t.g.load(gs + o);
             t.k.load(ks + o);
@@ -282,21 +279,21 @@ __global__ void __launch_bounds__(SC_THREADS) delta_scan_kernel(const __grid_con
         float* dst = out + static_cast<size_t>(t0) * a.heads * a.vdim + static_cast<size_t>(h) * a.vdim + col;
         const size_t row_o = static_cast<size_t>(a.heads) * a.vdim;
         uint32_t j0 = 0;
-        for (; j0 + 8 <= n; j0 += 8) {                       // eight tokens without a branch; lane i of a group stores token i
-            float r[8];
+        for (; j0 + 16 <= n; j0 += 16) {                     // sixteen tokens without a branch; lane i of a group stores token i
+            float r[16];
             DeltaOperands<RQ> t = fetch(j0);
 #pragma unroll
-            for (uint32_t u = 0; u < 8; ++u) {
-                const DeltaOperands<RQ> next = fetch(j0 + (u < 7 ? u + 1 : 7));
+            for (uint32_t u = 0; u < 16; ++u) {
+                const DeltaOperands<RQ> next = fetch(j0 + (u < 15 ? u + 1 : 15));
                 r[u] = delta_token<RQ>(S, t);
                 t = next;
             }
-            const float x = group8_transpose_sum(r, l8);
-            if (live) dst[(j0 + l8) * row_o] = x;
+            const float x = group_transpose_sum(r, lg);
+            if (live) dst[(j0 + lg) * row_o] = x;
         }
         for (; j0 < n; ++j0) {
-            const float r = group8_sum(delta_token<RQ>(S, fetch(j0)));
-            if (l8 == 0 && live) dst[j0 * row_o] = r;
+            const float r = group_sum(delta_token<RQ>(S, fetch(j0)));
+            if (lg == 0 && live) dst[j0 * row_o] = r;
         }
         __syncthreads();
     }
@@ -332,15 +329,15 @@ __global__ void __launch_bounds__(SC_THREADS) delta_step_kernel(const __grid_con
     extern __shared__ __align__(16) float lr[];                     // a1 [a_rank_ld], g1 [g_rank_ld]
     pdl_trigger();
     const uint32_t h = blockIdx.x, slice = blockIdx.y, rep = a.heads / a.kv_heads, kvh = h / rep;
-    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, l8 = lane & 7;
-    const uint32_t col_s = warp * 4 + (lane >> 3), col0 = slice * SC_COLS, col = col0 + col_s;
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, lg = lane & 15;
+    const uint32_t col_s = warp * 2 + (lane >> 4), col0 = slice * SC_COLS, col = col0 + col_s;
     const uint32_t n_cols = min(static_cast<uint32_t>(SC_COLS), a.vdim - col0);
     const bool live = col < a.vdim;
     for (uint32_t i = threadIdx.x; i < a.dim; i += SC_THREADS)       // weights: towards L2 before the wait
         for (uint32_t c = 0; c < a.a_rank_ld; c += 64) prefetch_l2(static_cast<const __nv_bfloat16*>(a.a2) + (static_cast<size_t>(h) * a.dim + i) * a.a_rank_ld + c);
     pdl_wait();
     Vec<RQ> S;
-    float* sp = a.s + (static_cast<size_t>(h) * a.vdim + (live ? col : 0)) * DP + 4 * l8;
+    float* sp = a.s + (static_cast<size_t>(h) * a.vdim + (live ? col : 0)) * DP + 2 * lg;
     if (live) S.load(sp); else S.zero();
     const uint32_t pos = *a.pos, qk = a.kv_heads * a.dim;
     for (uint32_t i = threadIdx.x; i < a.a_rank_ld; i += SC_THREADS) lr[i] = a.proj[a.a1_off + i];
@@ -387,15 +384,15 @@ __global__ void __launch_bounds__(SC_THREADS) delta_step_kernel(const __grid_con
     }
     __syncthreads();
     DeltaOperands<RQ> t;
-    t.g.load(gs + 4 * l8);
-    t.k.load(ks + 4 * l8);
-    t.q.load(qs + 4 * l8);
+    t.g.load(gs + 2 * lg);
+    t.k.load(ks + 2 * lg);
+    t.q.load(qs + 2 * lg);
     t.v = vs[col_s];
     t.beta = sigmoidf(a.proj[a.b_off + h]);
-    const float r = group8_sum(delta_token<RQ>(S, t));
+    const float r = group_sum(delta_token<RQ>(S, t));
     if (live) {
         S.store(sp);
-        if (l8 == 0) out[h * a.vdim + col] = r;
+        if (lg == 0) out[h * a.vdim + col] = r;
     }
 }
 
