@@ -18,7 +18,8 @@ from . import _lib, ops
 from .decoder import GreedyDecoder
 from .mixers import MIXERS, LayerRun, Workspace
 from .safetensors import SafetensorsFile
-from .seqops import (EPI_ADD, EPI_GELU, EPI_NONE, EPI_SOFTCAP, PRO_NONE, PRO_NORM, DenseWeight, Embed, Matvec, PreNorm, SeqOps, pad8, ptr, struct)
+from .state import StatePool
+from .seqops import (EPI_ADD, EPI_GELU, EPI_NONE, EPI_SOFTCAP, PRO_NONE, PRO_NORM, DenseWeight, Embed, Matvec, PreNorm, SeqOps, pad8, struct)
 
 
 def _bad(msg: str):
@@ -155,7 +156,6 @@ class FomatarDecoder(GreedyDecoder):
         if (self.head.n, self.head.k_raw) != (cfg.vocab, w):
             raise _bad(f"head: shape {[self.head.n, self.head.k_raw]}, expected {[cfg.vocab, w]}")
 
-        from .state import StatePool
         self.pool = StatePool(n_slots, dev)
         for r, run in enumerate(self.runs):
             self.pool.recurrent(f"r{r}.shift", 2, w)

@@ -11,7 +11,7 @@ from dataclasses import dataclass
 
 import torch
 
-from .seqops import (EPI_ADD, EPI_NONE, PRO_GATED, Delta, DenseWeight, GatedHeads, MLstm, Matvec, SeqOps, WindowAttn, pad8, pad32, ptr, struct)
+from .seqops import EPI_ADD, PRO_GATED, Delta, DenseWeight, GatedHeads, MLstm, Matvec, SeqOps, WindowAttn, pad8, pad32, struct
 from .ops import DT_BF16, DT_F32
 
 

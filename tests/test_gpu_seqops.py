@@ -30,7 +30,7 @@ def rel(got, want):
 
 
 # ---- products ---------------------------------------------------------------------------------------------------
-@pytest.mark.parametrize("m,n,k", [(1, 5, 8), (2, 300, 72), (3, 64, 4096), (8, 129, 1000), (9, 24, 8), (64, 640, 320), (130, 301, 72), (257, 1030, 200),
+@pytest.mark.parametrize("m,n,k", [(1, 5, 8), (2, 300, 72), (3, 64, 4096), (8, 129, 1000), (9, 24, 8), (64, 616, 312), (130, 301, 72), (257, 1030, 200),
                                    (600, 4096, 512), (1500, 2304, 264)])
 @pytest.mark.parametrize("xd", [torch.float32, torch.bfloat16])
 def test_product_and_epilogues(sop, m, n, k, xd):
@@ -76,7 +76,7 @@ def test_product_refuses_bad_arguments(sop):
 
 
 # ---- row prologues ------------------------------------------------------------------------------------------------
-@pytest.mark.parametrize("width", [1, 52, 320, 4096])
+@pytest.mark.parametrize("width", [1, 52, 344, 4096])
 @pytest.mark.parametrize("m", [1, 2, 7])
 def test_pre_norm_and_token_shift(sop, width, m):
     rng = np.random.default_rng(width + m)
