@@ -102,20 +102,32 @@ SIGNATURES = {
     "hf2q_cuda_attn_prefill": (i32, [vp, vp, vp, u32, u32, vp, u32, vp, u32]),
     "hf2q_cuda_argmax": (i32, [vp, vp, vp, u32, vp, vp]),
     "hf2q_cuda_add": (i32, [vp, vp, vp, vp, u64]),
-    "hf2q_cuda_dense_matmul": (i32, [vp, vp, vp, u32, u32, vp, vp, u32, u32, u32, u32, u32, u32, vp, C.c_float]),
+    "hf2q_cuda_dense_matmul": (i32, [vp, vp, vp, u32, u32, vp, vp, u32, u32, u32, u32, u32, u32, vp, C.c_float, vp]),
+    "hf2q_cuda_dense_grouped": (i32, [vp, vp, vp, vp, u32, u32, vp, vp, u32, u32, u32, u32, u32, u32, C.c_float]),
+    "hf2q_cuda_moe_sigmoid_topk": (i32, [vp, vp, vp, u32, vp, vp, u32, u32, u32]),
+    "hf2q_cuda_sort_rows": (i32, [vp, vp, vp, u32, u32, u32, u32, vp, u32, u32, vp, vp, vp, vp]),
     "hf2q_cuda_pre_norm": (i32, [vp, vp, vp, u32, vp, u32, u32, vp]),
     "hf2q_cuda_gated_heads": (i32, [vp, vp, vp, u32, vp, u32, u32]),
+    "hf2q_cuda_hyper_norm": (i32, [vp, vp, vp, u32, vp, u32, u32]),
+    "hf2q_cuda_expert_glu_step": (i32, [vp, vp, vp]),
+    "hf2q_cuda_expert_down_step": (i32, [vp, vp, vp]),
     "hf2q_cuda_dense_matvec": (i32, [vp, vp, u32, vp, u32]),
     "hf2q_cuda_embed": (i32, [vp, vp, vp, vp, u32, vp]),
     "hf2q_cuda_window_attn_scratch_bytes": (i32, [vp, vp, C.POINTER(u64)]),
     "hf2q_cuda_window_attn_decode": (i32, [vp, vp, vp, vp, vp, u64]),
     "hf2q_cuda_window_attn_append": (i32, [vp, vp, vp, u32, vp]),
     "hf2q_cuda_window_attn_prefill": (i32, [vp, vp, vp, u32, vp, vp, u32, vp, u32, u32]),
+    "hf2q_cuda_latent_scratch_bytes": (i32, [vp, vp, C.POINTER(u64)]),
+    "hf2q_cuda_latent_decode": (i32, [vp, vp, vp, vp, vp, u64]),
+    "hf2q_cuda_latent_append": (i32, [vp, vp, vp, u32, vp]),
     "hf2q_cuda_mlstm": (i32, [vp, vp, vp, u32, vp]),
     "hf2q_cuda_delta_step": (i32, [vp, vp, vp, vp, vp]),
     "hf2q_cuda_delta_prep": (i32, [vp, vp, vp, u32, vp, vp, vp, vp, u32]),
     "hf2q_cuda_delta_decay": (i32, [vp, vp, vp, u32, vp]),
     "hf2q_cuda_delta_scan": (i32, [vp, vp, vp, u32, vp, vp, vp, vp]),
+    "hf2q_cuda_ssd_step": (i32, [vp, vp, vp, vp]),
+    "hf2q_cuda_ssd_prep": (i32, [vp, vp, vp, u32, vp, vp, vp]),
+    "hf2q_cuda_ssd_scan": (i32, [vp, vp, vp, u32, vp, vp, vp, vp]),
     "hf2q_cuda_state_tail": (i32, [vp, vp, vp, u32, vp, vp, u32, vp]),
     "hf2q_cuda_launch_count": (u64, [vp]),
     "hf2q_cuda_sm_count": (i32, [vp]),

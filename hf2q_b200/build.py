@@ -15,7 +15,7 @@ PKG = Path(__file__).resolve().parent
 CSRC = PKG / "csrc"
 OUT = PKG / "libhf2q_cuda.so"
 SOURCES = ["api.cu", "k0_dequant.cu", "k1_gemv.cu", "k1_gemv_mma.cu", "k2_gemm_tc.cu", "k4_moe_prep.cu", "moe_router.cu", "ffn_elementwise.cu", "decoder_ops.cu", "comm_nccl.cu", "ffn_builders.cu",
-           "dense_bf16.cu", "seq_ops.cu", "scan.cu", "window_attn.cu"]
+           "dense_bf16.cu", "seq_ops.cu", "scan.cu", "window_attn.cu", "latent_attn.cu", "experts_bf16.cu"]
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
     "-Xcompiler", "-fPIC,-fvisibility=hidden",
@@ -48,11 +48,14 @@ def build(force: bool = False, verbose: bool = False) -> Path:
     env.pop("CXX", None)
     env.pop("CC", None)
     objs, procs = [], []
+    headers = max(d.stat().st_mtime for d in [*CSRC.glob("*.cuh"), *CSRC.glob("*.h"), PKG.parent / "include" / "hf2q_cuda.h"])
     for src in SOURCES:
         obj = objdir / (src + ".o")
+        objs.append(str(obj))
+        if not force and obj.exists() and obj.stat().st_mtime > max(headers, (CSRC / src).stat().st_mtime):
+            continue
         cmd = [_nvcc(), *NVCC_FLAGS, *shlex.split(os.environ.get("HF2Q_NVCC_EXTRA", "")), "-ccbin", "g++", "-c", str(CSRC / src), "-o", str(obj)]
         procs.append((src, subprocess.Popen(cmd, env=env, stdout=subprocess.PIPE, stderr=subprocess.STDOUT, text=True)))
-        objs.append(str(obj))
     log = []
     for src, p in procs:
         out, _ = p.communicate()

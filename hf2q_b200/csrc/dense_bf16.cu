@@ -7,6 +7,8 @@
 //                         swizzle, two accumulator buffers in tensor memory so that the epilogue of a tile runs under
 //                         the main loop of the next.
 //   dense_gemm_f32_kernel more rows, f32 activations: CUDA-core tiles in full 32-bit arithmetic.
+// Both take rows sorted by group (expert) with one weight matrix per group as well.
+#include "matvec_stream.cuh"
 #include "seq_common.cuh"
 #include "tc_common.cuh"
 
@@ -17,6 +19,7 @@ using namespace seq;
 __device__ __forceinline__ float epilogue_value(float v, uint32_t epi, float cap) {
     if (epi == HF2Q_EPI_GELU) return gelu_tanhf(v);
     if (epi == HF2Q_EPI_SOFTCAP) return cap * tanhf(v / cap);
+    if (epi == HF2Q_EPI_SCALE) return v * cap;
     return v;
 }
 
@@ -73,42 +76,30 @@ struct MatvecSegs {
     uint32_t blocks0;        // CTAs of segment 0
 };
 
-// One-row product.  A CTA owns a contiguous range of weight rows, cut into chunks of MV_CHUNK elements; its warps take
-// the chunks in turn, each through a private ring of bulk copies that starts filling before the wait for the previous
-// kernel (weights never change).  Chunk sums of a block of rows meet in shared memory and are added in chunk order.
-constexpr int MR_WARPS = 16, MR_THREADS = MR_WARPS * 32, MV_CHUNK = 1024, MR_STAGES = 3, MR_PART = 2048;
-constexpr uint32_t MR_RING = MR_WARPS * MR_STAGES * MV_CHUNK * 2;
-
+// One-row product: the CTA's weight rows run through a MatvecStream; the layer's row prologue fills x in front of it.
 template <int PRO>
 __global__ void __launch_bounds__(MR_THREADS) dense_matvec_kernel(const __grid_constant__ MatvecSegs p, uint32_t* status) {
     extern __shared__ __align__(128) uint8_t mv_smem[];                 // ring, then x [k] f32
     __shared__ float red[64];
-    __shared__ float part[2][MR_PART];
-    __shared__ uint64_t bars[MR_WARPS][MR_STAGES];
+    __shared__ MatvecShared sh;
     pdl_trigger();
     const bool second = blockIdx.x >= p.blocks0;
     const hf2q_matvec& s = p.s[second];
     const uint32_t blk = blockIdx.x - (second ? p.blocks0 : 0u), n_blk = second ? gridDim.x - p.blocks0 : p.blocks0;
-    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    __nv_bfloat16* ring = reinterpret_cast<__nv_bfloat16*>(mv_smem) + static_cast<size_t>(warp) * MR_STAGES * MV_CHUNK;
+    const uint32_t warp = threadIdx.x >> 5;
     float* xs = reinterpret_cast<float*>(mv_smem + MR_RING);
+    const bool pairs = epi_pairs(s.epilogue);
     // rows [row0, row1) of this CTA, spread evenly
-    const uint32_t row0 = static_cast<uint32_t>(static_cast<uint64_t>(s.n) * blk / n_blk), row1 = static_cast<uint32_t>(static_cast<uint64_t>(s.n) * (blk + 1) / n_blk);
-    const uint32_t per_row = (s.k + MV_CHUNK - 1) / MV_CHUNK, n_chunks = (row1 - row0) * per_row;
+    const uint32_t unit = pairs ? 2 : 1, units = s.n / unit;
+    const uint32_t row0 = unit * static_cast<uint32_t>(static_cast<uint64_t>(units) * blk / n_blk), row1 = unit * static_cast<uint32_t>(static_cast<uint64_t>(units) * (blk + 1) / n_blk);
+    const uint32_t per_row = (s.k + MV_CHUNK - 1) / MV_CHUNK;
     const __nv_bfloat16* w = static_cast<const __nv_bfloat16*>(s.w) + static_cast<size_t>(row0) * s.k;
-    auto issue = [&](uint32_t i) {                                      // this warp's chunk number i
-        const uint32_t c = i * MR_WARPS + warp;
-        if (c >= n_chunks) return;
-        const uint32_t k0 = (c % per_row) * MV_CHUNK, bytes = min(static_cast<uint32_t>(MV_CHUNK), s.k - k0) * 2;
-        uint64_t* bar = &bars[warp][i % MR_STAGES];
-        mbar_arrive_expect_tx(bar, bytes);
-        bulk_g2s(ring + (i % MR_STAGES) * MV_CHUNK, w + static_cast<size_t>(c / per_row) * s.k + k0, bytes, bar);
+    auto chunk = [&](uint32_t c) {
+        const uint32_t k0 = (c % per_row) * MV_CHUNK;
+        return MatvecChunk{w + static_cast<size_t>(c / per_row) * s.k + k0, k0, min(static_cast<uint32_t>(MV_CHUNK), s.k - k0)};
     };
-    if (lane == 0) {
-        for (int i = 0; i < MR_STAGES; ++i) mbar_init(&bars[warp][i], 1);
-        mbar_fence_init();
-        for (int i = 0; i < MR_STAGES; ++i) issue(i);
-    }
+    MatvecStream stream(mv_smem, sh, (row1 - row0) * per_row, status);
+    stream.start(chunk);
     pdl_wait();
     if constexpr (PRO == HF2Q_PRO_NONE) {
         for (uint32_t i = threadIdx.x; i < s.k; i += MR_THREADS) xs[i] = s.x[i];
@@ -132,63 +123,52 @@ __global__ void __launch_bounds__(MR_THREADS) dense_matvec_kernel(const __grid_c
             }
             xs[i] = h;
         }
+    } else if constexpr (PRO == HF2Q_PRO_HYPER) {
+        const hf2q_hyper& q = s.hyper;
+        __shared__ float coef[HYPER_COEF];
+        // every CTA makes the whole row and stores its share of the new streams
+        const uint32_t lo = static_cast<uint32_t>(static_cast<uint64_t>(q.width) * blk / n_blk) & ~3u;
+        const uint32_t hi = blk + 1 == n_blk ? q.width : static_cast<uint32_t>(static_cast<uint64_t>(q.width) * (blk + 1) / n_blk) & ~3u;
+        const float inv = hyper_row(q, 0, xs, coef, red, lo, hi);
+        for (uint32_t i = threadIdx.x; i < s.k; i += MR_THREADS) {
+            const float h = i < q.width ? (q.norm ? xs[i] * inv * q.norm[i] : xs[i]) : 0.f;
+            xs[i] = h;
+            if (q.h_out && i >= lo && i < hi) q.h_out[i] = h;
+        }
     } else {
         for (uint32_t i = s.gated.heads * s.gated.head_dim + threadIdx.x; i < s.k; i += MR_THREADS) xs[i] = 0.f;
-        gated_heads_row<float>(s.gated, 0, xs, warp, MR_WARPS);
+        if (s.gated.kind == HF2Q_GATE_SILU_FIRST) silu_group_norm_row<float>(s.gated, 0, xs, xs);
+        else gated_heads_row<float>(s.gated, 0, xs, warp, MR_WARPS);
     }
     __syncthreads();
-    const uint32_t block_rows = max(1u, MR_PART / per_row);
-    bool ok = true;
-    uint32_t i = 0;                                                     // this warp's chunk counter
-    for (uint32_t r0 = 0, pb = 0; r0 < row1 - row0; r0 += block_rows, pb ^= 1) {
-        const uint32_t rows = min(block_rows, row1 - row0 - r0), c_end = (r0 + rows) * per_row;
-        for (uint32_t c = i * MR_WARPS + warp; c < c_end; ++i, c += MR_WARPS) {
-            const uint32_t st = i % MR_STAGES, kc = c % per_row, k0 = kc * MV_CHUNK, len = min(static_cast<uint32_t>(MV_CHUNK), s.k - k0);
-            if (ok) ok = mbar_wait_bounded(&bars[warp][st], (i / MR_STAGES) & 1, status);
-            ok = __all_sync(0xffffffffu, ok);
-            float acc = 0.f;
-            if (ok) {
-                const uint4* wv = reinterpret_cast<const uint4*>(ring + st * MV_CHUNK);
-                const float* xv = xs + k0;
-#pragma unroll
-                for (int u = 0; u < MV_CHUNK / 256; ++u) {
-                    const uint32_t e = lane + 32 * u;
-                    if (8 * e < len) {
-                        const uint4 v = wv[e];
-                        const float4 a = *reinterpret_cast<const float4*>(xv + 8 * e), b = *reinterpret_cast<const float4*>(xv + 8 * e + 4);
-                        acc = fmaf(bf_lo(v.x), a.x, acc); acc = fmaf(bf_hi(v.x), a.y, acc); acc = fmaf(bf_lo(v.y), a.z, acc); acc = fmaf(bf_hi(v.y), a.w, acc);
-                        acc = fmaf(bf_lo(v.z), b.x, acc); acc = fmaf(bf_hi(v.z), b.y, acc); acc = fmaf(bf_lo(v.w), b.z, acc); acc = fmaf(bf_hi(v.w), b.w, acc);
-                    }
-                }
-            }
-            __syncwarp();                                               // every lane has read the stage
-            if (lane == 0 && ok) issue(i + MR_STAGES);
-            acc = warp_sum(acc);
-            if (lane == 0) part[pb][c - r0 * per_row] = acc;
-        }
-        __syncthreads();                                                // (the other half of `part` is free: its readers passed this barrier)
-        for (uint32_t r = threadIdx.x; r < rows; r += MR_THREADS) {
-            float v = 0.f;
-            for (uint32_t kc = 0; kc < per_row; ++kc) v += part[pb][r * per_row + kc];
-            const uint32_t row = row0 + r0 + r;
-            v = epilogue_value(v, s.epilogue, s.cap);
-            if (s.epilogue == HF2Q_EPI_ADD) v += s.residual[row];
-            s.y[row] = v;
-        }
-    }
+    stream.run(chunk, xs, row1 - row0, per_row, unit, [&](uint32_t r, float v0, float v1) {
+        const uint32_t row = row0 + r;
+        if (s.bias) { v0 += s.bias[row]; if (pairs) v1 += s.bias[row + 1]; }
+        if (pairs) { s.y[row / 2] = glu_value(v0, v1, s.epilogue, s.cap); return; }
+        float v = epilogue_value(v0, s.epilogue, s.cap);
+        if (s.epilogue == HF2Q_EPI_ADD) v += s.residual[row];
+        s.y[row] = v;
+    });
 }
 
 struct DenseArgs {
     const void* x;
     const __nv_bfloat16* w;
     void* y;
-    const float* residual;
+    const float *residual, *bias;
     uint32_t ldx, ldy, m, n, k, epi;
     float cap;
+    hf2q_row_groups g;       // grouped products: rows of x sorted by group, w [groups][n][k]
 };
+// where a grouped product's output row goes, and what it is scaled with before the activation
+struct GroupRow { size_t out; float scale; };
+__device__ __forceinline__ GroupRow group_row(const DenseArgs& p, uint32_t sorted) {
+    const uint32_t routed = p.g.perm[sorted];
+    return {p.g.scatter ? routed : sorted, p.g.row_scale ? p.g.row_scale[routed] : 1.0f};
+}
 
-template <typename X, typename Y, int M>
-__global__ void __launch_bounds__(MV_THREADS) dense_matvec_m_kernel(const DenseArgs p) {
+template <typename X, typename Y, int M, int RW>
+__global__ void __launch_bounds__(MV_THREADS) dense_matvec_m_kernel(const DenseArgs p) {          // RW = 2: rows are pairs
     extern __shared__ __align__(16) float xs[];
     pdl_trigger();
     pdl_wait();
@@ -197,19 +177,26 @@ __global__ void __launch_bounds__(MV_THREADS) dense_matvec_m_kernel(const DenseA
         for (uint32_t i = threadIdx.x; i < p.k; i += MV_THREADS)
             xs[static_cast<size_t>(m) * p.k + i] = m < static_cast<int>(p.m) ? to_f32(x[static_cast<size_t>(m) * p.ldx + i]) : 0.f;
     __syncthreads();
-    const uint32_t row = blockIdx.x * MV_WARPS + (threadIdx.x >> 5);
+    const uint32_t row = (blockIdx.x * MV_WARPS + (threadIdx.x >> 5)) * RW;
     if (row >= p.n) return;
-    float acc[1][M];
+    float acc[RW][M];
 #pragma unroll
-    for (int m = 0; m < M; ++m) acc[0][m] = 0.f;
-    matvec_rows<1, M>(p.w, row, p.n, p.k, xs, acc);
+    for (int r = 0; r < RW; ++r)
+#pragma unroll
+        for (int m = 0; m < M; ++m) acc[r][m] = 0.f;
+    matvec_rows<RW, M>(p.w, row, p.n, p.k, xs, acc);
     if ((threadIdx.x & 31) == 0) {
 #pragma unroll
         for (int m = 0; m < M; ++m)
             if (m < static_cast<int>(p.m)) {
-                const size_t o = static_cast<size_t>(m) * p.ldy + row;
-                float v = epilogue_value(acc[0][m], p.epi, p.cap);
-                if (p.epi == HF2Q_EPI_ADD) v += p.residual[o];
+                const size_t o = static_cast<size_t>(m) * p.ldy + row / RW;
+                float v = acc[0][m] + (p.bias ? p.bias[row] : 0.f);
+                if constexpr (RW == 2) {
+                    v = glu_value(v, acc[1][m] + (p.bias ? p.bias[row + 1] : 0.f), p.epi, p.cap);
+                } else {
+                    v = epilogue_value(v, p.epi, p.cap);
+                    if (p.epi == HF2Q_EPI_ADD) v += p.residual[o];
+                }
                 static_cast<Y*>(p.y)[o] = from_f32<Y>(v);
             }
     }
@@ -218,20 +205,29 @@ __global__ void __launch_bounds__(MV_THREADS) dense_matvec_m_kernel(const DenseA
 // ---------------------------------------------------------------- fp32 product on the CUDA cores
 constexpr int FT = 64, FK = 16;
 
-template <typename X, typename Y>
+template <typename X, typename Y, bool GROUPED>
 __global__ void __launch_bounds__(256) dense_gemm_f32_kernel(const DenseArgs p) {
     __shared__ float as[FK][FT + 4], bs[FK][FT + 4];
     pdl_trigger();
     pdl_wait();
     const X* x = static_cast<const X*>(p.x);
-    const uint32_t m0 = blockIdx.y * FT, n0 = blockIdx.x * FT;
+    uint32_t m0 = blockIdx.y * FT, m_end = p.m;
+    const uint32_t n0 = blockIdx.x * FT;
+    const __nv_bfloat16* w = p.w;
+    if constexpr (GROUPED) {
+        if (blockIdx.y >= p.g.header[0]) return;
+        const uint4 tile = reinterpret_cast<const uint4*>(p.g.tiles)[blockIdx.y];           // group, first sorted row, rows
+        w += static_cast<size_t>(tile.x) * p.n * p.k;
+        m0 = tile.y;
+        m_end = tile.y + tile.z;
+    }
     const uint32_t tr = threadIdx.x / 16, tc = threadIdx.x % 16;
     float acc[4][4] = {};
     for (uint32_t k0 = 0; k0 < p.k; k0 += FK) {
         for (uint32_t i = threadIdx.x; i < FT * FK; i += 256) {
             const uint32_t r = i / FK, c = i % FK;
-            as[c][r] = m0 + r < p.m && k0 + c < p.k ? to_f32(x[static_cast<size_t>(m0 + r) * p.ldx + k0 + c]) : 0.f;
-            bs[c][r] = n0 + r < p.n && k0 + c < p.k ? to_f32(p.w[static_cast<size_t>(n0 + r) * p.k + k0 + c]) : 0.f;
+            as[c][r] = m0 + r < m_end && k0 + c < p.k ? to_f32(x[static_cast<size_t>(m0 + r) * p.ldx + k0 + c]) : 0.f;
+            bs[c][r] = n0 + r < p.n && k0 + c < p.k ? to_f32(w[static_cast<size_t>(n0 + r) * p.k + k0 + c]) : 0.f;
         }
         __syncthreads();
 #pragma unroll
@@ -245,15 +241,27 @@ __global__ void __launch_bounds__(256) dense_gemm_f32_kernel(const DenseArgs p) 
         }
         __syncthreads();
     }
-    for (int i = 0; i < 4; ++i)
+    const bool pairs = epi_pairs(p.epi);
+    for (int i = 0; i < 4; ++i) {
+        const uint32_t r = m0 + 4 * tr + i;
+        if (r >= m_end) continue;
+        size_t row = r;
+        float scale = 1.0f;
+        if constexpr (GROUPED) { const GroupRow q = group_row(p, r); row = q.out; scale = q.scale; }
         for (int j = 0; j < 4; ++j) {
-            const uint32_t r = m0 + 4 * tr + i, c = n0 + 4 * tc + j;
-            if (r >= p.m || c >= p.n) continue;
-            const size_t o = static_cast<size_t>(r) * p.ldy + c;
-            float v = epilogue_value(acc[i][j], p.epi, p.cap);
-            if (p.epi == HF2Q_EPI_ADD) v += p.residual[o];
+            const uint32_t c = n0 + 4 * tc + j;
+            if (c >= p.n || (pairs && (j & 1))) continue;
+            const size_t o = row * p.ldy + (pairs ? c / 2 : c);
+            float v = acc[i][j] * scale + (p.bias ? p.bias[c] : 0.f);
+            if (pairs) {
+                v = glu_value(v, acc[i][j + 1 < 4 ? j + 1 : j] * scale + (p.bias ? p.bias[c + 1] : 0.f), p.epi, p.cap);
+            } else {
+                v = epilogue_value(v, p.epi, p.cap);
+                if (p.epi == HF2Q_EPI_ADD) v += p.residual[o];
+            }
             static_cast<Y*>(p.y)[o] = from_f32<Y>(v);
         }
+    }
 }
 
 // ---------------------------------------------------------------- tcgen05 product
@@ -276,7 +284,23 @@ __device__ __forceinline__ void st_global_v8(float* p, const float* v) {
                  : "memory");
 }
 
-template <int NT, typename Y>
+// sixteen consecutive outputs, 32-byte aligned for f32 and 16-byte aligned for bf16
+__device__ __forceinline__ void store16(float* y, const float* v) {
+    st_global_v8(y, v);
+    st_global_v8(y + 8, v + 8);
+}
+__device__ __forceinline__ void store16(__nv_bfloat16* y, const float* v) {
+    uint32_t q[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+        const __nv_bfloat162 h = __floats2bfloat162_rn(v[2 * j], v[2 * j + 1]);
+        q[j] = *reinterpret_cast<const uint32_t*>(&h);
+    }
+    reinterpret_cast<uint4*>(y)[0] = make_uint4(q[0], q[1], q[2], q[3]);
+    reinterpret_cast<uint4*>(y)[1] = make_uint4(q[4], q[5], q[6], q[7]);
+}
+
+template <int NT, typename Y, bool GROUPED>
 __global__ void __launch_bounds__(TC_THREADS, 1) dense_gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w,
                                                                       const DenseArgs p, uint32_t* status) {
     extern __shared__ uint8_t smem_raw[];
@@ -286,7 +310,7 @@ __global__ void __launch_bounds__(TC_THREADS, 1) dense_gemm_tc_kernel(const __gr
     __shared__ uint64_t full[ST], empty[ST], d_full[2], d_empty[2];
     __shared__ uint32_t tmem_slot;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const uint32_t mt = (p.m + TC_M - 1) / TC_M, n_tiles = mt * ((p.n + NT - 1) / NT), nkb = (p.k + TC_K - 1) / TC_K;
+    const uint32_t nkb = (p.k + TC_K - 1) / TC_K;
     if (threadIdx.x == 0) {
         for (int i = 0; i < ST; ++i) { mbar_init(&full[i], 1); mbar_init(&empty[i], 1); }
         for (int i = 0; i < 2; ++i) { mbar_init(&d_full[i], 1); mbar_init(&d_empty[i], 4); }
@@ -299,12 +323,19 @@ __global__ void __launch_bounds__(TC_THREADS, 1) dense_gemm_tc_kernel(const __gr
     const uint32_t tmem = tmem_slot;
     pdl_trigger();
     pdl_wait();
+    const uint32_t mt = GROUPED ? p.g.header[0] : (p.m + TC_M - 1) / TC_M, n_tiles = mt * ((p.n + NT - 1) / NT);
+    const uint4* group_tiles = reinterpret_cast<const uint4*>(p.g.tiles);                // group, first sorted row, rows
     if (warp == 0) {
         if (lane == 0) {
             uint32_t it = 0;
             bool ok = true;
             for (uint32_t tile = blockIdx.x; tile < n_tiles && ok; tile += gridDim.x) {
-                const int row_x = static_cast<int>((tile % mt) * TC_M), row_w = static_cast<int>((tile / mt) * NT);
+                int row_x = static_cast<int>((tile % mt) * TC_M), row_w = static_cast<int>((tile / mt) * NT);
+                if constexpr (GROUPED) {
+                    const uint4 q = group_tiles[tile % mt];
+                    row_x = static_cast<int>(q.y);
+                    row_w += static_cast<int>(q.x * p.n);
+                }
                 for (uint32_t kb = 0; kb < nkb; ++kb, ++it) {
                     const uint32_t s = it % ST;
                     if (it >= ST) ok = mbar_wait_bounded(&empty[s], (it / ST - 1) & 1, status);
@@ -350,20 +381,49 @@ __global__ void __launch_bounds__(TC_THREADS, 1) dense_gemm_tc_kernel(const __gr
             ok = __all_sync(0xffffffffu, ok);
             if (!ok) break;
             tc::tc_fence_after();
-            const uint32_t row = (tile % mt) * TC_M + quad * 32 + lane, n0 = (tile / mt) * NT;
-            const uint32_t n_cols = min(static_cast<uint32_t>(NT), p.n - n0);
+            const uint32_t n0 = (tile / mt) * NT, n_cols = min(static_cast<uint32_t>(NT), p.n - n0);
+            size_t row = (tile % mt) * TC_M + quad * 32 + lane;
+            bool live = row < p.m;
+            float scale = 1.0f;
+            if constexpr (GROUPED) {
+                const uint4 q = group_tiles[tile % mt];
+                live = quad * 32 + lane < q.z;
+                if (live) { const GroupRow gr = group_row(p, q.y + quad * 32 + lane); row = gr.out; scale = gr.scale; }
+            }
 #pragma unroll 1
             for (uint32_t c0 = 0; c0 < n_cols; c0 += 32) {
                 uint32_t r[32];
                 tc::tmem_ld32(tmem + b * NT + ((quad * 32u) << 16) + c0, r);
                 tc::tmem_wait_ld();
-                if (row < p.m) {
+                if (live) {
                 float v[32];
 #pragma unroll
                 for (int j = 0; j < 32; ++j) v[j] = __uint_as_float(r[j]);
-                const size_t o = static_cast<size_t>(row) * p.ldy + n0 + c0;
+                if constexpr (GROUPED) {
+#pragma unroll
+                    for (int j = 0; j < 32; ++j) v[j] *= scale;
+                }
+                if (p.bias) {
+#pragma unroll
+                    for (int j = 0; j < 32; ++j)
+                        if (c0 + j < n_cols) v[j] += p.bias[n0 + c0 + j];
+                }
+                if (epi_pairs(p.epi)) {                                  // 32 columns -> 16 outputs
+                    Y* y = static_cast<Y*>(p.y) + row * p.ldy + (n0 + c0) / 2;
+                    float g[16];
+#pragma unroll
+                    for (int j = 0; j < 16; ++j) g[j] = glu_value(v[2 * j], v[2 * j + 1], p.epi, p.cap);
+                    if (wide && c0 + 32 <= n_cols) {
+                        store16(y, g);
+                    } else {
+#pragma unroll
+                        for (int j = 0; j < 16; ++j)
+                            if (c0 + 2 * j < n_cols) y[j] = from_f32<Y>(g[j]);
+                    }
+                } else {
+                const size_t o = row * p.ldy + n0 + c0;
                 Y* y = static_cast<Y*>(p.y) + o;
-                if (p.epi == HF2Q_EPI_GELU || p.epi == HF2Q_EPI_SOFTCAP) {
+                if (p.epi == HF2Q_EPI_GELU || p.epi == HF2Q_EPI_SOFTCAP || p.epi == HF2Q_EPI_SCALE) {
 #pragma unroll
                     for (int j = 0; j < 32; ++j) v[j] = epilogue_value(v[j], p.epi, p.cap);
                 }
@@ -375,19 +435,8 @@ __global__ void __launch_bounds__(TC_THREADS, 1) dense_gemm_tc_kernel(const __gr
                             v[j] += q.x; v[j + 1] += q.y; v[j + 2] += q.z; v[j + 3] += q.w;
                         }
                     }
-                    if constexpr (sizeof(Y) == 4) {
-#pragma unroll
-                        for (int j = 0; j < 32; j += 8) st_global_v8(reinterpret_cast<float*>(y) + j, v + j);
-                    } else {
-                        uint32_t q[16];
-#pragma unroll
-                        for (int j = 0; j < 16; ++j) {
-                            const __nv_bfloat162 h = __floats2bfloat162_rn(v[2 * j], v[2 * j + 1]);
-                            q[j] = *reinterpret_cast<const uint32_t*>(&h);
-                        }
-#pragma unroll
-                        for (int j = 0; j < 4; ++j) reinterpret_cast<uint4*>(y)[j] = make_uint4(q[4 * j], q[4 * j + 1], q[4 * j + 2], q[4 * j + 3]);
-                    }
+                    store16(y, v);
+                    store16(y + 16, v + 16);
                 } else {
 #pragma unroll
                     for (int j = 0; j < 32; ++j)
@@ -396,6 +445,7 @@ __global__ void __launch_bounds__(TC_THREADS, 1) dense_gemm_tc_kernel(const __gr
                             if (p.epi == HF2Q_EPI_ADD) q += p.residual[o + j];
                             y[j] = from_f32<Y>(q);
                         }
+                }
                 }
                 }
                 __syncwarp();
@@ -436,34 +486,39 @@ bool encode_rows(CUtensorMap* map, const void* base, uint32_t rows, uint32_t k, 
               CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
-template <int NT, typename Y>
-cudaError_t launch_tc(const DenseArgs& a, int sms, uint32_t* status, cudaStream_t st) {
+template <int NT, typename Y, bool GROUPED>
+cudaError_t launch_tc(const DenseArgs& a, uint32_t m_tiles, int sms, uint32_t* status, cudaStream_t st) {
     CUtensorMap mx, mw;
-    if (!encode_rows(&mx, a.x, a.m, a.k, a.ldx, TC_M) || !encode_rows(&mw, a.w, a.n, a.k, a.k, NT)) return cudaErrorInvalidValue;
+    const uint32_t w_rows = GROUPED ? a.n * a.g.groups : a.n;
+    if (!encode_rows(&mx, a.x, a.m, a.k, a.ldx, TC_M) || !encode_rows(&mw, a.w, w_rows, a.k, a.k, NT)) return cudaErrorInvalidValue;
     const size_t smem = 1024 + static_cast<size_t>(tc_stages(NT)) * tc_stage_bytes(NT);
     static PerDeviceFlag flag;
-    if (const cudaError_t e = ensure_max_dynamic_smem(dense_gemm_tc_kernel<NT, Y>, static_cast<int>(smem), flag); e != cudaSuccess) return e;
-    const uint32_t tiles = ((a.m + TC_M - 1) / TC_M) * ((a.n + NT - 1) / NT);
+    if (const cudaError_t e = ensure_max_dynamic_smem(dense_gemm_tc_kernel<NT, Y, GROUPED>, static_cast<int>(smem), flag); e != cudaSuccess) return e;
+    const uint32_t tiles = m_tiles * ((a.n + NT - 1) / NT);
     const uint32_t grid = tiles < static_cast<uint32_t>(sms) ? tiles : static_cast<uint32_t>(sms);
-    return launch_pdl(dense_gemm_tc_kernel<NT, Y>, dim3(grid), dim3(TC_THREADS), smem, st, mx, mw, a, status);
+    return launch_pdl(dense_gemm_tc_kernel<NT, Y, GROUPED>, dim3(grid), dim3(TC_THREADS), smem, st, mx, mw, a, status);
 }
-template <typename Y>
-cudaError_t launch_tc_any(const DenseArgs& a, int sms, uint32_t* status, cudaStream_t st) {
-    const uint32_t mt = (a.m + TC_M - 1) / TC_M;
+// m_tiles: activation tiles, for a grouped product the most there can be
+template <typename Y, bool GROUPED>
+cudaError_t launch_tc_any(const DenseArgs& a, uint32_t m_tiles, int sms, uint32_t* status, cudaStream_t st) {
     // the widest tile that still gives (nearly) every SM work
-    if (mt * ((a.n + 255) / 256) >= static_cast<uint32_t>(sms) * 3 / 4) return launch_tc<256, Y>(a, sms, status, st);
-    if (mt * ((a.n + 127) / 128) >= static_cast<uint32_t>(sms) * 3 / 4) return launch_tc<128, Y>(a, sms, status, st);
-    return launch_tc<64, Y>(a, sms, status, st);
+    if (m_tiles * ((a.n + 255) / 256) >= static_cast<uint32_t>(sms) * 3 / 4) return launch_tc<256, Y, GROUPED>(a, m_tiles, sms, status, st);
+    if (m_tiles * ((a.n + 127) / 128) >= static_cast<uint32_t>(sms) * 3 / 4) return launch_tc<128, Y, GROUPED>(a, m_tiles, sms, status, st);
+    return launch_tc<64, Y, GROUPED>(a, m_tiles, sms, status, st);
 }
 
 constexpr uint32_t MV_SMEM = 200 * 1024;
 
+template <typename X, typename Y, int M, int RW>
+cudaError_t launch_mv_rw(const DenseArgs& a, cudaStream_t st) {
+    static PerDeviceFlag flag;
+    if (const cudaError_t e = ensure_max_dynamic_smem(dense_matvec_m_kernel<X, Y, M, RW>, MV_SMEM, flag); e != cudaSuccess) return e;
+    return launch_pdl(dense_matvec_m_kernel<X, Y, M, RW>, dim3((a.n / RW + MV_WARPS - 1) / MV_WARPS), dim3(MV_THREADS),
+                      static_cast<size_t>(M) * a.k * 4, st, a);
+}
 template <typename X, typename Y, int M>
 cudaError_t launch_mv_m(const DenseArgs& a, cudaStream_t st) {
-    static PerDeviceFlag flag;
-    if (const cudaError_t e = ensure_max_dynamic_smem(dense_matvec_m_kernel<X, Y, M>, MV_SMEM, flag); e != cudaSuccess) return e;
-    return launch_pdl(dense_matvec_m_kernel<X, Y, M>, dim3((a.n + MV_WARPS - 1) / MV_WARPS), dim3(MV_THREADS),
-                      static_cast<size_t>(M) * a.k * 4, st, a);
+    return epi_pairs(a.epi) ? launch_mv_rw<X, Y, M, 2>(a, st) : launch_mv_rw<X, Y, M, 1>(a, st);
 }
 template <typename X, typename Y>
 cudaError_t launch_mv(DenseArgs a, cudaStream_t st, uint64_t* launches) {
@@ -500,12 +555,11 @@ cudaError_t dense_any(const DenseArgs& a, int sms, uint32_t* status, cudaStream_
     if (a.m <= 8 && a.k * 4 <= MV_SMEM) return launch_mv<X, Y>(a, st, launches);
     *launches = 1;
     if constexpr (sizeof(X) == 2) {
-        if (a.ldx % 8 == 0 && reinterpret_cast<uintptr_t>(a.x) % 16 == 0) return launch_tc_any<Y>(a, sms, status, st);
+        if (a.ldx % 8 == 0 && reinterpret_cast<uintptr_t>(a.x) % 16 == 0) return launch_tc_any<Y, false>(a, (a.m + TC_M - 1) / TC_M, sms, status, st);
     }
-    return launch_pdl(dense_gemm_f32_kernel<X, Y>, dim3((a.n + FT - 1) / FT, (a.m + FT - 1) / FT), dim3(256), 0, st, a);
+    return launch_pdl(dense_gemm_f32_kernel<X, Y, false>, dim3((a.n + FT - 1) / FT, (a.m + FT - 1) / FT), dim3(256), 0, st, a);
 }
 
-constexpr uint32_t MR_MAX_SMEM = 208 * 1024;
 template <int PRO>
 cudaError_t launch_fused(const MatvecSegs& p, uint32_t blocks, size_t smem, uint32_t* status, cudaStream_t st) {
     static PerDeviceFlag flag;
@@ -522,15 +576,15 @@ extern "C" {
 
 HF2Q_API int32_t hf2q_cuda_dense_matmul(hf2q_ctx* ctx, void* stream, const void* x, uint32_t x_dtype, uint32_t ldx, const void* w, void* y,
                                         uint32_t y_dtype, uint32_t ldy, uint32_t m, uint32_t n, uint32_t k, uint32_t epilogue,
-                                        const float* residual, float cap) {
+                                        const float* residual, float cap, const float* bias) {
     if (!ctx) return HF2Q_ERR_INVALID_ARGUMENT;
-    if (!x || !w || !y || n == 0 || k == 0 || k % 8 || ldx < k || ldy < n || reinterpret_cast<uintptr_t>(w) % 16)
+    if (!x || !w || !y || n == 0 || k == 0 || k % 8 || ldx < k || ldy < (epi_pairs(epilogue) ? n / 2 : n) || reinterpret_cast<uintptr_t>(w) % 16)
         return ctx_fail(ctx, HF2Q_ERR_INVALID_ARGUMENT, "dense_matmul: null pointer, k not a multiple of 8, a short row pitch or an unaligned weight");
-    if (epilogue > HF2Q_EPI_SOFTCAP || (epilogue == HF2Q_EPI_ADD && !residual) || (epilogue == HF2Q_EPI_SOFTCAP && !(cap > 0.f)))
+    if (epilogue > HF2Q_EPI_CLAMP_GLU || (epilogue == HF2Q_EPI_ADD && !residual) || (epi_needs_cap(epilogue) && !(cap > 0.f)) || (epi_pairs(epilogue) && n % 2))
         return ctx_fail(ctx, HF2Q_ERR_INVALID_ARGUMENT, "dense_matmul: bad epilogue");
     if (m == 0) return HF2Q_OK;
     if (m > 65535u * 64u) return ctx_fail(ctx, HF2Q_ERR_INVALID_ARGUMENT, "dense_matmul: too many rows");
-    const DenseArgs a{x, static_cast<const __nv_bfloat16*>(w), y, residual, ldx, ldy, m, n, k, epilogue, cap};
+    const DenseArgs a{x, static_cast<const __nv_bfloat16*>(w), y, residual, bias, ldx, ldy, m, n, k, epilogue, cap, {}};
     const cudaStream_t st = static_cast<cudaStream_t>(stream);
     uint32_t* status = ctx_status_word(ctx);
     const int sms = ctx_sm_count(ctx);
@@ -543,9 +597,30 @@ HF2Q_API int32_t hf2q_cuda_dense_matmul(hf2q_ctx* ctx, void* stream, const void*
     return ctx_cuda_result(ctx, e, "dense_matmul", launches);
 }
 
+HF2Q_API int32_t hf2q_cuda_dense_grouped(hf2q_ctx* ctx, void* stream, const hf2q_row_groups* g, const void* x, uint32_t dtype, uint32_t ldx, const void* w,
+                                         void* y, uint32_t y_dtype, uint32_t ldy, uint32_t rows, uint32_t n, uint32_t k, uint32_t epilogue, float cap) {
+    if (!ctx) return HF2Q_ERR_INVALID_ARGUMENT;
+    if (!g || !g->header || !g->tiles || !g->perm || g->groups == 0 || !x || !w || !y || n == 0 || k == 0 || k % 8 || ldx < k || ldx % 8 ||
+        ldy < (epi_pairs(epilogue) ? n / 2 : n) || reinterpret_cast<uintptr_t>(w) % 16 || reinterpret_cast<uintptr_t>(x) % 16 || epilogue > HF2Q_EPI_CLAMP_GLU ||
+        epilogue == HF2Q_EPI_ADD || (epi_needs_cap(epilogue) && !(cap > 0.f)) || (epi_pairs(epilogue) && n % 2) || static_cast<uint64_t>(g->groups) * n > 0x7fffffffu)
+        return ctx_fail(ctx, HF2Q_ERR_INVALID_ARGUMENT, "dense_grouped: null or unaligned pointer, or a bad size or epilogue");
+    if (rows == 0) return HF2Q_OK;
+    if (g->tile_rows != (dtype == HF2Q_DT_BF16 ? HF2Q_GROUP_TILE_BF16 : HF2Q_GROUP_TILE_F32))
+        return ctx_fail(ctx, HF2Q_ERR_INVALID_ARGUMENT, "dense_grouped: the rows were sorted for another tile height");
+    DenseArgs a{x, static_cast<const __nv_bfloat16*>(w), y, nullptr, nullptr, ldx, ldy, rows, n, k, epilogue, cap, *g};
+    const cudaStream_t st = static_cast<cudaStream_t>(stream);
+    const uint32_t most = rows / g->tile_rows + (rows < g->groups ? rows : g->groups);     // sum of ceil(count / tile_rows)
+    cudaError_t e = cudaErrorInvalidValue;
+    if (dtype == HF2Q_DT_BF16 && y_dtype == HF2Q_DT_BF16) e = launch_tc_any<__nv_bfloat16, true>(a, most, ctx_sm_count(ctx), ctx_status_word(ctx), st);
+    else if (dtype == HF2Q_DT_BF16 && y_dtype == HF2Q_DT_F32) e = launch_tc_any<float, true>(a, most, ctx_sm_count(ctx), ctx_status_word(ctx), st);
+    else if (dtype == HF2Q_DT_F32 && y_dtype == HF2Q_DT_F32 && most <= 65535)
+        e = launch_pdl(dense_gemm_f32_kernel<float, float, true>, dim3((n + FT - 1) / FT, most), dim3(256), 0, st, a);
+    return ctx_cuda_result(ctx, e, "dense_grouped", 1);
+}
+
 HF2Q_API int32_t hf2q_cuda_dense_matvec(hf2q_ctx* ctx, void* stream, uint32_t prologue, const hf2q_matvec* segs, uint32_t n_segs) {
     if (!ctx) return HF2Q_ERR_INVALID_ARGUMENT;
-    if (!segs || n_segs == 0 || n_segs > 2 || prologue > HF2Q_PRO_GATED) return ctx_fail(ctx, HF2Q_ERR_INVALID_ARGUMENT, "dense_matvec: bad segments");
+    if (!segs || n_segs == 0 || n_segs > 2 || prologue > HF2Q_PRO_HYPER) return ctx_fail(ctx, HF2Q_ERR_INVALID_ARGUMENT, "dense_matvec: bad segments");
     MatvecSegs p{};
     uint32_t kmax = 0;
     uint64_t chunks[2] = {0, 0};
@@ -554,8 +629,9 @@ HF2Q_API int32_t hf2q_cuda_dense_matvec(hf2q_ctx* ctx, void* stream, uint32_t pr
         if (!s.w || !s.y || s.n == 0 || s.k == 0 || s.k % 8 || reinterpret_cast<uintptr_t>(s.w) % 16 || MR_RING + s.k * 4ull > MR_MAX_SMEM ||
             (prologue == HF2Q_PRO_NONE && !s.x) ||
             (prologue == HF2Q_PRO_NORM && (!s.pre.x || !s.pre.norm || s.pre.width > s.k || !pre_norm_aligned(s.pre) || (s.pre.a && (!s.pre.b || !s.pre.a_norm || !s.pre.b_norm)) || (s.pre.shift && (!s.pre.shift_state || !s.pre.pos)))) ||
-            (prologue == HF2Q_PRO_GATED && (!s.gated.o || !s.gated.gate || s.gated.heads * s.gated.head_dim > s.k)) ||
-            (s.epilogue == HF2Q_EPI_ADD && !s.residual))
+            (prologue == HF2Q_PRO_GATED && (!gated_ok(s.gated) || s.gated.heads * s.gated.head_dim > s.k)) ||
+            (prologue == HF2Q_PRO_HYPER && (!hyper_ok(s.hyper) || s.hyper.width > s.k || s.hyper.x_out == s.hyper.x)) || s.epilogue > HF2Q_EPI_CLAMP_GLU ||
+            (s.epilogue == HF2Q_EPI_ADD && !s.residual) || (epi_needs_cap(s.epilogue) && !(s.cap > 0.f)) || (epi_pairs(s.epilogue) && s.n % 2))
             return ctx_fail(ctx, HF2Q_ERR_INVALID_ARGUMENT, "dense_matvec: bad segment");
         p.s[i] = s;
         chunks[i] = static_cast<uint64_t>(s.n) * ((s.k + MV_CHUNK - 1) / MV_CHUNK);
@@ -573,6 +649,7 @@ HF2Q_API int32_t hf2q_cuda_dense_matvec(hf2q_ctx* ctx, void* stream, uint32_t pr
     switch (prologue) {
         case HF2Q_PRO_NONE: e = launch_fused<HF2Q_PRO_NONE>(p, blocks, smem, status, st); break;
         case HF2Q_PRO_NORM: e = launch_fused<HF2Q_PRO_NORM>(p, blocks, smem, status, st); break;
+        case HF2Q_PRO_HYPER: e = launch_fused<HF2Q_PRO_HYPER>(p, blocks, smem, status, st); break;
         default: e = launch_fused<HF2Q_PRO_GATED>(p, blocks, smem, status, st); break;
     }
     return ctx_cuda_result(ctx, e, "dense_matvec", 1);

@@ -185,17 +185,22 @@ MoeScratch moe_scratch_layout(uint32_t n_experts, uint32_t rows, uint32_t k) {
     return s;
 }
 
+cudaError_t launch_moe_sort(const uint32_t* ids, uint32_t rows, uint32_t n_experts, uint32_t nt, uint32_t* header, void* tiles, uint32_t* perm,
+                            float* y, float* y2, uint32_t n, uint32_t* status, cudaStream_t st) {
+    const size_t smem = (4 * static_cast<size_t>(n_experts) + 2 + 68) * 4;
+    if (smem > 48 * 1024) return cudaErrorInvalidValue;
+    moe_sort_kernel<<<1, SORT_THREADS, smem, st>>>(ids, rows, n_experts, nt, header, static_cast<uint4*>(tiles), perm, y, y2, n, status);
+    return cudaGetLastError();
+}
+
 cudaError_t launch_moe_prep(const uint32_t* ids, uint32_t rows, uint32_t n_experts, uint32_t top_k, uint32_t nt, const void* x,
                             uint32_t x_dtype, uint32_t k, float* y, float* y2, uint32_t n, void* scratch, const MoeScratch& lay,
                             uint32_t* status, int sm_count, cudaStream_t st) {
     uint8_t* base = static_cast<uint8_t*>(scratch);
     uint32_t* header = reinterpret_cast<uint32_t*>(base);
-    uint4* tiles = reinterpret_cast<uint4*>(base + lay.tiles_off);
     uint32_t* perm = reinterpret_cast<uint32_t*>(base + lay.perm_off);
     __half* xg = reinterpret_cast<__half*>(base + lay.xg_off);
-    const size_t smem = (4 * static_cast<size_t>(n_experts) + 2 + 68) * 4;
-    moe_sort_kernel<<<1, SORT_THREADS, smem, st>>>(ids, rows, n_experts, nt, header, tiles, perm, y, y2, n, status);
-    cudaError_t e = cudaGetLastError();
+    const cudaError_t e = launch_moe_sort(ids, rows, n_experts, nt, header, base + lay.tiles_off, perm, y, y2, n, status, st);
     if (e != cudaSuccess) return e;
     const unsigned grid = rows < static_cast<uint32_t>(sm_count) * 8 ? rows : static_cast<uint32_t>(sm_count) * 8;
     moe_gather_kernel<<<grid, 256, 0, st>>>(x, x_dtype == HF2Q_DT_BF16, top_k, k, header, perm, xg, status);

@@ -159,6 +159,13 @@ cudaError_t gemm_tc_static_scratch(int device, void** out);
 cudaError_t launch_softmax_topk(const float* logits, uint32_t* ids, float* weights,
                                 uint32_t n_tokens, uint32_t n_experts, uint32_t top_k,
                                 cudaStream_t st);
+// sigmoid -> top-k, scores as weights; logits rows are ld floats apart
+cudaError_t launch_sigmoid_topk(const float* logits, uint32_t ld, uint32_t* ids, float* weights, uint32_t n_tokens,
+                                uint32_t n_experts, uint32_t top_k, cudaStream_t st);
+// counting sort of routed rows by expert (the first stage of launch_moe_prep): tiles of nt rows, header, perm; rows of an id
+// out of range are left out of the order and their outputs y / y2 [rows][n] zeroed (NULL: none)
+cudaError_t launch_moe_sort(const uint32_t* ids, uint32_t rows, uint32_t n_experts, uint32_t nt, uint32_t* header, void* tiles, uint32_t* perm,
+                            float* y, float* y2, uint32_t n, uint32_t* status, cudaStream_t st);
 
 
 // ---- the glue of a full decoder forward (decoder_ops.cu) ----

@@ -4,6 +4,7 @@
 // dispatch_moe_softmax_topk (gpu_ffn.rs:2551): descending probability, equal probabilities keep
 // the lower expert index first (the reference sorts stably), weights = p / sum(selected p), with
 // the same 1e-20 guards.  One warp per token; probabilities live in shared memory.
+// Sigmoid scores without renormalisation take the same selection.
 #include <math_constants.h>
 
 #include "common.cuh"
@@ -14,7 +15,8 @@ namespace hf2q {
 namespace {
 constexpr int WARPS = 4;
 
-__global__ void __launch_bounds__(WARPS * 32) softmax_topk_kernel(const float* __restrict__ logits,
+template <bool SIGMOID>
+__global__ void __launch_bounds__(WARPS * 32) topk_kernel(const float* __restrict__ logits, uint32_t ld,
                                                                   uint32_t* __restrict__ ids,
                                                                   float* __restrict__ weights,
                                                                   uint32_t n_tokens, uint32_t n_experts,
@@ -24,20 +26,24 @@ __global__ void __launch_bounds__(WARPS * 32) softmax_topk_kernel(const float* _
     const uint32_t t = blockIdx.x * WARPS + warp;
     if (t >= n_tokens) return;
     float* probs = probs_all + static_cast<size_t>(warp) * n_experts;
-    const float* row = logits + static_cast<size_t>(t) * n_experts;
+    const float* row = logits + static_cast<size_t>(t) * ld;
 
-    float mx = -CUDART_INF_F;
-    for (uint32_t e = lane; e < n_experts; e += 32) mx = fmaxf(mx, row[e]);
-    for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-    float denom = 0.f;
-    for (uint32_t e = lane; e < n_experts; e += 32) {
-        const float v = expf(row[e] - mx);
-        probs[e] = v;
-        denom += v;
+    if constexpr (SIGMOID) {
+        for (uint32_t e = lane; e < n_experts; e += 32) probs[e] = 1.0f / (1.0f + expf(-row[e]));
+    } else {
+        float mx = -CUDART_INF_F;
+        for (uint32_t e = lane; e < n_experts; e += 32) mx = fmaxf(mx, row[e]);
+        for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+        float denom = 0.f;
+        for (uint32_t e = lane; e < n_experts; e += 32) {
+            const float v = expf(row[e] - mx);
+            probs[e] = v;
+            denom += v;
+        }
+        for (int o = 16; o > 0; o >>= 1) denom += __shfl_xor_sync(0xffffffffu, denom, o);
+        const float inv_d = denom > 1e-20f ? 1.0f / denom : 1.0f;
+        for (uint32_t e = lane; e < n_experts; e += 32) probs[e] *= inv_d;
     }
-    for (int o = 16; o > 0; o >>= 1) denom += __shfl_xor_sync(0xffffffffu, denom, o);
-    const float inv_d = denom > 1e-20f ? 1.0f / denom : 1.0f;
-    for (uint32_t e = lane; e < n_experts; e += 32) probs[e] *= inv_d;
     __syncwarp();
 
     // Selection is total: a NaN probability (a NaN logit, or a row whose logits are all -inf) ranks
@@ -81,6 +87,7 @@ __global__ void __launch_bounds__(WARPS * 32) softmax_topk_kernel(const float* _
             }
         }
     }
+    if constexpr (SIGMOID) return;
     __syncwarp();
     const float inv_sum = sum_sel > 1e-20f ? 1.0f / sum_sel : 1.0f / static_cast<float>(top_k);
     for (uint32_t s = lane; s < top_k; s += 32) weights[static_cast<size_t>(t) * top_k + s] *= inv_sum;
@@ -92,7 +99,16 @@ cudaError_t launch_softmax_topk(const float* logits, uint32_t* ids, float* weigh
     const size_t smem = static_cast<size_t>(WARPS) * n_experts * sizeof(float);
     if (smem > 48 * 1024) return cudaErrorInvalidValue;
     const unsigned grid = (n_tokens + WARPS - 1) / WARPS;
-    softmax_topk_kernel<<<grid, WARPS * 32, smem, st>>>(logits, ids, weights, n_tokens, n_experts, top_k);
+    topk_kernel<false><<<grid, WARPS * 32, smem, st>>>(logits, n_experts, ids, weights, n_tokens, n_experts, top_k);
+    return cudaGetLastError();
+}
+
+cudaError_t launch_sigmoid_topk(const float* logits, uint32_t ld, uint32_t* ids, float* weights, uint32_t n_tokens,
+                                uint32_t n_experts, uint32_t top_k, cudaStream_t st) {
+    const size_t smem = static_cast<size_t>(WARPS) * n_experts * sizeof(float);
+    if (smem > 48 * 1024) return cudaErrorInvalidValue;
+    const unsigned grid = (n_tokens + WARPS - 1) / WARPS;
+    topk_kernel<true><<<grid, WARPS * 32, smem, st>>>(logits, ld, ids, weights, n_tokens, n_experts, top_k);
     return cudaGetLastError();
 }
 

@@ -2,8 +2,9 @@
 //
 //   mlstm   exponential input / forget gates with a running maximum (matrix memory of xLSTM)
 //   delta   gated delta rule, one decay per head and key channel
+//   ssd     scalar decay per head and token (Mamba-2)
 //
-// Both keep S[key channel][value column] and treat a value column independently, so the state lives in registers:
+// All keep S[key channel][value column] and treat a value column independently, so the state lives in registers:
 // sixteen lanes share a column (each holds key channels 32 c + 2 l and + 1), a warp carries two columns, a CTA of eight
 // warps sixteen columns of one head: the token chain is latency-bound, so many short warps beat few long ones.  A token costs no block barrier; sums over the key channels are four shuffles.
 // Tokens are staged in shared memory in batches by asynchronous copies, two batches in flight.  The state in memory
@@ -447,6 +448,182 @@ __global__ void __launch_bounds__(256) delta_decay_kernel(const float* __restric
     }
 }
 
+// ---------------------------------------------------------------- state space with a scalar decay
+__device__ __forceinline__ uint32_t ssd_channels(const hf2q_ssd& a) { return a.heads * a.vdim + 2 * a.groups * a.state; }
+
+// S <- keep S + dt B x^T;  y = S^T C + d x
+template <int RQ>
+__global__ void __launch_bounds__(SC_THREADS) ssd_scan_kernel(const __grid_constant__ hf2q_ssd a, uint32_t m, const float* __restrict__ xbc,
+                                                              const float* __restrict__ dt, const float* __restrict__ la, float* __restrict__ y) {
+    constexpr uint32_t DP = 32 * RQ;
+    extern __shared__ __align__(16) float dsm[];                    // B, C: [2][SC_TB][DP] each
+    float* ks = dsm;
+    float* qs = dsm + 2 * SC_TB * DP;
+    __shared__ __align__(16) float vs[2][SC_TB][SC_COLS];
+    __shared__ float gk[2][SC_TB], gw[2][SC_TB];                    // decay, step size
+    pdl_trigger();
+    pdl_wait();
+    const uint32_t h = blockIdx.x, slice = blockIdx.y, grp = h / (a.heads / a.groups);
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, lg = lane & 15;
+    const uint32_t col_s = warp * 2 + (lane >> 4), col0 = slice * SC_COLS, col = col0 + col_s;
+    const uint32_t n_cols = min(static_cast<uint32_t>(SC_COLS), a.vdim - col0);
+    const bool live = col < a.vdim;
+    const uint32_t channels = ssd_channels(a), inner = a.heads * a.vdim;
+    // the convolution's reader has finished: the last inputs go to the state
+    for (uint32_t i = (blockIdx.y * gridDim.x + blockIdx.x) * SC_THREADS + threadIdx.x; i < channels; i += gridDim.x * gridDim.y * SC_THREADS) {
+        const uint32_t pos = *a.pos, keep = min(a.taps - 1, m);
+        for (uint32_t j = 0; j < keep; ++j)
+            a.conv_state[static_cast<size_t>(i) * a.taps + (pos + m - 1 - j) % a.taps] = a.proj[static_cast<size_t>(m - 1 - j) * a.ld + a.off + i];
+    }
+    for (uint32_t i = threadIdx.x; i < 4 * SC_TB * DP; i += SC_THREADS) dsm[i] = 0.f;
+    for (uint32_t i = threadIdx.x; i < 2 * SC_TB * SC_COLS; i += SC_THREADS) (&vs[0][0][0])[i] = 0.f;
+    __syncthreads();
+    auto stage = [&](uint32_t t0, uint32_t b) {
+        const uint32_t n = min(static_cast<uint32_t>(SC_TB), m - t0);
+        const float* row = xbc + static_cast<size_t>(t0) * channels;
+        stage_rows(ks + b * SC_TB * DP, DP, row + inner + grp * a.state, channels, n, a.state);
+        stage_rows(qs + b * SC_TB * DP, DP, row + inner + (a.groups + grp) * a.state, channels, n, a.state);
+        stage_rows(vs[b][0], SC_COLS, row + h * a.vdim + col0, channels, n, n_cols);
+        if (threadIdx.x < n) {
+            const size_t o = static_cast<size_t>(t0 + threadIdx.x) * a.heads + h;
+            gk[b][threadIdx.x] = expf(la[o]);
+            gw[b][threadIdx.x] = dt[o];
+        }
+        cp_async_commit();
+    };
+    Vec<RQ> S;
+    float* sp = a.s + (static_cast<size_t>(h) * a.vdim + (live ? col : 0)) * DP + 2 * lg;
+    const float skip = a.d[h];
+    if (live) S.load(sp); else S.zero();
+    stage(0, 0);
+    for (uint32_t t0 = 0, b = 0; t0 < m; t0 += SC_TB, b ^= 1) {
+        if (t0 + SC_TB < m) { stage(t0 + SC_TB, b ^ 1); cp_async_wait<1>(); }
+        else cp_async_wait<0>();
+        __syncthreads();
+        const uint32_t n = min(static_cast<uint32_t>(SC_TB), m - t0);
+        struct Operands { Vec<RQ> k, q; float keep, write, v; };
+        auto fetch = [&](uint32_t j) {
+            Operands t;
+            t.k.load(ks + (b * SC_TB + j) * DP + 2 * lg);
+            t.q.load(qs + (b * SC_TB + j) * DP + 2 * lg);
+            t.keep = gk[b][j];
+            t.write = gw[b][j];
+            t.v = vs[b][j][col_s];
+            return t;
+        };
+        auto finish = [&](uint32_t j, float s) {
+            if (live) y[static_cast<size_t>(t0 + j) * inner + static_cast<size_t>(h) * a.vdim + col] = s + skip * vs[b][j][col_s];
+        };
+        uint32_t j0 = 0;
+        for (; j0 + 16 <= n; j0 += 16) {                     // sixteen tokens without a branch; lane i of a group finishes token i
+            float r[16];
+            Operands t = fetch(j0);
+#pragma unroll
+            for (uint32_t u = 0; u < 16; ++u) {
+                const Operands next = fetch(j0 + (u < 15 ? u + 1 : 15));
+                S.decay_axpy(t.keep, t.k, t.write * t.v);
+                r[u] = S.dot(t.q);
+                t = next;
+            }
+            finish(j0 + lg, group_transpose_sum(r, lg));
+        }
+        for (; j0 < n; ++j0) {
+            const Operands t = fetch(j0);
+            S.decay_axpy(t.keep, t.k, t.write * t.v);
+            const float r = group_sum(S.dot(t.q));
+            if (lg == 0) finish(j0, r);
+        }
+        __syncthreads();
+    }
+    if (live) S.store(sp);
+}
+
+__device__ __forceinline__ void ssd_gates(const hf2q_ssd& a, uint32_t h, float raw, float& dt, float& la) {
+    dt = softplusf(raw + a.dt_bias[h]);
+    la = -expf(a.a_log[h]) * dt;
+}
+template <typename Before>
+__device__ __forceinline__ float conv_bias_silu(const float* w, float bias, uint32_t taps, float now, Before before) {
+    float s = fmaf(now, w[taps - 1], bias);
+    for (uint32_t j = 1; j < taps; ++j) s = fmaf(before(j), w[taps - 1 - j], s);
+    return siluf(s);
+}
+
+// One CTA per token.
+__global__ void __launch_bounds__(256) ssd_prep_kernel(const __grid_constant__ hf2q_ssd a, float* __restrict__ xbc, float* __restrict__ dt, float* __restrict__ la) {
+    pdl_trigger();
+    pdl_wait();
+    const uint32_t t = blockIdx.x, pos = *a.pos, channels = ssd_channels(a);
+    const float* row = a.proj + static_cast<size_t>(t) * a.ld + a.off;
+    float* dst = xbc + static_cast<size_t>(t) * channels;
+    for (uint32_t c = threadIdx.x; c < channels; c += 256)
+        dst[c] = conv_bias_silu(a.conv + static_cast<size_t>(c) * a.taps, a.conv_bias[c], a.taps, row[c], [&](uint32_t j) {
+            return j <= t ? row[static_cast<ptrdiff_t>(c) - static_cast<ptrdiff_t>(j) * a.ld] : a.conv_state[static_cast<size_t>(c) * a.taps + (pos + t + a.taps - j) % a.taps];
+        });
+    for (uint32_t h = threadIdx.x; h < a.heads; h += 256) {
+        const size_t o = static_cast<size_t>(t) * a.heads + h;
+        ssd_gates(a, h, row[channels + h], dt[o], la[o]);
+    }
+}
+
+// One token from the raw projection row: convolution, SiLU, step size and the state update.
+template <int RQ>
+__global__ void __launch_bounds__(SC_THREADS) ssd_step_kernel(const __grid_constant__ hf2q_ssd a, float* __restrict__ y) {
+    constexpr uint32_t DP = 32 * RQ;
+    __shared__ __align__(16) float ks[DP], qs[DP], vs[SC_COLS];
+    pdl_trigger();
+    const uint32_t h = blockIdx.x, slice = blockIdx.y, rep = a.heads / a.groups, grp = h / rep;
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, lg = lane & 15;
+    const uint32_t col_s = warp * 2 + (lane >> 4), col0 = slice * SC_COLS, col = col0 + col_s;
+    const uint32_t n_cols = min(static_cast<uint32_t>(SC_COLS), a.vdim - col0);
+    const bool live = col < a.vdim;
+    pdl_wait();
+    Vec<RQ> S;
+    float* sp = a.s + (static_cast<size_t>(h) * a.vdim + (live ? col : 0)) * DP + 2 * lg;
+    if (live) S.load(sp); else S.zero();
+    const uint32_t pos = *a.pos, channels = ssd_channels(a), inner = a.heads * a.vdim;
+    const float* row = a.proj + a.off;
+    // the state ring has one column more than the taps look back, so this token's column is read by nobody
+    auto channel = [&](uint32_t c, bool keep) {
+        float* st = a.conv_state + static_cast<size_t>(c) * a.taps;
+        const float now = row[c];
+        const float v = conv_bias_silu(a.conv + static_cast<size_t>(c) * a.taps, a.conv_bias[c], a.taps, now, [&](uint32_t j) { return st[(pos + a.taps - j) % a.taps]; });
+        if (keep) st[pos % a.taps] = now;
+        return v;
+    };
+    const bool first = slice == 0 && h % rep == 0;
+    for (uint32_t i = threadIdx.x; i < 2 * DP; i += SC_THREADS) {
+        const uint32_t j = i % DP;
+        const float v = j < a.state ? channel(inner + (i < DP ? grp : a.groups + grp) * a.state + j, first) : 0.f;
+        (i < DP ? ks : qs)[j] = v;
+    }
+    if (threadIdx.x < SC_COLS) vs[threadIdx.x] = threadIdx.x < n_cols ? channel(h * a.vdim + col0 + threadIdx.x, true) : 0.f;
+    float dt, la;
+    ssd_gates(a, h, row[channels + h], dt, la);
+    __syncthreads();
+    Vec<RQ> k, q;
+    k.load(ks + 2 * lg);
+    q.load(qs + 2 * lg);
+    S.decay_axpy(expf(la), k, dt * vs[col_s]);
+    const float r = group_sum(S.dot(q));
+    if (live) {
+        S.store(sp);
+        if (lg == 0) y[h * a.vdim + col] = r + a.d[h] * vs[col_s];
+    }
+}
+
+bool ssd_ok(const hf2q_ssd* a) {
+    return a && a->proj && a->conv && a->conv_bias && a->dt_bias && a->a_log && a->d && a->conv_state && a->s && a->pos && a->heads && a->groups &&
+           a->heads % a->groups == 0 && a->state && a->state <= 256 && a->vdim && a->taps;
+}
+template <int RQ>
+cudaError_t launch_ssd_scan(const hf2q_ssd& a, uint32_t m, const float* xbc, const float* dt, const float* la, float* y, cudaStream_t st) {
+    static PerDeviceFlag flag;
+    const size_t smem = 4ull * SC_TB * 32 * RQ * sizeof(float);
+    if (const cudaError_t e = ensure_max_dynamic_smem(ssd_scan_kernel<RQ>, static_cast<int>(smem), flag); e != cudaSuccess) return e;
+    return launch_pdl(ssd_scan_kernel<RQ>, dim3(a.heads, (a.vdim + SC_COLS - 1) / SC_COLS), dim3(SC_THREADS), smem, st, a, m, xbc, dt, la, y);
+}
+
 bool delta_ok(const hf2q_delta* a) {
     return a && a->proj && a->q_conv && a->k_conv && a->v_conv && a->a_log && a->dt_bias && a->a2 && a->g2 && a->conv_state && a->s && a->pos &&
            a->heads && a->kv_heads && a->heads % a->kv_heads == 0 && a->dim && a->dim <= 256 && a->vdim && a->taps && a->a_rank_ld % 8 == 0 &&
@@ -549,6 +726,41 @@ HF2Q_API int32_t hf2q_cuda_delta_scan(hf2q_ctx* ctx, void* stream, const hf2q_de
         default: break;
     }
     return ctx_cuda_result(ctx, e, "delta_scan", 1);
+}
+
+HF2Q_API int32_t hf2q_cuda_ssd_step(hf2q_ctx* ctx, void* stream, const hf2q_ssd* a, float* y) {
+    if (!ctx) return HF2Q_ERR_INVALID_ARGUMENT;
+    if (!ssd_ok(a) || !y) return ctx_fail(ctx, HF2Q_ERR_INVALID_ARGUMENT, "ssd_step: null pointer or an unsupported size");
+    const dim3 grid(a->heads, (a->vdim + SC_COLS - 1) / SC_COLS);
+    cudaError_t e = cudaErrorInvalidValue;
+    switch ((a->state + 31) / 32) {
+#define F(RQ) case RQ: e = launch_pdl(ssd_step_kernel<RQ>, grid, dim3(SC_THREADS), 0, static_cast<cudaStream_t>(stream), *a, y); break;
+        HF2Q_RQ_CASES(F)
+#undef F
+        default: break;
+    }
+    return ctx_cuda_result(ctx, e, "ssd_step", 1);
+}
+
+HF2Q_API int32_t hf2q_cuda_ssd_prep(hf2q_ctx* ctx, void* stream, const hf2q_ssd* a, uint32_t m, float* xbc, float* dt, float* la) {
+    if (!ctx) return HF2Q_ERR_INVALID_ARGUMENT;
+    if (!ssd_ok(a) || !xbc || !dt || !la) return ctx_fail(ctx, HF2Q_ERR_INVALID_ARGUMENT, "ssd_prep: null pointer or an unsupported size");
+    if (m == 0) return HF2Q_OK;
+    return ctx_cuda_result(ctx, launch_pdl(ssd_prep_kernel, dim3(m), dim3(256), 0, static_cast<cudaStream_t>(stream), *a, xbc, dt, la), "ssd_prep", 1);
+}
+
+HF2Q_API int32_t hf2q_cuda_ssd_scan(hf2q_ctx* ctx, void* stream, const hf2q_ssd* a, uint32_t m, const float* xbc, const float* dt, const float* la, float* y) {
+    if (!ctx) return HF2Q_ERR_INVALID_ARGUMENT;
+    if (!ssd_ok(a) || !xbc || !dt || !la || !y) return ctx_fail(ctx, HF2Q_ERR_INVALID_ARGUMENT, "ssd_scan: null pointer or an unsupported size");
+    if (m == 0) return HF2Q_OK;
+    cudaError_t e = cudaErrorInvalidValue;
+    switch ((a->state + 31) / 32) {
+#define F(RQ) case RQ: e = launch_ssd_scan<RQ>(*a, m, xbc, dt, la, y, static_cast<cudaStream_t>(stream)); break;
+        HF2Q_RQ_CASES(F)
+#undef F
+        default: break;
+    }
+    return ctx_cuda_result(ctx, e, "ssd_scan", 1);
 }
 
 }  // extern "C"

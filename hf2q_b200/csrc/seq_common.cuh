@@ -35,6 +35,15 @@ __device__ __forceinline__ float gelu_tanhf(float x) {
     return 0.5f * x * (1.0f + tanhf(0.7978845608028654f * (x + 0.044715f * x * x * x)));
 }
 
+// ---- product epilogues that take rows in pairs (gate, up)
+__host__ __device__ constexpr bool epi_pairs(uint32_t epi) { return epi == HF2Q_EPI_SWIGLU || epi == HF2Q_EPI_CLAMP_GLU; }
+__host__ __device__ constexpr bool epi_needs_cap(uint32_t epi) { return epi == HF2Q_EPI_SOFTCAP || epi == HF2Q_EPI_CLAMP_GLU; }
+__device__ __forceinline__ float glu_value(float gate, float up, uint32_t epi, float cap) {
+    if (epi == HF2Q_EPI_SWIGLU) return siluf(gate) * up;
+    const float g = fminf(gate, cap), u = fminf(fmaxf(up, -cap), cap);
+    return g * sigmoidf(1.702f * g) * (u + 1.0f);
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
@@ -192,6 +201,133 @@ __device__ __forceinline__ void gated_heads_row(const hf2q_gated_heads& g, uint3
             out[c0 + i] = from_f32<OUT>(v * sigmoidf(gate[c0 + i]));
         }
     }
+}
+
+// One row of a gated, group-normed output: v = o * silu(gate), every one of `heads` equal groups of `head_dim` elements
+// divided by its own root mean square, times norm [heads * head_dim].  buf: f32 row in shared memory; out may be buf.
+// The whole block takes part; ends without a barrier.
+constexpr uint32_t GROUP_MAX = 512;
+template <typename OUT>
+__device__ __forceinline__ void silu_group_norm_row(const hf2q_gated_heads& g, uint32_t t, float* buf, OUT* out) {
+    __shared__ float sums[GROUP_MAX];
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
+    const uint32_t sub = max(1u, n_warps / g.heads), units = g.heads * sub;     // warps that share a group
+    const float* o = g.o + static_cast<size_t>(t) * g.ldo;
+    const float* gate = g.gate + static_cast<size_t>(t) * g.ldg;
+    const bool quads = g.head_dim % 4 == 0 && ((reinterpret_cast<uintptr_t>(o) | reinterpret_cast<uintptr_t>(gate)) & 15) == 0;
+    for (uint32_t u = warp; u < units; u += n_warps) {
+        const uint32_t c0 = u / sub * g.head_dim, part = u % sub;
+        float s = 0.f;
+        if (quads) {
+            for (uint32_t i = 4 * (lane + 32 * part); i < g.head_dim; i += 128 * sub) {
+                const float4 a = *reinterpret_cast<const float4*>(o + c0 + i), b = *reinterpret_cast<const float4*>(gate + c0 + i);
+                const float4 v = make_float4(a.x * siluf(b.x), a.y * siluf(b.y), a.z * siluf(b.z), a.w * siluf(b.w));
+                *reinterpret_cast<float4*>(buf + c0 + i) = v;
+                s += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+            }
+        } else {
+            for (uint32_t i = lane + 32 * part; i < g.head_dim; i += 32 * sub) {
+                const float v = o[c0 + i] * siluf(gate[c0 + i]);
+                buf[c0 + i] = v;
+                s += v * v;
+            }
+        }
+        s = warp_sum(s);
+        if (lane == 0) sums[u] = s;
+    }
+    __syncthreads();
+    for (uint32_t u = warp; u < units; u += n_warps) {
+        const uint32_t c0 = u / sub * g.head_dim, part = u % sub;
+        float s = 0.f;
+        for (uint32_t k = 0; k < sub; ++k) s += sums[u / sub * sub + k];
+        const float inv = 1.0f / sqrtf(s / static_cast<float>(g.head_dim) + g.eps);
+        for (uint32_t i = lane + 32 * part; i < g.head_dim; i += 32 * sub) out[c0 + i] = from_f32<OUT>(buf[c0 + i] * inv * g.norm[c0 + i]);
+    }
+}
+inline bool gated_ok(const hf2q_gated_heads& g) {
+    return g.o && g.gate && g.heads && g.head_dim && g.kind <= HF2Q_GATE_SILU_FIRST && (g.kind == HF2Q_GATE_SIGMOID_LAST || (g.norm && g.heads <= GROUP_MAX));
+}
+
+// ---- several residual streams
+constexpr uint32_t HYPER_MAX = 16, HYPER_COEF = HYPER_MAX * HYPER_MAX + 2 * HYPER_MAX;
+
+inline bool hyper_ok(const hf2q_hyper& p) {
+    if (!p.x || !p.streams || p.streams > HYPER_MAX || (p.x_streams != 1 && p.x_streams != p.streams) || !p.width || (p.y && (!p.mix || !p.out || !p.y_parts)) ||
+        (p.x_out == p.x && p.x_streams != p.streams))
+        return false;
+    if (p.width % 4) return true;
+    const void* all[] = {p.x, p.x_out, p.y};
+    for (const void* q : all)
+        if (reinterpret_cast<uintptr_t>(q) % 16) return false;
+    return true;
+}
+
+// V: float or float4 (width a multiple of four)
+__device__ __forceinline__ void axpy(float& d, float a, float x) { d = fmaf(a, x, d); }
+__device__ __forceinline__ void axpy(float4& d, float a, const float4& x) { d.x = fmaf(a, x.x, d.x); d.y = fmaf(a, x.y, d.y); d.z = fmaf(a, x.z, d.z); d.w = fmaf(a, x.w, d.w); }
+__device__ __forceinline__ float square_sum(float v) { return v * v; }
+__device__ __forceinline__ float square_sum(const float4& v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
+
+template <int S, typename V>
+__device__ __forceinline__ float hyper_elements(const hf2q_hyper& p, uint32_t t, float* xs, const float* coef, uint32_t lo, uint32_t hi) {
+    constexpr uint32_t E = sizeof(V) / 4;
+    const uint32_t n = p.width / E;
+    const V* x = reinterpret_cast<const V*>(p.x + static_cast<size_t>(t) * p.x_streams * p.width);
+    V* xo = reinterpret_cast<V*>(p.x_out + static_cast<size_t>(t) * p.streams * p.width);
+    const V* y = reinterpret_cast<const V*>(p.y + static_cast<size_t>(t) * p.y_parts * p.width);
+    const float *mix = coef, *out = coef + S * S, *in = out + S;
+    float ss = 0.f;
+    for (uint32_t i = threadIdx.x; i < n; i += blockDim.x) {
+        V old[S], yv{}, u{};
+#pragma unroll
+        for (int s = 0; s < S; ++s) old[s] = s < static_cast<int>(p.streams) ? x[(p.x_streams == 1 ? 0u : s * n) + i] : V{};
+        if (p.y)
+            for (uint32_t k = 0; k < p.y_parts; ++k) axpy(yv, 1.0f, y[k * n + i]);
+        const bool own = p.x_out && E * i >= lo && E * i < hi;
+#pragma unroll
+        for (int d = 0; d < S; ++d) {
+            if (d >= static_cast<int>(p.streams)) continue;
+            V v = old[d];
+            if (p.y) {
+                v = V{};
+#pragma unroll
+                for (int s = 0; s < S; ++s) axpy(v, mix[s * S + d], old[s]);
+                axpy(v, out[d], yv);
+            }
+            if (own) xo[d * n + i] = v;
+            axpy(u, in[d], v);
+        }
+        reinterpret_cast<V*>(xs)[i] = u;
+        ss += square_sum(u);
+    }
+    return ss;
+}
+template <int S>
+__device__ __forceinline__ float hyper_row_s(const hf2q_hyper& p, uint32_t t, float* xs, float* coef, uint32_t lo, uint32_t hi) {
+    // [S][S] mix, [S] out, [S] in; absent streams have zeros
+    for (uint32_t i = threadIdx.x; i < S * S + 2 * S; i += blockDim.x) {
+        const uint32_t a = i / S, b = i % S;
+        float v = 0.f;
+        if (b < p.streams) {
+            if (a < S) v = p.y && a < p.streams ? p.mix[a * p.streams + b] : 0.f;
+            else if (a == S) v = p.y ? p.out[b] : 0.f;
+            else v = p.in ? p.in[b] : 1.0f;
+        }
+        coef[i] = v;
+    }
+    __syncthreads();
+    return p.width % 4 == 0 ? hyper_elements<S, float4>(p, t, xs, coef, lo, hi) : hyper_elements<S, float>(p, t, xs, coef, lo, hi);
+}
+// Row t of the streams (hf2q_hyper): the pending update, stored for elements [lo, hi), and the row that the sublayer reads
+// into xs[0..width) (shared memory, 16-byte aligned).  Returns the reciprocal root mean square of it.
+__device__ __forceinline__ float hyper_row(const hf2q_hyper& p, uint32_t t, float* xs, float* coef, float* red, uint32_t lo, uint32_t hi) {
+    float s[1];
+    if (p.streams <= 2) s[0] = hyper_row_s<2>(p, t, xs, coef, lo, hi);
+    else if (p.streams <= 4) s[0] = hyper_row_s<4>(p, t, xs, coef, lo, hi);
+    else if (p.streams <= 8) s[0] = hyper_row_s<8>(p, t, xs, coef, lo, hi);
+    else s[0] = hyper_row_s<16>(p, t, xs, coef, lo, hi);
+    block_sum(s, red);
+    return 1.0f / sqrtf(s[0] / static_cast<float>(p.width) + p.eps);
 }
 
 }  // namespace seq

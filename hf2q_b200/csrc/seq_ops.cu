@@ -1,5 +1,5 @@
 // Row-wise steps around the products of a bf16-weight decoder: embedding rows with the hashed bigram table, the
-// residual update + RMS norm + token shift in front of a product, gated head outputs, and the hand-over of the
+// residual update + RMS norm + token shift in front of a product, the same for a residual in several streams, gated head outputs, and the hand-over of the
 // shift / convolution state after a portion of several tokens.
 #include "seq_common.cuh"
 
@@ -101,13 +101,48 @@ __global__ void __launch_bounds__(512) pre_norm_kernel(const __grid_constant__ h
 }
 
 template <typename OUT>
+__global__ void __launch_bounds__(512) hyper_norm_kernel(const __grid_constant__ hf2q_hyper p, OUT* __restrict__ out, uint32_t ldo) {
+    extern __shared__ __align__(16) float xs[];
+    __shared__ float coef[HYPER_COEF];
+    __shared__ float red[32];
+    pdl_trigger();
+    pdl_wait();
+    const uint32_t t = blockIdx.x;
+    const float inv = hyper_row(p, t, xs, coef, red, 0, p.width);
+    OUT* row = out + static_cast<size_t>(t) * ldo;
+    if (p.width % 4 == 0 && ldo % 4 == 0 && ((reinterpret_cast<uintptr_t>(p.norm) | reinterpret_cast<uintptr_t>(out)) & 15) == 0) {
+        for (uint32_t i = threadIdx.x; i < ldo / 4; i += blockDim.x) {
+            float4 h = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (4 * i < p.width) {
+                h = reinterpret_cast<const float4*>(xs)[i];
+                if (p.norm) {
+                    const float4 w = reinterpret_cast<const float4*>(p.norm)[i];
+                    h = make_float4(h.x * inv * w.x, h.y * inv * w.y, h.z * inv * w.z, h.w * inv * w.w);
+                }
+            }
+            if constexpr (sizeof(OUT) == 4) {
+                reinterpret_cast<float4*>(row)[i] = h;
+            } else {
+                const __nv_bfloat162 a = __floats2bfloat162_rn(h.x, h.y), b = __floats2bfloat162_rn(h.z, h.w);
+                reinterpret_cast<uint2*>(row)[i] = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+            }
+        }
+        return;
+    }
+    for (uint32_t i = threadIdx.x; i < ldo; i += blockDim.x)
+        row[i] = from_f32<OUT>(i < p.width ? (p.norm ? xs[i] * inv * p.norm[i] : xs[i]) : 0.f);
+}
+
+template <typename OUT>
 __global__ void __launch_bounds__(256) gated_heads_kernel(const __grid_constant__ hf2q_gated_heads g, OUT* __restrict__ out, uint32_t ldo) {
     pdl_trigger();
     pdl_wait();
     const uint32_t t = blockIdx.x;
     OUT* row = out + static_cast<size_t>(t) * ldo;
     for (uint32_t i = g.heads * g.head_dim + threadIdx.x; i < ldo; i += blockDim.x) row[i] = from_f32<OUT>(0.f);
-    gated_heads_row<OUT>(g, t, row, threadIdx.x >> 5, blockDim.x >> 5);
+    extern __shared__ __align__(16) float buf[];
+    if (g.kind == HF2Q_GATE_SILU_FIRST) silu_group_norm_row<OUT>(g, t, buf, row);
+    else gated_heads_row<OUT>(g, t, row, threadIdx.x >> 5, blockDim.x >> 5);
 }
 
 __global__ void __launch_bounds__(256) state_tail_kernel(const uint32_t* __restrict__ pos_dev, uint32_t m, const float* __restrict__ h_last,
@@ -176,13 +211,41 @@ HF2Q_API int32_t hf2q_cuda_pre_norm(hf2q_ctx* ctx, void* stream, const hf2q_pre_
 
 HF2Q_API int32_t hf2q_cuda_gated_heads(hf2q_ctx* ctx, void* stream, const hf2q_gated_heads* g, uint32_t m, void* out, uint32_t out_dtype, uint32_t ldo) {
     if (!ctx) return HF2Q_ERR_INVALID_ARGUMENT;
-    if (!g || !g->o || !g->gate || !out || ldo < g->heads * g->head_dim) return ctx_fail(ctx, HF2Q_ERR_INVALID_ARGUMENT, "gated_heads: null pointer or a short row");
+    if (!g || !gated_ok(*g) || !out || ldo < g->heads * g->head_dim) return ctx_fail(ctx, HF2Q_ERR_INVALID_ARGUMENT, "gated_heads: null pointer or a short row");
     if (m == 0) return HF2Q_OK;
     const cudaStream_t st = static_cast<cudaStream_t>(stream);
+    const size_t smem = g->kind == HF2Q_GATE_SILU_FIRST ? static_cast<size_t>(g->heads) * g->head_dim * 4 : 0;
+    if (smem > 200 * 1024) return ctx_fail(ctx, HF2Q_ERR_INVALID_ARGUMENT, "gated_heads: row too long");
+    static PerDeviceFlag f32f, bff;
     cudaError_t e = cudaErrorInvalidValue;
-    if (out_dtype == HF2Q_DT_F32) e = launch_pdl(gated_heads_kernel<float>, dim3(m), dim3(256), 0, st, *g, static_cast<float*>(out), ldo);
-    else if (out_dtype == HF2Q_DT_BF16) e = launch_pdl(gated_heads_kernel<__nv_bfloat16>, dim3(m), dim3(256), 0, st, *g, static_cast<__nv_bfloat16*>(out), ldo);
+    if (out_dtype == HF2Q_DT_F32) {
+        e = ensure_max_dynamic_smem(gated_heads_kernel<float>, 200 * 1024, f32f);
+        if (e == cudaSuccess) e = launch_pdl(gated_heads_kernel<float>, dim3(m), dim3(256), smem, st, *g, static_cast<float*>(out), ldo);
+    } else if (out_dtype == HF2Q_DT_BF16) {
+        e = ensure_max_dynamic_smem(gated_heads_kernel<__nv_bfloat16>, 200 * 1024, bff);
+        if (e == cudaSuccess) e = launch_pdl(gated_heads_kernel<__nv_bfloat16>, dim3(m), dim3(256), smem, st, *g, static_cast<__nv_bfloat16*>(out), ldo);
+    }
     return ctx_cuda_result(ctx, e, "gated_heads", 1);
+}
+
+HF2Q_API int32_t hf2q_cuda_hyper_norm(hf2q_ctx* ctx, void* stream, const hf2q_hyper* p, uint32_t m, void* out, uint32_t out_dtype, uint32_t ldo) {
+    if (!ctx) return HF2Q_ERR_INVALID_ARGUMENT;
+    if (!p || !hyper_ok(*p) || !out || ldo < p->width) return ctx_fail(ctx, HF2Q_ERR_INVALID_ARGUMENT, "hyper_norm: null or unaligned pointer, a bad number of streams or a short row");
+    if (m == 0) return HF2Q_OK;
+    const size_t smem = static_cast<size_t>(p->width) * 4;
+    if (smem > 200 * 1024) return ctx_fail(ctx, HF2Q_ERR_INVALID_ARGUMENT, "hyper_norm: width too large");
+    const cudaStream_t st = static_cast<cudaStream_t>(stream);
+    const dim3 block(p->width >= 2048 ? 512 : 256);
+    static PerDeviceFlag f32f, bff;
+    cudaError_t e = cudaErrorInvalidValue;
+    if (out_dtype == HF2Q_DT_F32) {
+        e = ensure_max_dynamic_smem(hyper_norm_kernel<float>, 200 * 1024, f32f);
+        if (e == cudaSuccess) e = launch_pdl(hyper_norm_kernel<float>, dim3(m), block, smem, st, *p, static_cast<float*>(out), ldo);
+    } else if (out_dtype == HF2Q_DT_BF16) {
+        e = ensure_max_dynamic_smem(hyper_norm_kernel<__nv_bfloat16>, 200 * 1024, bff);
+        if (e == cudaSuccess) e = launch_pdl(hyper_norm_kernel<__nv_bfloat16>, dim3(m), block, smem, st, *p, static_cast<__nv_bfloat16*>(out), ldo);
+    }
+    return ctx_cuda_result(ctx, e, "hyper_norm", 1);
 }
 
 HF2Q_API int32_t hf2q_cuda_state_tail(hf2q_ctx* ctx, void* stream, const uint32_t* pos, uint32_t m, const float* h_last, float* shift_state,

@@ -1,5 +1,6 @@
 // Sliding-window attention over a ring cache (position p in slot p % capacity) with grouped query heads, optional
-// per-head RMS norm of q and k and an optional logarithmic distance term taken off the scores.
+// per-head RMS norm of q and k and an optional logarithmic distance term taken off the scores.  The prefill also runs over
+// plain rows of keys and values, with a part of every key shared by the heads (expanded latents).
 //
 //   append    prefill: normalised queries to a buffer, normalised keys and values to the cache
 //   prefill   bf16 cache: tiles of 64 queries x 64 keys on the tensor cores (f32 scores, softmax and accumulators, bf16
@@ -21,6 +22,33 @@ __device__ __forceinline__ float score_of(float dot, float scale, float r1, floa
     if (bias) s -= r1 * logf(1.0f + r2 * static_cast<float>(dist));
     return s;
 }
+
+// where a KV head's keys and values are: rings, or plain rows that start at position `first`
+template <typename T>
+struct KeyRows {
+    const T *k, *v, *shared;
+    uint32_t k_row, v_row, first, capacity, s_row, s_capacity, dp, sp;      // sp: padded size of the shared part
+    bool linear;
+    __device__ __forceinline__ KeyRows(const hf2q_window_attn& a, uint32_t kvh, uint32_t pos0) {
+        const uint32_t dvp = pad8(a.vdim);
+        dp = pad8(a.dim);
+        sp = pad8(a.shared_dim);
+        linear = a.linear;
+        capacity = a.capacity;
+        k_row = linear ? a.row_stride : dp;
+        v_row = linear ? a.row_stride : dvp;
+        first = linear && pos0 + 1 > a.window ? pos0 + 1 - a.window : 0u;
+        k = static_cast<const T*>(a.k_cache) + (linear ? static_cast<size_t>(kvh) * a.k_head_stride : static_cast<size_t>(kvh) * a.capacity * dp);
+        v = static_cast<const T*>(a.v_cache) + (linear ? static_cast<size_t>(kvh) * a.v_head_stride : static_cast<size_t>(kvh) * a.capacity * dvp);
+        shared = static_cast<const T*>(a.k_shared);
+        s_row = a.shared_stride;
+        s_capacity = a.shared_capacity;
+    }
+    __device__ __forceinline__ uint32_t slot(uint32_t p) const { return linear ? p - first : p % capacity; }
+    __device__ __forceinline__ const T* key(uint32_t p) const { return k + static_cast<size_t>(slot(p)) * k_row; }
+    __device__ __forceinline__ const T* value(uint32_t p) const { return v + static_cast<size_t>(slot(p)) * v_row; }
+    __device__ __forceinline__ const T* shared_key(uint32_t p) const { return shared + static_cast<size_t>(p % s_capacity) * s_row; }
+};
 
 // one head vector of up to 256 elements held by a warp (element lane + 32 j), divided by its root mean square
 struct HeadVec {
@@ -86,26 +114,29 @@ struct WarpAttn {
             for (int c = 0; c < NC; ++c) acc[g][c][0] = acc[g][c][1] = 0.f;
         }
     }
-    __device__ __forceinline__ void keys(const hf2q_window_attn& a, const T* kc, const T* vc, const float* qs, float* ps, const float (&r1)[GR],
+    __device__ __forceinline__ void keys(const hf2q_window_attn& a, const KeyRows<T>& kv, const float* qs, float* ps, const float (&r1)[GR],
                                          const float (&r2)[GR], uint32_t pos, uint32_t p0, uint32_t hi) {
-        const uint32_t lane = threadIdx.x & 31, dp = pad8(a.dim), dvp = pad8(a.vdim);
+        const uint32_t lane = threadIdx.x & 31, dq = kv.dp + kv.sp, dvp = pad8(a.vdim);
         const uint32_t p = p0 + lane;
         const bool live = p < hi;
         float s[GR];
 #pragma unroll
         for (int g = 0; g < GR; ++g) s[g] = 0.f;
         if (live) {
-            const T* kr = kc + static_cast<size_t>(p % a.capacity) * dp;
+            auto part = [&](const T* kr, uint32_t n, const float* q0) {
 #pragma unroll 4
-            for (uint32_t c = 0; c < dp; c += 8) {
-                float k[8];
-                load8(kr + c, k);
+                for (uint32_t c = 0; c < n; c += 8) {
+                    float k[8];
+                    load8(kr + c, k);
 #pragma unroll
-                for (int g = 0; g < GR; ++g) {
-                    const float4 x = *reinterpret_cast<const float4*>(qs + g * dp + c), y = *reinterpret_cast<const float4*>(qs + g * dp + c + 4);
-                    s[g] += k[0] * x.x + k[1] * x.y + k[2] * x.z + k[3] * x.w + k[4] * y.x + k[5] * y.y + k[6] * y.z + k[7] * y.w;
+                    for (int g = 0; g < GR; ++g) {
+                        const float4 x = *reinterpret_cast<const float4*>(q0 + g * dq + c), y = *reinterpret_cast<const float4*>(q0 + g * dq + c + 4);
+                        s[g] += k[0] * x.x + k[1] * x.y + k[2] * x.z + k[3] * x.w + k[4] * y.x + k[5] * y.y + k[6] * y.z + k[7] * y.w;
+                    }
                 }
-            }
+            };
+            part(kv.key(p), kv.dp, qs);
+            if (kv.sp) part(kv.shared_key(p), kv.sp, qs + kv.dp);
         }
 #pragma unroll
         for (int g = 0; g < GR; ++g) {
@@ -124,7 +155,7 @@ struct WarpAttn {
         const uint32_t cnt = min(32u, hi - p0);
 #pragma unroll 4
         for (uint32_t i = 0; i < cnt; ++i) {
-            const T* vr = vc + static_cast<size_t>((p0 + i) % a.capacity) * dvp;
+            const T* vr = kv.value(p0 + i);
 #pragma unroll
             for (int c = 0; c < NC; ++c) {
                 const uint32_t d = 2 * lane + 64 * c;
@@ -197,9 +228,10 @@ __global__ void __launch_bounds__(WD_WARPS * 32) window_decode_kernel(const __gr
         r2[g] = a.r1 ? a.r2[h0 + min(static_cast<uint32_t>(g), n_g - 1)] : 0.f;
     }
     __syncthreads();
+    const KeyRows<T> kv(a, kvh, pos);
     WarpAttn<T, GR, NC> w;
     w.init();
-    for (uint32_t p0 = lo + warp * 32; p0 < hi; p0 += WD_WARPS * 32) w.keys(a, kc, vc, qs, ps + warp * GR * 32, r1, r2, pos, p0, hi);
+    for (uint32_t p0 = lo + warp * 32; p0 < hi; p0 += WD_WARPS * 32) w.keys(a, kv, qs, ps + warp * GR * 32, r1, r2, pos, p0, hi);
 #pragma unroll
     for (int g = 0; g < GR; ++g) {
         if (lane == 0) { rm[warp * GR + g] = w.mx[g]; rl[warp * GR + g] = w.l[g]; }
@@ -253,26 +285,27 @@ __global__ void __launch_bounds__(WD_WARPS * 32) window_decode_kernel(const __gr
     }
 }
 
+constexpr uint32_t QK_MAX = 320;                        // dim and shared_dim together, padded
+
 // ---------------------------------------------------------------- prefill, f32: one warp per (query, head)
 template <typename T, typename OUT, int NC>
 __global__ void __launch_bounds__(256) window_prefill_f32_kernel(const __grid_constant__ hf2q_window_attn a, uint32_t m, const T* __restrict__ q,
                                                                  const float* __restrict__ gate, uint32_t ldg, OUT* __restrict__ out, uint32_t ldo) {
-    __shared__ __align__(16) float qs[8][256];
+    __shared__ __align__(16) float qs[8][QK_MAX];
     __shared__ float ps[8][32];
     pdl_trigger();
     pdl_wait();
     const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, h = blockIdx.y, t = blockIdx.x * 8 + warp;
     if (t >= m) return;
-    const uint32_t dp = pad8(a.dim), dvp = pad8(a.vdim), kvh = h / (a.heads / a.kv_heads);
-    for (uint32_t i = lane; i < dp; i += 32) qs[warp][i] = to_f32(q[(static_cast<size_t>(t) * a.heads + h) * dp + i]);
+    const KeyRows<T> kv(a, h / (a.heads / a.kv_heads), *a.pos);
+    const uint32_t dq = kv.dp + kv.sp;
+    for (uint32_t i = lane; i < dq; i += 32) qs[warp][i] = to_f32(q[(static_cast<size_t>(t) * a.heads + h) * dq + i]);
     __syncwarp();
     const uint32_t pos = *a.pos + t, n = min(pos + 1, a.window), hi = pos + 1;
-    const T* kc = static_cast<const T*>(a.k_cache) + static_cast<size_t>(kvh) * a.capacity * dp;
-    const T* vc = static_cast<const T*>(a.v_cache) + static_cast<size_t>(kvh) * a.capacity * dvp;
     const float r1[1] = {a.r1 ? a.r1[h] : 0.f}, r2[1] = {a.r1 ? a.r2[h] : 0.f};
     WarpAttn<T, 1, NC> w;
     w.init();
-    for (uint32_t p0 = hi - n; p0 < hi; p0 += 32) w.keys(a, kc, vc, qs[warp], ps[warp], r1, r2, pos, p0, hi);
+    for (uint32_t p0 = hi - n; p0 < hi; p0 += 32) w.keys(a, kv, qs[warp], ps[warp], r1, r2, pos, p0, hi);
 #pragma unroll
     for (int c = 0; c < NC; ++c)
 #pragma unroll
@@ -307,57 +340,58 @@ __device__ __forceinline__ uint32_t pack_bf16(float a, float b) {
     return *reinterpret_cast<const uint32_t*>(&h);
 }
 
-// grid (query tiles, heads); DM >= dim, vdim.  Keys are walked from the first one the tile's first query sees.
-template <int DM, typename OUT>
+// grid (query tiles, heads); DK >= dim + shared_dim, DV >= vdim.  Keys are walked from the first one the tile's first
+// query sees.
+template <int DK, int DV, typename OUT>
 __global__ void __launch_bounds__(WP_WARPS * 32) window_prefill_mma_kernel(const __grid_constant__ hf2q_window_attn a, uint32_t m,
                                                                            const __nv_bfloat16* __restrict__ q, const float* __restrict__ gate, uint32_t ldg,
                                                                            OUT* __restrict__ out, uint32_t ldo) {
-    constexpr uint32_t PITCH = DM + 8, TILE = WP_K * PITCH;         // elements
+    constexpr uint32_t KP = DK + 8, VP = DV + 8, K_TILE = WP_K * KP, TILES = K_TILE + WP_K * VP;      // pitches and sizes in elements
     extern __shared__ __align__(16) __nv_bfloat16 kv[];             // [2][K tile, V tile]
     pdl_trigger();
     pdl_wait();
     const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, t4 = lane & 3;
-    const uint32_t h = blockIdx.y, t0 = blockIdx.x * WP_Q, kvh = h / (a.heads / a.kv_heads);
-    const uint32_t dp = pad8(a.dim), dvp = pad8(a.vdim), nk = (dp + 15) / 16, nv = (dvp + 15) / 16;
-    const uint32_t pos0 = *a.pos, q_lo = pos0 + t0, q_hi = pos0 + min(t0 + WP_Q, m) - 1;
+    const uint32_t h = blockIdx.y, t0 = blockIdx.x * WP_Q;
+    const uint32_t pos0 = *a.pos;
+    const KeyRows<__nv_bfloat16> rows(a, h / (a.heads / a.kv_heads), pos0);
+    const uint32_t dq = rows.dp + rows.sp, dvp = pad8(a.vdim), nk = (dq + 15) / 16, nv = (dvp + 15) / 16;
+    const uint32_t q_lo = pos0 + t0, q_hi = pos0 + min(t0 + WP_Q, m) - 1;
     const uint32_t j0 = q_lo + 1 > a.window ? q_lo + 1 - a.window : 0u;
-    const __nv_bfloat16* kc = static_cast<const __nv_bfloat16*>(a.k_cache) + static_cast<size_t>(kvh) * a.capacity * dp;
-    const __nv_bfloat16* vc = static_cast<const __nv_bfloat16*>(a.v_cache) + static_cast<size_t>(kvh) * a.capacity * dvp;
     // elements past dim / vdim, and keys never loaded, must be finite zeros
-    for (uint32_t i = threadIdx.x; i < 4 * TILE / 8; i += WP_WARPS * 32) reinterpret_cast<uint4*>(kv)[i] = make_uint4(0, 0, 0, 0);
+    for (uint32_t i = threadIdx.x; i < 2 * TILES / 8; i += WP_WARPS * 32) reinterpret_cast<uint4*>(kv)[i] = make_uint4(0, 0, 0, 0);
     __syncthreads();
     auto stage = [&](uint32_t key0, uint32_t b) {
-        __nv_bfloat16* ks = kv + b * 2 * TILE;
-        __nv_bfloat16* vs = ks + TILE;
-        const uint32_t ck = dp / 8, cv = dvp / 8;
+        __nv_bfloat16* ks = kv + b * TILES;
+        __nv_bfloat16* vs = ks + K_TILE;
+        const uint32_t ck = dq / 8, cv = dvp / 8, cd = rows.dp / 8;
         for (uint32_t i = threadIdx.x; i < WP_K * ck; i += WP_WARPS * 32) {
             const uint32_t r = i / ck, c = i % ck;
-            if (key0 + r <= q_hi) cp_async16(ks + r * PITCH + 8 * c, kc + static_cast<size_t>((key0 + r) % a.capacity) * dp + 8 * c);
+            if (key0 + r <= q_hi) cp_async16(ks + r * KP + 8 * c, c < cd ? rows.key(key0 + r) + 8 * c : rows.shared_key(key0 + r) + 8 * (c - cd));
         }
         for (uint32_t i = threadIdx.x; i < WP_K * cv; i += WP_WARPS * 32) {
             const uint32_t r = i / cv, c = i % cv;
-            if (key0 + r <= q_hi) cp_async16(vs + r * PITCH + 8 * c, vc + static_cast<size_t>((key0 + r) % a.capacity) * dvp + 8 * c);
+            if (key0 + r <= q_hi) cp_async16(vs + r * VP + 8 * c, rows.value(key0 + r) + 8 * c);
         }
         cp_async_commit();
     };
     stage(j0, 0);
-    uint32_t qa[DM / 16][4];
+    uint32_t qa[DK / 16][4];
     uint32_t row[2], qpos[2];
 #pragma unroll
     for (int u = 0; u < 2; ++u) { row[u] = t0 + warp * 16 + gid + 8 * u; qpos[u] = pos0 + row[u]; }
 #pragma unroll
-    for (int k = 0; k < DM / 16; ++k)
+    for (int k = 0; k < DK / 16; ++k)
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
             const uint32_t r = row[i & 1], c = 16 * k + 8 * (i >> 1) + 2 * t4;
-            qa[k][i] = r < m && c < dp ? *reinterpret_cast<const uint32_t*>(q + (static_cast<size_t>(r) * a.heads + h) * dp + c) : 0u;
+            qa[k][i] = r < m && c < dq ? *reinterpret_cast<const uint32_t*>(q + (static_cast<size_t>(r) * a.heads + h) * dq + c) : 0u;
         }
     const bool bias = a.r1 != nullptr;
     const float r1 = bias ? a.r1[h] : 0.f, r2 = bias ? a.r2[h] : 0.f;
     float mx[2] = {-CUDART_INF_F, -CUDART_INF_F}, l[2] = {0.f, 0.f};
-    float o[DM / 8][4];
+    float o[DV / 8][4];
 #pragma unroll
-    for (int i = 0; i < DM / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+    for (int i = 0; i < DV / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
     const uint32_t n_tiles = (q_hi - j0) / WP_K + 1;
     const uint32_t w_lo = pos0 + t0 + warp * 16, w_hi = w_lo + 15;           // this warp's query positions
     for (uint32_t kt = 0; kt < n_tiles; ++kt) {
@@ -367,17 +401,17 @@ __global__ void __launch_bounds__(WP_WARPS * 32) window_prefill_mma_kernel(const
         __syncthreads();
         // keys above this warp's last query or below its first window edge touch none of its rows
         if (key0 <= w_hi && key0 + WP_K - 1 + a.window > w_lo) {
-            const uint32_t ks = smem_u32(kv + b * 2 * TILE), vs = ks + TILE * 2;
+            const uint32_t ks = smem_u32(kv + b * TILES), vs = ks + K_TILE * 2;
             float s[WP_K / 8][4];
 #pragma unroll
             for (int i = 0; i < WP_K / 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
 #pragma unroll
-            for (int k = 0; k < DM / 16; ++k) {
+            for (int k = 0; k < DK / 16; ++k) {
                 if (k < static_cast<int>(nk)) {
 #pragma unroll
                     for (int n2 = 0; n2 < WP_K / 16; ++n2) {
                         uint32_t f[4];
-                        ldmatrix4(f, ks + ((n2 * 16 + (lane >> 4) * 8 + (lane & 7)) * PITCH + 16 * k + ((lane >> 3) & 1) * 8) * 2);
+                        ldmatrix4(f, ks + ((n2 * 16 + (lane >> 4) * 8 + (lane & 7)) * KP + 16 * k + ((lane >> 3) & 1) * 8) * 2);
                         mma_bf16(s[2 * n2], qa[k], f[0], f[1]);
                         mma_bf16(s[2 * n2 + 1], qa[k], f[2], f[3]);
                     }
@@ -407,7 +441,7 @@ __global__ void __launch_bounds__(WP_WARPS * 32) window_prefill_mma_kernel(const
                 l[u] *= corr;
                 mx[u] = top;
 #pragma unroll
-                for (int i = 0; i < DM / 8; ++i) { o[i][2 * u] *= corr; o[i][2 * u + 1] *= corr; }
+                for (int i = 0; i < DV / 8; ++i) { o[i][2 * u] *= corr; o[i][2 * u + 1] *= corr; }
             }
 #pragma unroll
             for (int n = 0; n < WP_K / 8; ++n)
@@ -422,10 +456,10 @@ __global__ void __launch_bounds__(WP_WARPS * 32) window_prefill_mma_kernel(const
 #pragma unroll
                 for (int i = 0; i < 4; ++i) pa[i] = pack_bf16(s[2 * k + (i >> 1)][2 * (i & 1)], s[2 * k + (i >> 1)][2 * (i & 1) + 1]);
 #pragma unroll
-                for (int n2 = 0; n2 < DM / 16; ++n2) {
+                for (int n2 = 0; n2 < DV / 16; ++n2) {
                     if (n2 < static_cast<int>(nv)) {
                         uint32_t f[4];
-                        ldmatrix4_trans(f, vs + ((16 * k + ((lane >> 3) & 1) * 8 + (lane & 7)) * PITCH + 16 * n2 + (lane >> 4) * 8) * 2);
+                        ldmatrix4_trans(f, vs + ((16 * k + ((lane >> 3) & 1) * 8 + (lane & 7)) * VP + 16 * n2 + (lane >> 4) * 8) * 2);
                         mma_bf16(o[2 * n2], pa, f[0], f[1]);
                         mma_bf16(o[2 * n2 + 1], pa, f[2], f[3]);
                     }
@@ -443,7 +477,7 @@ __global__ void __launch_bounds__(WP_WARPS * 32) window_prefill_mma_kernel(const
         OUT* dst = out + static_cast<size_t>(row[u]) * ldo + h * a.vdim;
         const float* gr = gate ? gate + static_cast<size_t>(row[u]) * ldg + h * a.vdim : nullptr;
 #pragma unroll
-        for (int n = 0; n < DM / 8; ++n)
+        for (int n = 0; n < DV / 8; ++n)
 #pragma unroll
             for (int i = 0; i < 2; ++i) {
                 const uint32_t d = 8 * n + 2 * t4 + i;
@@ -463,7 +497,17 @@ bool window_ok(const hf2q_window_attn* a) {
     return a && a->qkv && a->k_cache && a->v_cache && a->pos && a->heads && a->kv_heads && a->heads % a->kv_heads == 0 && a->dim && a->dim <= 256 &&
            a->vdim && a->vdim <= 256 && a->window && a->capacity >= a->window && (a->r1 == nullptr) == (a->r2 == nullptr) &&
            (a->cache_dtype == HF2Q_DT_F32 || a->cache_dtype == HF2Q_DT_BF16) && reinterpret_cast<uintptr_t>(a->k_cache) % 16 == 0 &&
-           reinterpret_cast<uintptr_t>(a->v_cache) % 16 == 0;
+           reinterpret_cast<uintptr_t>(a->v_cache) % 16 == 0 && !a->linear && !a->shared_dim;
+}
+// what the prefill takes beyond that: plain rows, a shared part of the keys
+bool window_rows_ok(const hf2q_window_attn* a) {
+    if (!a || (!a->linear && !a->shared_dim)) return window_ok(a);
+    hf2q_window_attn b = *a;
+    b.qkv = b.qkv ? b.qkv : static_cast<const float*>(a->k_cache);           // the queries come apart
+    b.linear = b.shared_dim = 0;
+    const bool shared = a->shared_dim == 0 || (a->k_shared && a->shared_capacity && a->shared_stride % 8 == 0 && a->shared_stride >= pad8(a->shared_dim) &&
+                                               reinterpret_cast<uintptr_t>(a->k_shared) % 16 == 0 && pad8(a->dim) + pad8(a->shared_dim) <= QK_MAX);
+    return window_ok(&b) && shared && (!a->linear || (a->row_stride % 8 == 0 && a->k_head_stride % 8 == 0 && a->v_head_stride % 8 == 0));
 }
 uint32_t decode_gr(const hf2q_window_attn& a) {
     const uint32_t rep = a.heads / a.kv_heads;
@@ -510,20 +554,22 @@ cudaError_t launch_prefill_f32(const hf2q_window_attn& a, uint32_t m, const void
     if (a.vdim <= 128) return launch_pdl(window_prefill_f32_kernel<T, OUT, 2>, grid, dim3(256), 0, st, a, m, qt, gate, ldg, o, ldo);
     return launch_pdl(window_prefill_f32_kernel<T, OUT, 4>, grid, dim3(256), 0, st, a, m, qt, gate, ldg, o, ldo);
 }
-template <int DM, typename OUT>
+template <int DK, int DV, typename OUT>
 cudaError_t launch_prefill_dm(const hf2q_window_attn& a, uint32_t m, const void* q, const float* gate, uint32_t ldg, void* out, uint32_t ldo, cudaStream_t st) {
     static PerDeviceFlag flag;
-    const size_t smem = 4ull * WP_K * (DM + 8) * 2;
-    if (const cudaError_t e = ensure_max_dynamic_smem(window_prefill_mma_kernel<DM, OUT>, static_cast<int>(smem), flag); e != cudaSuccess) return e;
-    return launch_pdl(window_prefill_mma_kernel<DM, OUT>, dim3((m + WP_Q - 1) / WP_Q, a.heads), dim3(WP_WARPS * 32), smem, st, a, m,
+    const size_t smem = 2ull * WP_K * (DK + 8 + DV + 8) * 2;
+    if (const cudaError_t e = ensure_max_dynamic_smem(window_prefill_mma_kernel<DK, DV, OUT>, static_cast<int>(smem), flag); e != cudaSuccess) return e;
+    return launch_pdl(window_prefill_mma_kernel<DK, DV, OUT>, dim3((m + WP_Q - 1) / WP_Q, a.heads), dim3(WP_WARPS * 32), smem, st, a, m,
                       static_cast<const __nv_bfloat16*>(q), gate, ldg, static_cast<OUT*>(out), ldo);
 }
 template <typename OUT>
 cudaError_t launch_prefill_mma(const hf2q_window_attn& a, uint32_t m, const void* q, const float* gate, uint32_t ldg, void* out, uint32_t ldo, cudaStream_t st) {
-    const uint32_t d = a.dim > a.vdim ? a.dim : a.vdim;
-    if (d <= 64) return launch_prefill_dm<64, OUT>(a, m, q, gate, ldg, out, ldo, st);
-    if (d <= 128) return launch_prefill_dm<128, OUT>(a, m, q, gate, ldg, out, ldo, st);
-    return launch_prefill_dm<256, OUT>(a, m, q, gate, ldg, out, ldo, st);
+    const uint32_t k = pad8(a.dim) + pad8(a.shared_dim), v = a.vdim;
+    if (k <= 64 && v <= 64) return launch_prefill_dm<64, 64, OUT>(a, m, q, gate, ldg, out, ldo, st);
+    if (k <= 128 && v <= 128) return launch_prefill_dm<128, 128, OUT>(a, m, q, gate, ldg, out, ldo, st);
+    if (k <= 192 && v <= 128) return launch_prefill_dm<192, 128, OUT>(a, m, q, gate, ldg, out, ldo, st);
+    if (k <= 256) return launch_prefill_dm<256, 256, OUT>(a, m, q, gate, ldg, out, ldo, st);
+    return launch_prefill_dm<QK_MAX, 256, OUT>(a, m, q, gate, ldg, out, ldo, st);
 }
 
 }  // namespace
@@ -571,7 +617,7 @@ HF2Q_API int32_t hf2q_cuda_window_attn_append(hf2q_ctx* ctx, void* stream, const
 HF2Q_API int32_t hf2q_cuda_window_attn_prefill(hf2q_ctx* ctx, void* stream, const hf2q_window_attn* a, uint32_t m, const void* q, const float* gate,
                                                uint32_t ldg, void* out, uint32_t out_dtype, uint32_t ldo) {
     if (!ctx) return HF2Q_ERR_INVALID_ARGUMENT;
-    if (!window_ok(a) || !q || !out || ldo < a->heads * a->vdim || a->window - 1 + static_cast<uint64_t>(m) > a->capacity)
+    if (!window_rows_ok(a) || !q || !out || ldo < a->heads * a->vdim || a->window - 1 + static_cast<uint64_t>(m) > a->capacity)
         return ctx_fail(ctx, HF2Q_ERR_INVALID_ARGUMENT, "window_attn_prefill: null pointer, an unsupported size or more tokens than the ring holds");
     if (m == 0) return HF2Q_OK;
     const cudaStream_t st = static_cast<cudaStream_t>(stream);

@@ -24,6 +24,7 @@ import numpy as np
 import torch
 
 from . import _lib, ops
+from .state import LayerRun, StatePool, Workspace
 
 
 @dataclass(frozen=True)
@@ -153,6 +154,100 @@ class GreedyDecoder:
                 self.decode_step()
             if collect:
                 out[t:t + 1].copy_(self.tok)
+        return out
+
+
+class SlotDecoder(GreedyDecoder):
+    """A decoder whose sequences live in the slots of a ``StatePool``; steps run one sequence at a time.
+
+    A design supplies ``decode_step``, ``_portion(ids, m)`` (m tokens from position ``*pos``; whatever it returns describes
+    their residual rows) and ``_head_rows(portion, rows)`` (logits of the given rows of it)."""
+
+    def __init__(self, ctx, cfg, dtype, max_seq: int, n_slots: int, prefill_chunk: int):
+        """``max_seq``: most tokens of one sequence.  The design declares its buffers in ``self.pool`` and allocates them."""
+        if dtype not in (torch.bfloat16, torch.float32):
+            raise ops.Hf2qError(_lib.ERR_INVALID_ARGUMENT, f"dtype {dtype} (want bfloat16 or float32)")
+        self.ctx, self.cfg, self.act, self.max_seq, self.n_slots = ctx, cfg, dtype, max_seq, n_slots
+        self.dev = torch.device("cuda", ctx.device)
+        self.chunk = min(prefill_chunk, max_seq)
+        self.pool = StatePool(n_slots, self.dev)
+        self.ws = Workspace(self.dev)
+        self.logits = torch.zeros((1, cfg.vocab), dtype=torch.float32, device=self.dev)
+        self._graphs: dict[int, object] = {}
+        self._slot = None
+        self._start = None              # position of the running portion's first token, None in decode steps
+        self.on_layer = None            # callable(run index, residual [m, width]) after every layer run: a probe for tests
+
+    def _portion(self, ids, m: int):
+        raise NotImplementedError
+
+    def _head_rows(self, portion, rows) -> torch.Tensor:
+        raise NotImplementedError
+
+    # ---- slots ----------------------------------------------------------------------------------
+    def open_slot(self) -> int:
+        return self.pool.open()
+
+    def close_slot(self, slot: int) -> None:
+        self.pool.close(slot)
+
+    def bind(self, slot: int) -> None:
+        if slot == self._slot:
+            return
+        if self._slot is not None:
+            self._graphs[self._slot] = self._graph
+        self._slot, self._graph = slot, self._graphs.get(slot)
+        p = self.pool
+        self.pos, self.tok, self.prev = p.pos[slot, :1], p.tok[slot, :1], p.prev[slot, :1]
+
+    def loop_state(self) -> list:
+        return [self.pos, self.tok, self.prev, self.pool.arena(self._slot)]
+
+    def _run(self, r: int) -> LayerRun:
+        return LayerRun(self.pool.views(self._slot), f"r{r}.", self.pos, self._start)
+
+    # ---- tokens ---------------------------------------------------------------------------------
+    def extend(self, slot: int, ids: torch.Tensor, want) -> torch.Tensor:
+        """The sequence's next tokens (prompt portions of any size, or single tokens through the captured decode step).
+        Leaves tok = the greedy next token and pos = the sequence's length, ready for ``generate``."""
+        n, start = int(ids.numel()), self.pool.length[slot]
+        if n == 0 or start + n > self.max_seq:
+            raise ops.Hf2qError(_lib.ERR_INVALID_ARGUMENT, f"{n} tokens after {start}: the model was loaded for sequences of 1..{self.max_seq}")
+        self.bind(slot)
+        ids = ids.to(self.dev, torch.int32).contiguous()
+        want = list(want)
+        out = torch.empty((len(want), self.cfg.vocab), dtype=torch.float32, device=self.dev)
+        for c0 in range(0, n, self.chunk):
+            m = min(self.chunk, n - c0)
+            here = [(j, p - c0) for j, p in enumerate(want) if c0 <= p < c0 + m]
+            last = c0 + m == n
+            self.pos.fill_(start + c0)
+            if m == 1 and self.on_layer is None:
+                self.tok.copy_(ids[c0:c0 + 1])
+                self.ensure_graph()
+                self._graph.replay()
+                if here:
+                    out[[j for j, _ in here]] = self.logits
+                continue
+            self._start = start + c0
+            x = self._portion(ids[c0:c0 + m], m)
+            self._start = None
+            rows = [p for _, p in here]
+            logits = self._head_rows(x, rows + [m - 1]) if last or rows else None
+            if rows:
+                out[torch.tensor([j for j, _ in here], device=self.dev)] = logits[:len(rows)]
+            if last:
+                self.logits.copy_(logits[-1:])
+                self.sop.argmax(self.logits, self.tok)
+                self.pos.fill_(start + n)
+        self.pool.length[slot] = start + n
+        return out
+
+    def generate(self, n: int, use_graph: bool = True, collect: bool = True):
+        if self.pool.length[self._slot] + n > self.max_seq:
+            raise ops.Hf2qError(_lib.ERR_INVALID_ARGUMENT, f"{n} more tokens do not fit the {self.max_seq} the model was loaded for")
+        out = super().generate(n, use_graph, collect)
+        self.pool.length[self._slot] += n
         return out
 
 

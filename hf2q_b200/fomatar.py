@@ -15,10 +15,9 @@ from pathlib import Path
 import torch
 
 from . import _lib, ops
-from .decoder import GreedyDecoder
-from .mixers import MIXERS, LayerRun, Workspace
+from .decoder import SlotDecoder
+from .mixers import MIXERS
 from .safetensors import SafetensorsFile
-from .state import StatePool
 from .seqops import (EPI_ADD, EPI_GELU, EPI_NONE, EPI_SOFTCAP, PRO_NONE, PRO_NORM, DenseWeight, Embed, Matvec, PreNorm, SeqOps, pad8, struct)
 
 
@@ -43,7 +42,7 @@ class FomatarConfig:
 
     def __post_init__(self):
         for i, e in enumerate(self.layers):
-            if e["type"] not in MIXERS:
+            if e["type"] not in ("parallel", "channel_delta"):
                 raise _bad(f"layer {i}: unknown mixer '{e['type']}'")
             if e.get("mlp") and e["mlp"].get("kind", "dense") != "dense":
                 raise _bad(f"layer {i}: unknown feed-forward '{e['mlp']['kind']}'")
@@ -122,7 +121,7 @@ class _Layer:
             self.down = DenseWeight(load(p)("mlp.down", w, ff), device)
 
 
-class FomatarDecoder(GreedyDecoder):
+class FomatarDecoder(SlotDecoder):
     """n_slots sequences may be open; steps run one sequence at a time."""
 
     def __init__(self, ctx: ops.GpuContext, cfg: FomatarConfig, get, dtype=torch.bfloat16, max_seq: int = 32768, n_slots: int = 1,
@@ -130,10 +129,8 @@ class FomatarDecoder(GreedyDecoder):
         """``get(name)`` returns a weight as a CPU tensor.  ``max_seq``: most tokens of one sequence."""
         if dtype not in (torch.bfloat16, torch.float32):
             raise _bad(f"dtype {dtype} (want bfloat16 or float32)")
-        self.ctx, self.cfg, self.act, self.max_seq, self.n_slots = ctx, cfg, dtype, max_seq, n_slots
-        self.dev = torch.device("cuda", ctx.device)
+        super().__init__(ctx, cfg, dtype, max_seq, n_slots, prefill_chunk)
         self.sop = SeqOps(ctx)
-        self.chunk = min(prefill_chunk, max_seq)
         w, dev = cfg.width, self.dev
         bf = lambda name: get(name).to(torch.bfloat16).contiguous().to(dev)
         self.embed_w = bf("embed")
@@ -156,16 +153,10 @@ class FomatarDecoder(GreedyDecoder):
         if (self.head.n, self.head.k_raw) != (cfg.vocab, w):
             raise _bad(f"head: shape {[self.head.n, self.head.k_raw]}, expected {[cfg.vocab, w]}")
 
-        self.pool = StatePool(n_slots, dev)
         for r, run in enumerate(self.runs):
             self.pool.recurrent(f"r{r}.shift", 2, w)
             self.layers[run.layer].mixer.declare(self.pool, f"r{r}.", self.chunk, dtype)
         self.pool.allocate()
-        self.ws = Workspace(dev)
-        self.logits = torch.zeros((1, cfg.vocab), dtype=torch.float32, device=dev)
-        self._graphs: dict[int, object] = {}
-        self._slot = None
-        self.on_layer = None            # callable(run index, residual [m, width]) after every layer run: a probe for tests
 
     @classmethod
     def from_directory(cls, ctx, path, **kw) -> "FomatarDecoder":
@@ -175,28 +166,6 @@ class FomatarDecoder(GreedyDecoder):
             return cls(ctx, FomatarConfig.load(path / "config.json"), st.load_tensor, **kw)
         finally:
             st.close()
-
-    # ---- slots ----------------------------------------------------------------------------------
-    def open_slot(self) -> int:
-        return self.pool.open()
-
-    def close_slot(self, slot: int) -> None:
-        self.pool.close(slot)
-
-    def bind(self, slot: int) -> None:
-        if slot == self._slot:
-            return
-        if self._slot is not None:
-            self._graphs[self._slot] = self._graph
-        self._slot, self._graph = slot, self._graphs.get(slot)
-        p = self.pool
-        self.pos, self.tok, self.prev = p.pos[slot, :1], p.tok[slot, :1], p.prev[slot, :1]
-
-    def loop_state(self) -> list:
-        return [self.pos, self.tok, self.prev, self.pool.arena(self._slot)]
-
-    def _run(self, r: int) -> LayerRun:
-        return LayerRun(self.pool.views(self._slot), f"r{r}.", self.pos)
 
     # ---- pieces shared by the two ways to run -----------------------------------------------------
     def _embed(self, ids, m, x):
@@ -310,47 +279,6 @@ class FomatarDecoder(GreedyDecoder):
         self.sop.pre_norm(self._pre(xs, None, self.final_norm), n, xn)
         out = torch.empty((n, c.vocab), dtype=torch.float32, device=self.dev)
         self.sop.matmul(xn, self.head, out, n, epilogue=EPI_SOFTCAP if c.softcap else EPI_NONE, cap=c.softcap or 0.0)
-        return out
-
-    def extend(self, slot: int, ids: torch.Tensor, want) -> torch.Tensor:
-        """The sequence's next tokens (prompt portions of any size, or single tokens through the captured decode step).
-        Leaves tok = the greedy next token and pos = the sequence's length, ready for ``generate``."""
-        n, start = int(ids.numel()), self.pool.length[slot]
-        if n == 0 or start + n > self.max_seq:
-            raise _bad(f"{n} tokens after {start}: the model was loaded for sequences of 1..{self.max_seq}")
-        self.bind(slot)
-        ids = ids.to(self.dev, torch.int32).contiguous()
-        want = list(want)
-        out = torch.empty((len(want), self.cfg.vocab), dtype=torch.float32, device=self.dev)
-        for c0 in range(0, n, self.chunk):
-            m = min(self.chunk, n - c0)
-            here = [(j, p - c0) for j, p in enumerate(want) if c0 <= p < c0 + m]
-            last = c0 + m == n
-            self.pos.fill_(start + c0)
-            if m == 1 and self.on_layer is None:
-                self.tok.copy_(ids[c0:c0 + 1])
-                self.ensure_graph()
-                self._graph.replay()
-                if here:
-                    out[[j for j, _ in here]] = self.logits
-                continue
-            x = self._portion(ids[c0:c0 + m], m)
-            rows = [p for _, p in here]
-            logits = self._head_rows(x, rows + [m - 1]) if last or rows else None
-            if rows:
-                out[torch.tensor([j for j, _ in here], device=self.dev)] = logits[:len(rows)]
-            if last:
-                self.logits.copy_(logits[-1:])
-                self.sop.argmax(self.logits, self.tok)
-                self.pos.fill_(start + n)
-        self.pool.length[slot] = start + n
-        return out
-
-    def generate(self, n: int, use_graph: bool = True, collect: bool = True):
-        if self.pool.length[self._slot] + n > self.max_seq:
-            raise _bad(f"{n} more tokens do not fit the {self.max_seq} the model was loaded for")
-        out = super().generate(n, use_graph, collect)
-        self.pool.length[self._slot] += n
         return out
 
     # ---- sizes --------------------------------------------------------------------------------------

@@ -2,45 +2,17 @@
 
 A mixer owns its weights, declares its per-sequence state in a ``StatePool`` and runs two ways on the current stream:
 ``decode`` (one token, prologues and epilogues fused into the products, capturable) and ``prefill`` (a portion of
-m tokens).  Both get the fused projection of the layer's input and leave the mixer's result either added to the
-residual stream (``adds_residual``) or as the two vectors that the next row prologue combines (``combines``).
+m tokens).  Both get the fused projection of the layer's input and leave the mixer's result added to the residual
+stream (``adds_residual``), as the two vectors that the next row prologue combines (``combines``), or else return it.
 """
 from __future__ import annotations
 
-from dataclasses import dataclass
-
 import torch
 
-from .seqops import EPI_ADD, PRO_GATED, Delta, DenseWeight, GatedHeads, MLstm, Matvec, SeqOps, WindowAttn, pad8, pad32, struct
 from .ops import DT_BF16, DT_F32
-
-
-@dataclass
-class Workspace:
-    """Named scratch buffers that grow to the largest use; a name is one buffer for all layers."""
-    device: object
-
-    def __post_init__(self):
-        self._bufs = {}
-
-    def get(self, name: str, rows: int, cols: int, dtype=torch.float32) -> torch.Tensor:
-        key = (name, dtype)
-        need = rows * cols
-        b = self._bufs.get(key)
-        if b is None or b.numel() < need:
-            b = torch.zeros(need, dtype=dtype, device=self.device)
-            self._bufs[key] = b
-        return b[:need].view(rows, cols)
-
-
-class LayerRun:
-    """What a mixer needs from the model for one execution of a layer on one sequence."""
-
-    def __init__(self, views: dict, prefix: str, pos: torch.Tensor):
-        self._views, self._prefix, self.pos = views, prefix, pos
-
-    def state(self, name: str) -> torch.Tensor:
-        return self._views[self._prefix + name]
+from .seqops import (EPI_ADD, GATE_SILU_FIRST, PRO_GATED, PRO_NONE, Delta, DenseWeight, GatedHeads, LatentAttn, MLstm, Matvec, SeqOps, Ssd, WindowAttn, pad8,
+                     pad32, struct)
+from .state import LayerRun, Workspace
 
 
 def _off(t: torch.Tensor, cols: int) -> int:
@@ -205,4 +177,134 @@ class ChannelDelta:
         return self.proj.nbytes + self.a2.nbytes + self.g2.nbytes + self.o.nbytes + 8 * c["heads"] * c["vdim"] * pad32(c["dim"])
 
 
-MIXERS = {"parallel": ParallelWindowMLstm, "channel_delta": ChannelDelta}
+class Mamba2:
+    """State-space layer with a scalar decay per head and token; short convolution on x, B and C; the output is gated
+    before it is normed in equal parts."""
+    combines, adds_residual = False, False
+
+    def __init__(self, sop: SeqOps, cfg: dict, eps: float, width: int, load, load_f32, device, act, window_cap: int):
+        self.sop, self.eps, self.width, self.act, self.c = sop, eps, width, act, cfg
+        H, G, N, taps = cfg["heads"], cfg["groups"], cfg["state"], cfg["conv"]
+        self.inner = H * cfg["vdim"]
+        self.channels = self.inner + 2 * G * N
+        if H % G or self.inner % cfg["norm_groups"]:
+            raise ValueError(f"mamba2: {H} heads in {G} groups, {self.inner} outputs in {cfg['norm_groups']} normed parts")
+        self.proj = DenseWeight(load("in", self.inner + self.channels + H, width), device)
+        self.o = DenseWeight(load("o", width, self.inner), device)
+        f = lambda n, *s: load_f32(n, *s).to(device)
+        self.conv, self.conv_b = f("conv", self.channels, taps), f("conv.b", self.channels)
+        self.dt_bias, self.a_log, self.d, self.norm = f("dt_bias", H), f("A_log", H), f("D", H), f("norm", self.inner)
+
+    def declare(self, pool, prefix: str, max_portion: int, cache_dtype) -> None:
+        c = self.c
+        pool.recurrent(prefix + "conv", self.channels, c["conv"])
+        pool.recurrent(prefix + "s", c["heads"], c["vdim"], pad32(c["state"]))
+
+    def _ssd(self, run: LayerRun, proj) -> Ssd:
+        c = self.c
+        return struct(Ssd, proj=proj, ld=proj.stride(0), off=self.inner, conv=self.conv, conv_bias=self.conv_b, dt_bias=self.dt_bias, a_log=self.a_log, d=self.d,
+                      conv_state=run.state("conv"), s=run.state("s"), heads=c["heads"], groups=c["groups"], state=c["state"], vdim=c["vdim"], taps=c["conv"],
+                      pos=run.pos)
+
+    def _gate(self, y, proj) -> GatedHeads:
+        n = self.c["norm_groups"]
+        return struct(GatedHeads, o=y, gate=proj, norm=self.norm, ldo=y.stride(0), ldg=proj.stride(0), heads=n, head_dim=self.inner // n, norm_all=1,
+                      eps=self.eps, kind=GATE_SILU_FIRST)
+
+    def decode(self, run: LayerRun, ws: Workspace, proj, x=None):
+        y, out = ws.get("d.mem", 1, self.inner), ws.get("d.y", 1, self.width)
+        self.sop.ssd_step(self._ssd(run, proj), y)
+        self.sop.matvec(PRO_GATED, struct(Matvec, w=self.o.w, y=out, gated=self._gate(y, proj), n=self.o.n, k=self.o.k))
+        return out
+
+    def prefill(self, run: LayerRun, ws: Workspace, proj, x, m: int):
+        sop, a, H = self.sop, self._ssd(run, proj), self.c["heads"]
+        xbc, dt, la = ws.get("xbc", m, self.channels), ws.get("dt", m, H), ws.get("la", m, H)
+        y, gated, out = ws.get("mem", m, self.inner), ws.get("gated", m, self.o.k, self.act), ws.get("y", m, self.width)
+        sop.ssd_prep(a, m, xbc, dt, la)
+        sop.ssd_scan(a, m, xbc, dt, la, y)
+        sop.gated_heads(self._gate(y, proj), m, gated)
+        sop.matmul(gated, self.o, out, m)
+        return out
+
+    def decode_bytes(self) -> int:
+        c = self.c
+        return self.proj.nbytes + self.o.nbytes + 8 * c["heads"] * c["vdim"] * pad32(c["state"])
+
+
+class LatentAttention:
+    """Sliding-window attention whose keys and values are expanded from one cached latent vector per token; a rotated part
+    of every key is shared by the heads.  Decoding moves the query into the latent space instead, portions expand the
+    window's latents."""
+    combines, adds_residual = False, False
+
+    def __init__(self, sop: SeqOps, cfg: dict, eps: float, width: int, load, load_f32, device, act, window_cap: int):
+        self.sop, self.eps, self.width, self.act, self.c = sop, eps, width, act, cfg
+        H, d, r, dv, rank, rot = cfg["heads"], cfg["dim"], cfg["rot_dim"], cfg["vdim"], cfg["kv_rank"], cfg["rot"]
+        if rot["dims"] % 2 or rot["dims"] > r:
+            raise ValueError(f"latent attention: {rot['dims']} turned dimensions of {r}")
+        self.window = min(cfg["mask"]["size"], window_cap)
+        self.proj = DenseWeight([load("q", H * (d + r), width), load("dkv", rank + r, width)], device)
+        uk, uv = load("uk", H * d, rank), load("uv", H * dv, rank)
+        self.dp, self.vp, self.rp, self.row = pad8(d), pad8(dv), pad8(rank), pad8(rank) + pad8(r)
+        # portions: every head's keys, then every head's values, at multiples of 8 columns
+        self.ukv = DenseWeight(list(uk.split(d)) + list(uv.split(dv)), device)
+        # decoding: uk transposed per head
+        self.uk_t = DenseWeight(uk.view(H, d, rank).transpose(1, 2).reshape(H * rank, d), device)
+        self.uv = DenseWeight(uv, device)
+        self.o = DenseWeight(load("o", width, H * dv), device)
+        self.norm = load_f32("dkv.norm", rank).to(device)
+        i = torch.arange(rot["dims"] // 2, dtype=torch.float64)
+        self.freq = (float(rot["base"]) ** (-2.0 * i / rot["dims"])).float().to(device)
+        if self.freq.numel() == 0:
+            self.freq = torch.zeros(1, device=device)
+        self.scratch = None
+
+    def declare(self, pool, prefix: str, max_portion: int, cache_dtype) -> None:
+        self.capacity, self.cache_dtype = self.window - 1 + max_portion, cache_dtype
+        pool.ring(prefix + "latent", (self.capacity, self.row), cache_dtype)
+
+    def _attn(self, run: LayerRun, proj) -> LatentAttn:
+        c = self.c
+        return struct(LatentAttn, proj=proj, ld=proj.stride(0), q_off=self.proj.offsets[0], c_off=self.proj.offsets[1], norm=self.norm, freq=self.freq,
+                      uk_t=self.uk_t.w, uv=self.uv.w, cache=run.state("latent"), heads=c["heads"], dim=c["dim"], rot_dim=c["rot_dim"],
+                      rot_pairs=c["rot"]["dims"] // 2, vdim=c["vdim"], kv_rank=c["kv_rank"], window=self.window, capacity=self.capacity,
+                      cache_dtype=DT_F32 if self.cache_dtype == torch.float32 else DT_BF16, scale=c["scale"], eps=self.eps, pos=run.pos)
+
+    def decode(self, run: LayerRun, ws: Workspace, proj, x=None):
+        c, sop = self.c, self.sop
+        att, out = ws.get("d.att", 1, self.o.k), ws.get("d.y", 1, self.width)
+        a = self._attn(run, proj)
+        if self.scratch is None:
+            self.scratch = sop.latent_scratch(a, ws.device)
+        sop.latent_decode(a, att, self.scratch)
+        sop.matvec(PRO_NONE, struct(Matvec, w=self.o.w, y=out, x=att, n=self.o.n, k=self.o.k))
+        return out
+
+    def prefill(self, run: LayerRun, ws: Workspace, proj, x, m: int):
+        c, sop, H, dt = self.c, self.sop, self.c["heads"], self.cache_dtype
+        a, cache = self._attn(run, proj), run.state("latent")
+        q = ws.get("q", m, H * (self.dp + pad8(c["rot_dim"])), dt)
+        sop.latent_append(a, m, q)
+        # keys and values of the window's tokens, oldest first; the ring's end cuts them in two at most
+        first = max(0, run.start - (self.window - 1))
+        n, at = run.start + m - first, first % self.capacity
+        kv = ws.get("kv", n, self.ukv.n, dt)
+        for lo, hi, slot in ((0, min(n, self.capacity - at), at), (min(n, self.capacity - at), n, 0)):
+            if hi > lo:
+                sop.matmul(cache[slot:slot + hi - lo], self.ukv, kv[lo:hi], hi - lo)
+        att, out = ws.get("att", m, self.o.k, self.act), ws.get("y", m, self.width)
+        w = struct(WindowAttn, qkv=proj, k_cache=kv, v_cache=_off(kv, H * self.dp), heads=H, kv_heads=H, dim=c["dim"], vdim=c["vdim"], window=self.window,
+                   capacity=self.capacity, cache_dtype=a.cache_dtype, scale=c["scale"], eps=self.eps, pos=run.pos, linear=1, row_stride=self.ukv.n,
+                   k_head_stride=self.dp, v_head_stride=self.vp, k_shared=_off(cache, self.rp), shared_dim=c["rot_dim"], shared_stride=self.row,
+                   shared_capacity=self.capacity)
+        sop.window_prefill(w, m, q, None, 0, att)
+        sop.matmul(att, self.o, out, m)
+        return out
+
+    def decode_bytes(self) -> int:
+        kv = self.window * self.row * (4 if self.act == torch.float32 else 2)
+        return self.proj.nbytes + self.uk_t.nbytes + self.uv.nbytes + self.o.nbytes + kv
+
+
+MIXERS = {"parallel": ParallelWindowMLstm, "channel_delta": ChannelDelta, "mamba2": Mamba2, "latent_attention": LatentAttention}

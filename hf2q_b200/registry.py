@@ -14,6 +14,11 @@ def _fomatar(ctx, path, dtype, max_seq, n_slots, prefill_chunk):
     return FomatarDecoder.from_directory(ctx, path, dtype=dtype, max_seq=max_seq, n_slots=n_slots, prefill_chunk=prefill_chunk)
 
 
+def _runopel(ctx, path, dtype, max_seq, n_slots, prefill_chunk):
+    from .runopel import RunopelDecoder
+    return RunopelDecoder.from_directory(ctx, path, dtype=dtype, max_seq=max_seq, n_slots=n_slots, prefill_chunk=prefill_chunk)
+
+
 def _llama(ctx, path, dtype, max_seq, n_slots, prefill_chunk):
     from .decoder import LlamaDecoder
     if dtype != torch.bfloat16:
@@ -22,7 +27,7 @@ def _llama(ctx, path, dtype, max_seq, n_slots, prefill_chunk):
 
 
 # config.json "architecture" of a model folder, or "general.architecture" of a GGUF file
-ARCHITECTURES = {"Fomatar": _fomatar, "llama": _llama}
+ARCHITECTURES = {"Fomatar": _fomatar, "Runopel": _runopel, "llama": _llama}
 
 
 def architecture_of(path) -> str:

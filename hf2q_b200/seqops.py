@@ -9,8 +9,10 @@ import torch
 from . import ops
 from .ops import DT_BF16, DT_F32, _TORCH_DT
 
-EPI_NONE, EPI_GELU, EPI_ADD, EPI_SOFTCAP = range(4)
-PRO_NONE, PRO_NORM, PRO_GATED = range(3)
+EPI_NONE, EPI_GELU, EPI_ADD, EPI_SOFTCAP, EPI_SCALE, EPI_SWIGLU, EPI_CLAMP_GLU = range(7)
+PRO_NONE, PRO_NORM, PRO_GATED, PRO_HYPER = range(4)
+GATE_SIGMOID_LAST, GATE_SILU_FIRST = range(2)
+GROUP_TILE = {torch.float32: 64, torch.bfloat16: 128}        # rows per tile of the grouped products
 _vp, _u32, _u64, _f32 = C.c_void_p, C.c_uint32, C.c_uint64, C.c_float
 
 
@@ -31,11 +33,23 @@ class PreNorm(C.Structure):
 
 
 class GatedHeads(C.Structure):
-    _fields_ = _fields("o gate norm", "ldo ldg heads head_dim norm_all", "eps")
+    _fields_ = _fields("o gate norm", "ldo ldg heads head_dim norm_all", "eps") + [("kind", _u32)]
+
+
+class Hyper(C.Structure):
+    _fields_ = _fields("x x_out y mix out c_in norm h_out", "x_streams streams y_parts width", "eps")
 
 
 class Matvec(C.Structure):
-    _fields_ = _fields("w y residual x") + [("pre", PreNorm), ("gated", GatedHeads)] + _fields("", "n k epilogue", "cap")
+    _fields_ = _fields("w y residual x") + [("pre", PreNorm), ("gated", GatedHeads)] + _fields("", "n k epilogue", "cap") + [("hyper", Hyper), ("bias", _vp)]
+
+
+class RowGroups(C.Structure):
+    _fields_ = _fields("header tiles perm row_scale", "groups tile_rows scatter reserved")
+
+
+class ExpertStep(C.Structure):
+    _fields_ = _fields("gate_up down logits h ids act y", "experts top ff width k_in")
 
 
 class Embed(C.Structure):
@@ -44,7 +58,17 @@ class Embed(C.Structure):
 
 class WindowAttn(C.Structure):
     _fields_ = _fields("qkv", "ld q_off k_off v_off") + _fields("q_norm k_norm r1 r2 k_cache v_cache",
-                                                                "heads kv_heads dim vdim window capacity cache_dtype", "scale eps") + _fields("pos")
+                                                                "heads kv_heads dim vdim window capacity cache_dtype", "scale eps") + _fields(
+        "pos", "linear row_stride k_head_stride v_head_stride") + _fields("k_shared", "shared_dim shared_stride shared_capacity reserved")
+
+
+class LatentAttn(C.Structure):
+    _fields_ = _fields("proj", "ld q_off c_off") + _fields("norm freq uk_t uv cache", "heads dim rot_dim rot_pairs vdim kv_rank window capacity cache_dtype",
+                                                           "scale eps") + _fields("pos")
+
+
+class Ssd(C.Structure):
+    _fields_ = _fields("proj", "ld off") + _fields("conv conv_bias dt_bias a_log d conv_state s", "heads groups state vdim taps") + _fields("pos")
 
 
 class MLstm(C.Structure):
@@ -100,9 +124,27 @@ class SeqOps:
     def embed(self, e: Embed, ids, m, x):
         self._call("embed", C.byref(e), ptr(ids), m, ptr(x))
 
-    def matmul(self, x, w: DenseWeight, y, m, epilogue=EPI_NONE, residual=None, cap=0.0):
+    def matmul(self, x, w: DenseWeight, y, m, epilogue=EPI_NONE, residual=None, cap=0.0, bias=None):
         self._call("dense_matmul", ptr(x), _TORCH_DT[x.dtype], x.stride(0), ptr(w.w), ptr(y), _TORCH_DT[y.dtype], y.stride(0), m, w.n, w.k, epilogue,
-                   ptr(residual), cap)
+                   ptr(residual), cap, ptr(bias))
+
+    def grouped(self, g: RowGroups, x, w: DenseWeight, y, rows, epilogue=EPI_NONE, cap=0.0):
+        """``w`` holds the matrices of all groups one below the other."""
+        self._call("dense_grouped", C.byref(g), ptr(x), _TORCH_DT[x.dtype], x.stride(0), ptr(w.w), ptr(y), _TORCH_DT[y.dtype], y.stride(0), rows,
+                   w.n // g.groups, w.k, epilogue, cap)
+
+    def sigmoid_topk(self, logits, ids, weights, m, experts, top):
+        self._call("moe_sigmoid_topk", ptr(logits), logits.stride(0), ptr(ids), ptr(weights), m, experts, top)
+
+    def sort_rows(self, ids, m, top, experts, x, header, tiles, perm, xg):
+        self._call("sort_rows", ptr(ids), m, top, experts, GROUP_TILE[x.dtype], ptr(x), _TORCH_DT[x.dtype], x.stride(0), ptr(header), ptr(tiles), ptr(perm), ptr(xg))
+
+    def expert_step(self, e: ExpertStep):
+        self._call("expert_glu_step", C.byref(e))
+        self._call("expert_down_step", C.byref(e))
+
+    def hyper_norm(self, p: Hyper, m, out):
+        self._call("hyper_norm", C.byref(p), m, ptr(out), _TORCH_DT[out.dtype], out.stride(0))
 
     def matvec(self, prologue, *segs: Matvec):
         self._call("dense_matvec", prologue, (Matvec * len(segs))(*segs), len(segs))
@@ -126,6 +168,26 @@ class SeqOps:
 
     def window_prefill(self, a: WindowAttn, m, q, gate_ptr, ldg, out):
         self._call("window_attn_prefill", C.byref(a), m, ptr(q), gate_ptr, ldg, ptr(out), _TORCH_DT[out.dtype], out.stride(0))
+
+    def latent_scratch(self, a: LatentAttn, device) -> torch.Tensor:
+        need = C.c_uint64()
+        self.ctx._check(self.lib.hf2q_cuda_latent_scratch_bytes(self.ctx._h, C.byref(a), C.byref(need)))
+        return torch.zeros(need.value, dtype=torch.uint8, device=device)
+
+    def latent_decode(self, a: LatentAttn, out, scratch):
+        self._call("latent_decode", C.byref(a), ptr(out), ptr(scratch), scratch.numel())
+
+    def latent_append(self, a: LatentAttn, m, q_out):
+        self._call("latent_append", C.byref(a), m, ptr(q_out))
+
+    def ssd_step(self, a: Ssd, y):
+        self._call("ssd_step", C.byref(a), ptr(y))
+
+    def ssd_prep(self, a: Ssd, m, xbc, dt, la):
+        self._call("ssd_prep", C.byref(a), m, ptr(xbc), ptr(dt), ptr(la))
+
+    def ssd_scan(self, a: Ssd, m, xbc, dt, la, y):
+        self._call("ssd_scan", C.byref(a), m, ptr(xbc), ptr(dt), ptr(la), ptr(y))
 
     def mlstm(self, a: MLstm, m, out):
         self._call("mlstm", C.byref(a), m, ptr(out))

@@ -6,6 +6,8 @@ buffers of a slot are views into one flat f32 arena, so giving a slot to a new s
 """
 from __future__ import annotations
 
+from dataclasses import dataclass
+
 import torch
 
 
@@ -71,3 +73,32 @@ class StatePool:
     @property
     def n_free(self) -> int:
         return len(self._free)
+
+
+@dataclass
+class Workspace:
+    """Named scratch buffers that grow to the largest use; a name is one buffer for all layers."""
+    device: object
+
+    def __post_init__(self):
+        self._bufs = {}
+
+    def get(self, name: str, rows: int, cols: int, dtype=torch.float32) -> torch.Tensor:
+        key = (name, dtype)
+        need = rows * cols
+        b = self._bufs.get(key)
+        if b is None or b.numel() < need:
+            b = torch.zeros(need, dtype=dtype, device=self.device)
+            self._bufs[key] = b
+        return b[:need].view(rows, cols)
+
+
+class LayerRun:
+    """What a mixer needs from the model for one execution of a layer on one sequence."""
+
+    def __init__(self, views: dict, prefix: str, pos: torch.Tensor, start: int | None = None):
+        """``pos``: the position on the device; ``start``: the same on the host, known for portions only."""
+        self._views, self._prefix, self.pos, self.start = views, prefix, pos, start
+
+    def state(self, name: str) -> torch.Tensor:
+        return self._views[self._prefix + name]

@@ -646,14 +646,42 @@ HF2Q_API int32_t hf2q_cuda_add(hf2q_ctx* ctx, void* stream, float* x, const floa
 /* ---- decoder designs with bf16 weights: products, recurrent mixers, windowed attention ------------------ *
  * Weights are row-major bf16 [n][k], k a multiple of 8 (pad with zero columns), 16-byte aligned.  Activations are
  * f32, or bf16 in front of the tensor-core product.  x f32 and no tensor-core use = every step in 32-bit. */
-enum { HF2Q_EPI_NONE = 0, HF2Q_EPI_GELU = 1, HF2Q_EPI_ADD = 2, HF2Q_EPI_SOFTCAP = 3 };
+enum { HF2Q_EPI_NONE = 0, HF2Q_EPI_GELU = 1, HF2Q_EPI_ADD = 2, HF2Q_EPI_SOFTCAP = 3, HF2Q_EPI_SCALE = 4, HF2Q_EPI_SWIGLU = 5, HF2Q_EPI_CLAMP_GLU = 6 };
 
 /* y[m][n] = epilogue(x[m][k] . w^T), rows of x / y are ldx / ldy elements apart.  m <= 8: mat-vec kernel (fp32
  * arithmetic); more rows: tcgen05 for bf16 x, a CUDA-core fp32 product for f32 x.  ADD: + residual (layout of y, may
- * be y); GELU: tanh form; SOFTCAP: cap * tanh(y / cap).  y_dtype f32 or bf16. */
+ * be y); GELU: tanh form; SOFTCAP: cap * tanh(y / cap); SCALE: cap * y.  SWIGLU and CLAMP_GLU take the rows of w in pairs
+ * (gate, up) and write n / 2 columns: silu(g) u, or with g = min(g, cap), u = clamp(u, -cap, cap): g sigmoid(1.702 g)
+ * (u + 1).  bias f32 [n] (NULL: none) is added first.  y_dtype f32 or bf16. */
 HF2Q_API int32_t hf2q_cuda_dense_matmul(hf2q_ctx* ctx, void* stream, const void* x, uint32_t x_dtype, uint32_t ldx,
                                         const void* w, void* y, uint32_t y_dtype, uint32_t ldy, uint32_t m, uint32_t n,
-                                        uint32_t k, uint32_t epilogue, const float* residual, float cap);
+                                        uint32_t k, uint32_t epilogue, const float* residual, float cap, const float* bias);
+
+/* Products of rows that are sorted by group (expert), group g with the matrix w[g] of [groups][n][k]. */
+enum { HF2Q_GROUP_TILE_F32 = 64, HF2Q_GROUP_TILE_BF16 = 128 };
+typedef struct hf2q_row_groups {
+    const uint32_t* header;      /* [0] number of tiles, [1] number of sorted rows (hf2q_cuda_sort_rows) */
+    const void* tiles;           /* uint4 [..]: group, first sorted row, rows, 0 */
+    const uint32_t* perm;        /* sorted row -> routed row */
+    const float* row_scale;      /* f32 by routed row: multiplies the sums before the epilogue (NULL: 1) */
+    uint32_t groups, tile_rows;
+    uint32_t scatter;            /* 1: y rows in routed order, 0: in sorted order */
+    uint32_t reserved;
+} hf2q_row_groups;
+/* rows: sorted rows of x (ldx apart, a multiple of 8 elements).  x bf16: tcgen05, y f32 or bf16; x f32: fp32 products, y f32. */
+HF2Q_API int32_t hf2q_cuda_dense_grouped(hf2q_ctx* ctx, void* stream, const hf2q_row_groups* g, const void* x, uint32_t dtype,
+                                         uint32_t ldx, const void* w, void* y, uint32_t y_dtype, uint32_t ldy, uint32_t rows,
+                                         uint32_t n, uint32_t k, uint32_t epilogue, float cap);
+/* Router scores and choice per token: s = sigmoid(logits), the `top` largest (equal scores: the lower index first) with
+ * their scores as weights, not renormalised.  logits f32, rows `ld` apart; ids, weights [m][top]. */
+HF2Q_API int32_t hf2q_cuda_moe_sigmoid_topk(hf2q_ctx* ctx, void* stream, const float* logits, uint32_t ld, uint32_t* ids,
+                                            float* weights, uint32_t m, uint32_t experts, uint32_t top);
+/* Groups m * top routed rows by expert: perm, tiles of at most tile_rows rows, header; and copies row (routed / top) of x
+ * (dtype, ldx apart, a multiple of 8 elements of 16-byte aligned rows) to sorted row order in xg [m * top][ldx].
+ * tiles holds m * top / tile_rows + min(m * top, experts) entries of 16 bytes. */
+HF2Q_API int32_t hf2q_cuda_sort_rows(hf2q_ctx* ctx, void* stream, const uint32_t* ids, uint32_t m, uint32_t top, uint32_t experts,
+                                     uint32_t tile_rows, const void* x, uint32_t dtype, uint32_t ldx, uint32_t* header, void* tiles,
+                                     uint32_t* perm, void* xg);
 
 /* What stands in front of a layer's product.  Residual update: x + (rms(a) a_norm + rms(b) b_norm) / 2 if a != NULL,
  * + add0 if not NULL, + step (one row) if not NULL; stored to x_out if not NULL (must not alias x).  Then
@@ -673,19 +701,38 @@ typedef struct hf2q_pre_norm {
 HF2Q_API int32_t hf2q_cuda_pre_norm(hf2q_ctx* ctx, void* stream, const hf2q_pre_norm* p, uint32_t m, void* out,
                                     uint32_t out_dtype, uint32_t ldo, float* h_last);
 
-/* (norm ? o / rms over the head * norm : o) * sigmoid(gate), per head; norm_all: the weight has heads * head_dim
- * elements, else head_dim shared by the heads. */
+/* kind SIGMOID_LAST: (norm ? o / rms over the head * norm : o) * sigmoid(gate), per head; norm_all: the weight has
+ * heads * head_dim elements, else head_dim shared by the heads.  SILU_FIRST: v = o * silu(gate), then v / rms over the group
+ * * norm, with `heads` groups of head_dim elements and norm [heads * head_dim]. */
+enum { HF2Q_GATE_SIGMOID_LAST = 0, HF2Q_GATE_SILU_FIRST = 1 };
 typedef struct hf2q_gated_heads {
     const float *o, *gate, *norm;
     uint32_t ldo, ldg, heads, head_dim, norm_all;
     float eps;
+    uint32_t kind;
 } hf2q_gated_heads;
 HF2Q_API int32_t hf2q_cuda_gated_heads(hf2q_ctx* ctx, void* stream, const hf2q_gated_heads* g, uint32_t m, void* out,
                                        uint32_t out_dtype, uint32_t ldo);
 
+/* Residual in several streams (hyper-connections).  x f32 [m][x_streams][width] (x_streams 1: all streams equal).  With a
+ * pending sublayer output y f32 [m][y_parts][width] (summed over the parts): x_t <- sum_s mix[s][t] x_s + out[t] y, stored
+ * to x_out [m][streams][width] if not NULL.  Then u = sum_s in[s] x_s (in NULL: the plain sum) and h = u / rms(u) * norm
+ * (norm NULL: h = u).  streams <= 16. */
+typedef struct hf2q_hyper {
+    const float* x;
+    float* x_out;            /* hf2q_cuda_hyper_norm: may be x; the fused product: may not */
+    const float *y, *mix, *out, *in, *norm;
+    float* h_out;            /* the fused product only: h, f32 [width] (NULL: not stored) */
+    uint32_t x_streams, streams, y_parts, width;
+    float eps;
+} hf2q_hyper;
+/* out[m][ldo] (f32 or bf16; columns width .. ldo zeroed). */
+HF2Q_API int32_t hf2q_cuda_hyper_norm(hf2q_ctx* ctx, void* stream, const hf2q_hyper* p, uint32_t m, void* out, uint32_t out_dtype,
+                                      uint32_t ldo);
+
 /* One-row products with their prologue and epilogue in the same launch (f32 arithmetic); up to two segments with
  * the same kind of prologue run side by side. */
-enum { HF2Q_PRO_NONE = 0, HF2Q_PRO_NORM = 1, HF2Q_PRO_GATED = 2 };
+enum { HF2Q_PRO_NONE = 0, HF2Q_PRO_NORM = 1, HF2Q_PRO_GATED = 2, HF2Q_PRO_HYPER = 3 };
 typedef struct hf2q_matvec {
     const void* w;
     float* y;
@@ -695,9 +742,24 @@ typedef struct hf2q_matvec {
     hf2q_gated_heads gated;  /* PRO_GATED */
     uint32_t n, k, epilogue;
     float cap;
+    hf2q_hyper hyper;        /* PRO_HYPER */
+    const float* bias;       /* [n] or NULL */
 } hf2q_matvec;
 HF2Q_API int32_t hf2q_cuda_dense_matvec(hf2q_ctx* ctx, void* stream, uint32_t prologue, const hf2q_matvec* segs,
                                         uint32_t n_segs);
+
+/* One token through its routed experts: the choice of hf2q_cuda_moe_sigmoid_topk, then per chosen expert
+ * act = silu(s g) * (s u) with (g, u) = gate_up . h, and y = sum over the chosen of down . act. */
+typedef struct hf2q_expert_step {
+    const void* gate_up;     /* bf16 [experts][2 ff][k_in], gate and up rows alternating */
+    const void* down;        /* bf16 [experts][width][ff] */
+    const float *logits, *h; /* [experts], [k_in] (zeros past the width) */
+    uint32_t* ids;           /* [top] written by the first call, read by the second */
+    float *act, *y;          /* [top][ff], [width] */
+    uint32_t experts, top, ff, width, k_in;      /* ff and k_in multiples of 8 (zero padding) */
+} hf2q_expert_step;
+HF2Q_API int32_t hf2q_cuda_expert_glu_step(hf2q_ctx* ctx, void* stream, const hf2q_expert_step* e);
+HF2Q_API int32_t hf2q_cuda_expert_down_step(hf2q_ctx* ctx, void* stream, const hf2q_expert_step* e);
 
 /* x[t,:] = embed[ids[t],:] (+ bigram[(before * mul_prev + ids[t] * mul_cur) mod buckets,:]; the first token of a sequence takes row
  * `buckets`).  prev: the token in front of ids[0]; left holding ids[m - 1].  embed / bigram bf16, bigram may be NULL. */
@@ -722,7 +784,39 @@ typedef struct hf2q_window_attn {
     uint32_t heads, kv_heads, dim, vdim, window, capacity, cache_dtype;
     float scale, eps;
     const uint32_t* pos;
+    /* hf2q_cuda_window_attn_prefill only.  linear 1: k_cache / v_cache are not rings but plain rows, row i for position
+     * first + i with first = max(0, *pos - (window - 1)), `row_stride` elements apart, a head's elements at head *
+     * k_head_stride / v_head_stride (multiples of 8).  shared_dim > 0: every key has shared_dim more elements that its
+     * heads share, in the ring k_shared [shared_capacity] with rows shared_stride apart; q rows are then
+     * [heads][dim padded to 8, shared_dim padded to 8]. */
+    uint32_t linear, row_stride, k_head_stride, v_head_stride;
+    const void* k_shared;
+    uint32_t shared_dim, shared_stride, shared_capacity, reserved;
 } hf2q_window_attn;
+
+/* Latent attention: one latent vector and one rotated key part per token, shared by all heads.  Rows of proj (ld apart)
+ * hold q [heads][dim + rot_dim] at q_off and [kv_rank + rot_dim] at c_off.  c = rms norm of the first kv_rank times norm;
+ * the rotated parts turn pair (2i, 2i + 1), i < rot_pairs, by position * freq[i].  Per head: key = [uk c, rotated part],
+ * value = uv c, score = q . key * scale; key j is visible to i when 0 <= i - j < window.  cache: ring [capacity][row],
+ * row = kv_rank padded to 8, then rot_dim padded to 8 (the padding stays zero), f32 or bf16. */
+typedef struct hf2q_latent_attn {
+    const float* proj;
+    uint32_t ld, q_off, c_off;
+    const float *norm, *freq;
+    const void *uk_t, *uv;       /* decode: bf16 [heads][kv_rank][dim padded to 8], [heads][vdim][kv_rank padded to 8] */
+    void* cache;
+    uint32_t heads, dim, rot_dim, rot_pairs, vdim, kv_rank, window, capacity, cache_dtype;
+    float scale, eps;
+    const uint32_t* pos;
+} hf2q_latent_attn;
+HF2Q_API int32_t hf2q_cuda_latent_scratch_bytes(hf2q_ctx* ctx, const hf2q_latent_attn* a, uint64_t* out);
+/* One token: latent to the cache, query moved into the latent space, attention over it, values: out f32 [heads * vdim]. */
+HF2Q_API int32_t hf2q_cuda_latent_decode(hf2q_ctx* ctx, void* stream, const hf2q_latent_attn* a, float* out, void* scratch,
+                                         uint64_t scratch_bytes);
+/* m tokens (window - 1 + m <= capacity): latents to the cache and rotated queries to q_out [m][heads][dim padded to 8, rot_dim
+ * padded to 8] (cache_dtype).  The caller expands the latents of the window (hf2q_cuda_dense_matmul) and runs
+ * hf2q_cuda_window_attn_prefill over them. */
+HF2Q_API int32_t hf2q_cuda_latent_append(hf2q_ctx* ctx, void* stream, const hf2q_latent_attn* a, uint32_t m, void* q_out);
 HF2Q_API int32_t hf2q_cuda_window_attn_scratch_bytes(hf2q_ctx* ctx, const hf2q_window_attn* a, uint64_t* out);
 /* One token: append and attend in one launch.  out f32 [heads * vdim]; scratch zeroed once when allocated. */
 HF2Q_API int32_t hf2q_cuda_window_attn_decode(hf2q_ctx* ctx, void* stream, const hf2q_window_attn* a, float* out,
@@ -776,6 +870,27 @@ HF2Q_API int32_t hf2q_cuda_delta_decay(hf2q_ctx* ctx, void* stream, const hf2q_d
 /* the recurrence over m tokens; out f32 [m][heads * vdim]. */
 HF2Q_API int32_t hf2q_cuda_delta_scan(hf2q_ctx* ctx, void* stream, const hf2q_delta* a, uint32_t m, const float* qkv,
                                       const float* beta, const float* g, float* out);
+
+/* State-space layer with a scalar decay per head and token (Mamba-2).  Rows of proj (ld apart) hold, from off: x
+ * [heads][vdim], B [groups][state], C [groups][state], dt [heads].  x, B, C pass a causal depth-wise convolution (weights
+ * f32 [channels][taps], bias [channels]) and SiLU; dt = softplus(dt + dt_bias).  Head h uses group h / (heads / groups):
+ * S = exp(-exp(a_log[h]) dt) S + dt B x^T, y = S^T C + d[h] x.  conv_state f32 [channels][taps]: the input of position p in
+ * column p % taps.  State f32 s [heads][vdim][state padded to 32]. */
+typedef struct hf2q_ssd {
+    const float* proj;
+    uint32_t ld, off;
+    const float *conv, *conv_bias, *dt_bias, *a_log, *d;
+    float *conv_state, *s;
+    uint32_t heads, groups, state, vdim, taps;
+    const uint32_t* pos;
+} hf2q_ssd;
+/* One token, everything in one launch: y f32 [heads * vdim]. */
+HF2Q_API int32_t hf2q_cuda_ssd_step(hf2q_ctx* ctx, void* stream, const hf2q_ssd* a, float* y);
+/* m tokens: convolution and SiLU -> xbc f32 [m][channels], step sizes and decay logarithms -> dt, la f32 [m][heads]. */
+HF2Q_API int32_t hf2q_cuda_ssd_prep(hf2q_ctx* ctx, void* stream, const hf2q_ssd* a, uint32_t m, float* xbc, float* dt, float* la);
+/* the recurrence over m tokens; y f32 [m][heads * vdim].  Also hands the last taps - 1 convolution inputs over to conv_state. */
+HF2Q_API int32_t hf2q_cuda_ssd_scan(hf2q_ctx* ctx, void* stream, const hf2q_ssd* a, uint32_t m, const float* xbc, const float* dt,
+                                    const float* la, float* y);
 
 /* After a portion of m > 1 tokens: h_last -> shift_state row (pos + m - 1) & 1 (shift_state NULL: none), and the last
  * convolution inputs -> delta->conv_state (delta NULL: none). */
