@@ -780,6 +780,75 @@ class _CallLog:
         return _timed(torch, _graph_of(torch, run).replay, reps), calls
 
 
+def _throughput(torch, ctx, dev, model, vocab, n_prompt, n_new):
+    """Prompt and greedy decoding rates through the decoder's sequence interface, device time; leaves the slot open."""
+    def timed_once(fn):
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        e0.record()
+        fn()
+        e1.record()
+        torch.cuda.synchronize()
+        return e0.elapsed_time(e1) * 1e-3
+
+    ids = torch.randint(0, vocab, (n_prompt,), dtype=torch.int32, device=dev, generator=torch.Generator(device=dev).manual_seed(0))
+    best = 1e9
+    for _ in range(4):
+        slot = model.open_slot()
+        model.bind(slot)
+        best = min(best, timed_once(lambda: model.extend(slot, ids, [])))
+        model.close_slot(slot)
+    slot = model.open_slot()
+    model.extend(slot, ids, [])
+    model.bind(slot)
+    model.generate(8, collect=False)
+    dt = timed_once(lambda: model.generate(n_new, collect=False))
+    ctx.check_status()
+    assert bool(torch.isfinite(model.logits).all())
+    return {"prefill_tok_s": round(n_prompt / best), "decode_tok_s": round(n_new / dt, 1), "decode_us_per_token": round(1e6 * dt / n_new, 1)}, slot
+
+
+def _fomatar_kernels(torch, dev, model, size, vocab, n_prompt, chunk) -> dict:
+    """Every kind of kernel of the Fomatar design alone."""
+    hbm, _ = measured_hbm_peak()
+    _, burst, _ = measured_tensor_peaks()
+    (w, h, g, rh, ff, window), layers = size, len(model.layers)
+    kernels = {}
+    # one decode step, kind by kind
+    with _CallLog(model.sop) as log:
+        model.decode_step()
+    n_par = layers // 2
+    st = 2 * 4 * 128 * 128
+    work = {"dense_matvec": sum(r.nbytes for l in model.layers for r in (l.mixer.proj, l.up, l.down)) + model.head.nbytes +
+            sum(l.mixer.lo.nbytes + l.mixer.ro.nbytes if l.mixer.combines else l.mixer.o.nbytes for l in model.layers),
+            "window_attn_decode": n_par * window * g * 256 * 2, "mlstm": n_par * rh * st,
+            "delta_step": n_par * (h * st + model.layers[1].mixer.a2.nbytes + model.layers[1].mixer.g2.nbytes)}
+    for name, nbytes in work.items():
+        dt, calls = log.time(torch, name)
+        kernels["decode " + name] = {"us": round(1e6 * dt / len(calls), 2), "GB/s": round(nbytes / dt / 1e9), "frac": round(nbytes / dt / 1e9 / hbm, 3)}
+    # one portion deep in a prompt
+    ids = torch.randint(0, vocab, (chunk,), dtype=torch.int32, device=dev)
+    model.pos.fill_(n_prompt - chunk)
+    with _CallLog(model.sop) as log:
+        model._portion(ids, chunk)
+    seen = sum(min(window, n_prompt - chunk + i + 1) for i in range(chunk))
+    flop = {"dense_matmul": 2 * chunk * sum(r.n * r.k for l in model.layers for r in (l.mixer.proj, l.up, l.down)) + 2 * chunk * sum(
+                l.mixer.lo.n * l.mixer.lo.k + l.mixer.ro.n * l.mixer.ro.k if l.mixer.combines else
+                l.mixer.o.n * l.mixer.o.k + l.mixer.a2.n * l.mixer.a2.k + l.mixer.g2.n * l.mixer.g2.k for l in model.layers),
+            "window_attn_prefill": n_par * seen * h * 2 * 256}
+    for name, fl in flop.items():
+        dt, calls = log.time(torch, name, 10)
+        kernels["prefill " + name] = {"us": round(1e6 * dt / len(calls), 1), "TFLOP/s": round(fl / dt / 1e12, 1), "frac": round(fl / dt / 1e12 / burst, 3)}
+    # the recurrences: bytes of their operands, each read or written once
+    io = {"mlstm": n_par * chunk * rh * 128 * 4 * 4, "delta_scan": n_par * chunk * (h // 2 * 2 + h * 3) * 128 * 4,
+          "delta_prep": n_par * chunk * (h // 2 * 2 + h) * 128 * 8, "delta_decay": n_par * chunk * h * 128 * 8, "gated_heads": chunk * 10 * 128 * n_par * (rh + h),
+          "pre_norm": chunk * w * 4 * (n_par * (1 + 0.5 + 4 + 0.5) + n_par * (1 + 0.5 + 1 + 0.5)), "window_attn_append": n_par * chunk * (h + 2 * g) * 128 * 6}
+    for name, nbytes in io.items():
+        dt, calls = log.time(torch, name, 10)
+        kernels["prefill " + name] = {"us": round(1e6 * dt / len(calls), 1), "GB/s": round(nbytes / dt / 1e9), "frac": round(nbytes / dt / 1e9 / hbm, 3)}
+    return kernels
+
+
 def bench_fomatar(hq, oracle, torch, ctx, dev, args) -> dict:
     """The Fomatar design beside the quantized Llama decoder at equal width, heads, head size, feed-forward and depth:
     prefill and decode throughput, and every kernel alone against its roofline.  Random weights, four layers (0.9 to
@@ -793,78 +862,20 @@ def bench_fomatar(hq, oracle, torch, ctx, dev, args) -> dict:
     sampler.start()
     l0, sizes = ctx.launch_count, {}
 
-    def timed_once(fn):
-        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-        torch.cuda.synchronize()
-        e0.record()
-        fn()
-        e1.record()
-        torch.cuda.synchronize()
-        return e0.elapsed_time(e1) * 1e-3
-
-    def throughput(model):
-        ids = torch.randint(0, vocab, (n_prompt,), dtype=torch.int32, device=dev, generator=torch.Generator(device=dev).manual_seed(0))
-        best = 1e9
-        for _ in range(4):
-            slot = model.open_slot()
-            model.bind(slot)
-            best = min(best, timed_once(lambda: model.extend(slot, ids, [])))
-            model.close_slot(slot)
-        slot = model.open_slot()
-        model.extend(slot, ids, [])
-        model.bind(slot)
-        model.generate(8, collect=False)
-        dt = timed_once(lambda: model.generate(n_new, collect=False))
-        ctx.check_status()
-        assert bool(torch.isfinite(model.logits).all())
-        return {"prefill_tok_s": round(n_prompt / best), "decode_tok_s": round(n_new / dt, 1), "decode_us_per_token": round(1e6 * dt / n_new, 1)}, slot
-
     for size, (w, h, g, rh, ff, window) in FOMATAR_SIZES.items():
         cfg = fomatar_config(size, layers, vocab)
         model = FomatarDecoder(ctx, FomatarConfig(cfg), fomatar_tensors(torch, cfg), max_seq=n_prompt + 1024, prefill_chunk=chunk)
-        ours, slot = throughput(model)
+        ours, slot = _throughput(torch, ctx, dev, model, vocab, n_prompt, n_new)
         per_token = model.decode_bytes_per_token()
         ours["decode_frac_of_hbm_roofline"] = round(per_token / (ours["decode_us_per_token"] * 1e-6) / 1e9 / hbm, 3)
-        kernels = {}
-        # one decode step, kind by kind
-        with _CallLog(model.sop) as log:
-            model.decode_step()
-        n_par = layers // 2
-        st = 2 * 4 * 128 * 128
-        work = {"dense_matvec": sum(r.nbytes for l in model.layers for r in (l.mixer.proj, l.up, l.down)) + model.head.nbytes +
-                sum(l.mixer.lo.nbytes + l.mixer.ro.nbytes if l.mixer.combines else l.mixer.o.nbytes for l in model.layers),
-                "window_attn_decode": n_par * window * g * 256 * 2, "mlstm": n_par * rh * st,
-                "delta_step": n_par * (h * st + model.layers[1].mixer.a2.nbytes + model.layers[1].mixer.g2.nbytes)}
-        for name, nbytes in work.items():
-            dt, calls = log.time(torch, name)
-            kernels["decode " + name] = {"us": round(1e6 * dt / len(calls), 2), "GB/s": round(nbytes / dt / 1e9), "frac": round(nbytes / dt / 1e9 / hbm, 3)}
-        # one portion deep in a prompt
-        ids = torch.randint(0, vocab, (chunk,), dtype=torch.int32, device=dev)
-        model.pos.fill_(n_prompt - chunk)
-        with _CallLog(model.sop) as log:
-            model._portion(ids, chunk)
-        seen = sum(min(window, n_prompt - chunk + i + 1) for i in range(chunk))
-        flop = {"dense_matmul": 2 * chunk * sum(r.n * r.k for l in model.layers for r in (l.mixer.proj, l.up, l.down)) + 2 * chunk * sum(
-                    l.mixer.lo.n * l.mixer.lo.k + l.mixer.ro.n * l.mixer.ro.k if l.mixer.combines else
-                    l.mixer.o.n * l.mixer.o.k + l.mixer.a2.n * l.mixer.a2.k + l.mixer.g2.n * l.mixer.g2.k for l in model.layers),
-                "window_attn_prefill": n_par * seen * h * 2 * 256}
-        for name, fl in flop.items():
-            dt, calls = log.time(torch, name, 10)
-            kernels["prefill " + name] = {"us": round(1e6 * dt / len(calls), 1), "TFLOP/s": round(fl / dt / 1e12, 1), "frac": round(fl / dt / 1e12 / burst, 3)}
-        # the recurrences: bytes of their operands, each read or written once
-        io = {"mlstm": n_par * chunk * rh * 128 * 4 * 4, "delta_scan": n_par * chunk * (h // 2 * 2 + h * 3) * 128 * 4,
-              "delta_prep": n_par * chunk * (h // 2 * 2 + h) * 128 * 8, "delta_decay": n_par * chunk * h * 128 * 8, "gated_heads": chunk * 10 * 128 * n_par * (rh + h),
-              "pre_norm": chunk * w * 4 * (n_par * (1 + 0.5 + 4 + 0.5) + n_par * (1 + 0.5 + 1 + 0.5)), "window_attn_append": n_par * chunk * (h + 2 * g) * 128 * 6}
-        for name, nbytes in io.items():
-            dt, calls = log.time(torch, name, 10)
-            kernels["prefill " + name] = {"us": round(1e6 * dt / len(calls), 1), "GB/s": round(nbytes / dt / 1e9), "frac": round(nbytes / dt / 1e9 / hbm, 3)}
+        kernels = _fomatar_kernels(torch, dev, model, FOMATAR_SIZES[size], vocab, n_prompt, chunk)
         model.close_slot(slot)
-        del model, log
+        del model
         torch.cuda.empty_cache()
 
         lc = D.LlamaConfig(n_layers=layers, hidden=w, n_heads=h, n_kv_heads=g, head_dim=128, ffn=ff, vocab=vocab, max_seq=n_prompt + 1024)
         llama = D.LlamaDecoder(ctx, lc, build_llama_weights(hq, oracle, torch, ctx, dev, lc), prefill_chunk=chunk)
-        theirs, slot = throughput(llama)
+        theirs, slot = _throughput(torch, ctx, dev, llama, vocab, n_prompt, n_new)
         theirs["decode_frac_of_hbm_roofline"] = round((llama.weight_bytes_per_token() + llama.kv_bytes_per_position() * n_prompt) /
                                                       (theirs["decode_us_per_token"] * 1e-6) / 1e9 / hbm, 3)
         like = {}
@@ -928,6 +939,127 @@ def bench_fomatar(hq, oracle, torch, ctx, dev, args) -> dict:
             "gpu_launches": int(ctx.launch_count - l0), "clocks": sampler.stop()}
 
 
+RUNOPEL_SIZES = {        # width, attention heads, state-space heads (64 wide) and groups, feed-forward, window, expert feed-forward
+    "2048": (2048, 16, 64, 4, 6144, 2048, 768),
+    "4096": (4096, 32, 128, 8, 14336, 4096, 1792),
+}
+RUNOPEL_EXPERTS, RUNOPEL_TOP = 32, 4
+
+
+def runopel_config(size: str, layers: int, vocab: int) -> dict:
+    """Layers of a real model's proportions: latent attention and state-space mixers, dense and routed feed-forwards, four streams."""
+    w, h, sh, groups, ff, window, eff = RUNOPEL_SIZES[size]
+    lat = {"type": "latent_attention", "mixer": {"heads": h, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "mask": {"size": window},
+                                                 "rot": {"base": 10000.0, "dims": 64}, "scale": 192 ** -0.5}}
+    ssm = {"type": "mamba2", "mixer": {"heads": sh, "vdim": 64, "state": 128, "groups": groups, "norm_groups": groups, "conv": 4}}
+    dense, moe = {"kind": "dense", "ff": ff, "limit": 7.0}, {"kind": "moe", "router": {"experts": RUNOPEL_EXPERTS, "top": RUNOPEL_TOP}, "expert": {"ff": eff}}
+    order = [(lat, dense), (ssm, moe), (ssm, dense), (lat, moe)]
+    return {"architecture": "Runopel", "width": w, "vocab": vocab, "streams": 4, "residual_mult": 0.5, "logit_scale": 1.0, "norm": {"eps": 1e-5},
+            "layers": [{**order[i % 4][0], "mlp": order[i % 4][1]} for i in range(layers)]}
+
+
+def runopel_tensors(torch, cfg):
+    """get(name) drawing each tensor when it is asked for (bf16 N(0, 1/sqrt(k)); norms one; decays moderate)."""
+    from tests.runopel_util import shapes as shapes_of
+    shapes = shapes_of(cfg)
+    g = torch.Generator(device="cuda").manual_seed(0)
+
+    def get(name):
+        s, leaf = shapes[name], name.rsplit(".", 1)[-1]
+        if leaf == "mix":
+            t = torch.eye(s[0])
+        elif len(s) == 1:
+            t = torch.full(s, -2.0 if leaf in ("A_log", "dt_bias") else 0.5 if leaf in ("in", "b", "D") else 1.0)
+        else:
+            t = torch.randn(s, generator=g, device="cuda") * (1.0 if leaf == "embed" else s[-1] ** -0.5)
+        return t.to(torch.bfloat16).cpu()
+    return get
+
+
+def bench_runopel(hq, oracle, torch, ctx, dev, args) -> dict:
+    """The Runopel design beside the Fomatar decoder (bf16 weights as well) at equal width, attention heads, dense feed-forward,
+    window and depth: prefill and decode throughput, and every kernel alone against its roofline beside the like kernel.
+    Random weights, four layers, 8192-token prompts in portions of 2048."""
+    from hf2q_b200.fomatar import FomatarConfig, FomatarDecoder
+    from hf2q_b200.runopel import RunopelConfig, RunopelDecoder
+    hbm, kind = measured_hbm_peak()
+    _, burst, _ = measured_tensor_peaks()
+    layers, vocab, n_prompt, n_new, chunk = 4, 32768, (args.tokens or 8192), 100, 2048
+    sampler = ClockSampler(ctx.device)
+    sampler.start()
+    l0, sizes = ctx.launch_count, {}
+    for size, (w, h, sh, groups, ff, window, eff) in RUNOPEL_SIZES.items():
+        model = RunopelDecoder(ctx, RunopelConfig(runopel_config(size, layers, vocab)), runopel_tensors(torch, runopel_config(size, layers, vocab)),
+                               max_seq=n_prompt + 1024, prefill_chunk=chunk)
+        ours, slot = _throughput(torch, ctx, dev, model, vocab, n_prompt, n_new)
+        ours["decode_frac_of_hbm_roofline"] = round(model.decode_bytes_per_token() / (ours["decode_us_per_token"] * 1e-6) / 1e9 / hbm, 3)
+        S, E, top = model.cfg.streams, RUNOPEL_EXPERTS, RUNOPEL_TOP
+        kernels, mix, ffs = {}, [l.mixer for l in model.layers], [l.ff for l in model.layers]
+        lat, ssm = [m for m in mix if hasattr(m, "uk_t")], [m for m in mix if hasattr(m, "conv")]
+        dense, moe = [f for f in ffs if hasattr(f, "limit")], [f for f in ffs if hasattr(f, "router")]
+        with _CallLog(model.sop) as log:
+            model.decode_step()
+        used = lambda f, t: t.nbytes * top // E
+        work = {"dense_matvec": sum(m.proj.nbytes + m.o.nbytes for m in mix) + sum(f.gate_up.nbytes + f.down.nbytes for f in dense) +
+                sum(f.router.nbytes for f in moe) + model.head.nbytes,
+                "latent_decode": sum(window * m.row * 2 + m.uk_t.nbytes + m.uv.nbytes for m in lat), "ssd_step": len(ssm) * 2 * sh * 64 * 128 * 4,
+                "expert_glu_step": sum(used(f, f.gate_up) for f in moe), "expert_down_step": sum(used(f, f.down) for f in moe)}
+        for name, nbytes in work.items():
+            dt, calls = log.time(torch, name)
+            kernels["decode " + name] = {"us": round(1e6 * dt / len(calls), 2), "GB/s": round(nbytes / dt / 1e9), "frac": round(nbytes / dt / 1e9 / hbm, 3)}
+        ids = torch.randint(0, vocab, (chunk,), dtype=torch.int32, device=dev)
+        model.pos.fill_(n_prompt - chunk)
+        model._start = n_prompt - chunk
+        with _CallLog(model.sop) as log:
+            model._portion(ids, chunk)
+        model._start = None
+        keys = min(window - 1, n_prompt - chunk) + chunk
+        seen = sum(min(window, n_prompt - chunk + i + 1) for i in range(chunk))
+        inner, chan = sh * 64, sh * 64 + 2 * groups * 128
+        flop = {"dense_matmul": 2 * chunk * (sum(m.proj.n * m.proj.k + m.o.n * m.o.k for m in mix) + sum(f.gate_up.n * f.gate_up.k + f.down.n * f.down.k for f in dense) +
+                                             sum(f.router.n * f.router.k for f in moe)) + 2 * keys * sum(m.ukv.n * m.ukv.k for m in lat),
+                "dense_grouped": 2 * chunk * top * sum((f.gate_up.n * f.gate_up.k + f.down.n * f.down.k) // E for f in moe),
+                "window_attn_prefill": len(lat) * seen * h * 2 * (192 + 128)}
+        for name in [n for n in ("ssd_scan", "ssd_chunks") if any(c[0] == n for c in log.calls)]:
+            flop[name] = len(ssm) * chunk * sh * 4 * 128 * 64
+        for name, fl in flop.items():
+            dt, calls = log.time(torch, name, 10)
+            kernels["prefill " + name] = {"us": round(1e6 * dt / len(calls), 1), "TFLOP/s": round(fl / dt / 1e12, 1), "frac": round(fl / dt / 1e12 / burst, 3)}
+        # operands read or written once
+        n_hyper = sum(1 for c in log.calls if c[0] == "hyper_norm")
+        parts = sum(1 + (top if f in moe else 1) for f in ffs)
+        io = {"hyper_norm": chunk * w * (4 * (2 * S * n_hyper + parts) + 2 * n_hyper), "ssd_prep": len(ssm) * chunk * (8 * chan + 12 * sh),
+              "gated_heads": len(ssm) * chunk * inner * 10, "latent_append": len(lat) * chunk * (h * 192 + 576) * 6, "sort_rows": len(moe) * chunk * w * 2 * (1 + top)}
+        for name in [n for n in ("ssd_scan", "ssd_chunks") if any(c[0] == n for c in log.calls)]:
+            io[name] = len(ssm) * chunk * (4 * (chan + inner) + 8 * sh)
+        for name, nbytes in io.items():
+            dt, calls = log.time(torch, name, 10)
+            k = kernels.setdefault("prefill " + name, {"us": round(1e6 * dt / len(calls), 1)})
+            k |= {"GB/s": round(nbytes / dt / 1e9), "frac_hbm" if "frac" in k else "frac": round(nbytes / dt / 1e9 / hbm, 3)}
+        model.close_slot(slot)
+        del model, log, mix, ffs, lat, ssm, dense, moe
+        torch.cuda.empty_cache()
+
+        fsize = FOMATAR_SIZES[size]
+        cfg = fomatar_config(size, layers, vocab)
+        model = FomatarDecoder(ctx, FomatarConfig(cfg), fomatar_tensors(torch, cfg), max_seq=n_prompt + 1024, prefill_chunk=chunk)
+        theirs, slot = _throughput(torch, ctx, dev, model, vocab, n_prompt, n_new)
+        theirs["decode_frac_of_hbm_roofline"] = round(model.decode_bytes_per_token() / (theirs["decode_us_per_token"] * 1e-6) / 1e9 / hbm, 3)
+        sizes[size] = {"runopel": ours, "fomatar": theirs, "runopel_kernels": kernels,
+                       "fomatar_kernels": _fomatar_kernels(torch, dev, model, fsize, vocab, n_prompt, chunk)}
+        model.close_slot(slot)
+        del model
+        torch.cuda.empty_cache()
+    big = sizes["4096"]["runopel"]
+    return {"metric": "Runopel decode tok/s", "value": big["decode_tok_s"], "unit": "tok/s", "higher_is_better": True, "dtype": "bf16 weights and operands, f32 accumulate and state",
+            "config": {"workload": f"{layers} layers (two latent attention, two Mamba-2; two dense, two routed to {RUNOPEL_TOP} of {RUNOPEL_EXPERTS} experts), four streams, widths "
+                                   f"{', '.join(RUNOPEL_SIZES)}, vocab {vocab}; prefill of {n_prompt} tokens in portions of {chunk}, then {n_new} greedy tokens from one CUDA "
+                                   "graph; beside the Fomatar decoder at equal width, attention heads, dense feed-forward, window and depth",
+                       "timing": "CUDA events; kernels alone from a CUDA graph of their calls over all layers (weights larger than L2)"},
+            "sizes": sizes, "roofline": {"hbm_gbs": hbm, "bf16_tflops_burst": burst, "peak_source": f"of {kind}"},
+            "gpu_launches": int(ctx.launch_count - l0), "clocks": sampler.stop()}
+
+
 def run_secondary(args) -> None:
     """One of the other workloads alone on one GPU: one JSON line."""
     import torch
@@ -949,6 +1081,8 @@ def run_secondary(args) -> None:
         line = bench_decode(hq, oracle, torch, ctx, dev, args)
     elif args.workload == "fomatar":
         line = bench_fomatar(hq, oracle, torch, ctx, dev, args)
+    elif args.workload == "runopel":
+        line = bench_runopel(hq, oracle, torch, ctx, dev, args)
     elif args.workload == "attention":
         line = bench_attention(hq, oracle, torch, ctx, dev, args)
     else:
@@ -974,10 +1108,11 @@ def main() -> None:
     ap.add_argument("--no-strong", action="store_true", help="several GPUs: skip the strong-scaling leg")
     ap.add_argument("--no-graph", action="store_true", help="issue launches eagerly instead of replaying a CUDA graph")
     ap.add_argument("--qtype", default="", help="matvec: one ggml type number (2, 8, 12, 13, 14) instead of all five")
-    ap.add_argument("--workload", default="gemv", choices=["gemv", "gemm", "moe", "matvec", "config1", "decode", "attention", "fomatar"],
+    ap.add_argument("--workload", default="gemv", choices=["gemv", "gemm", "moe", "matvec", "config1", "decode", "attention", "fomatar", "runopel"],
                     help="gemv: the headline Q6_K decode sweep (default, carries the others as `secondary`); gemm: Q4_K_M prefill "
                          "GEMM sweep; moe: Qwen3-style A3B expert layer (Q5_K mul_mat_id); matvec: all block formats; config1: Q4_K 4096^2 f32; "
-                         "fomatar: the bf16 design with recurrent mixers beside the quantized decoder at equal size")
+                         "fomatar: the bf16 design with recurrent mixers beside the quantized decoder at equal size; "
+                         "runopel: the multi-stream design with latent attention, state-space mixers and routed experts beside that one")
     ap.add_argument("--tokens", type=int, default=0, help="gemm/moe: one token count instead of the sweep")
     args = ap.parse_args()
     if args.warmup < 3:

@@ -77,7 +77,7 @@ struct MatvecSegs {
 };
 
 // One-row product: the CTA's weight rows run through a MatvecStream; the layer's row prologue fills x in front of it.
-template <int PRO>
+template <int PRO, bool PAIRS>
 __global__ void __launch_bounds__(MR_THREADS) dense_matvec_kernel(const __grid_constant__ MatvecSegs p, uint32_t* status) {
     extern __shared__ __align__(128) uint8_t mv_smem[];                 // ring, then x [k] f32
     __shared__ float red[64];
@@ -88,9 +88,9 @@ __global__ void __launch_bounds__(MR_THREADS) dense_matvec_kernel(const __grid_c
     const uint32_t blk = blockIdx.x - (second ? p.blocks0 : 0u), n_blk = second ? gridDim.x - p.blocks0 : p.blocks0;
     const uint32_t warp = threadIdx.x >> 5;
     float* xs = reinterpret_cast<float*>(mv_smem + MR_RING);
-    const bool pairs = epi_pairs(s.epilogue);
     // rows [row0, row1) of this CTA, spread evenly
-    const uint32_t unit = pairs ? 2 : 1, units = s.n / unit;
+    constexpr uint32_t unit = PAIRS ? 2 : 1;
+    const uint32_t units = s.n / unit;
     const uint32_t row0 = unit * static_cast<uint32_t>(static_cast<uint64_t>(units) * blk / n_blk), row1 = unit * static_cast<uint32_t>(static_cast<uint64_t>(units) * (blk + 1) / n_blk);
     const uint32_t per_row = (s.k + MV_CHUNK - 1) / MV_CHUNK;
     const __nv_bfloat16* w = static_cast<const __nv_bfloat16*>(s.w) + static_cast<size_t>(row0) * s.k;
@@ -141,14 +141,21 @@ __global__ void __launch_bounds__(MR_THREADS) dense_matvec_kernel(const __grid_c
         else gated_heads_row<float>(s.gated, 0, xs, warp, MR_WARPS);
     }
     __syncthreads();
-    stream.run(chunk, xs, row1 - row0, per_row, unit, [&](uint32_t r, float v0, float v1) {
-        const uint32_t row = row0 + r;
-        if (s.bias) { v0 += s.bias[row]; if (pairs) v1 += s.bias[row + 1]; }
-        if (pairs) { s.y[row / 2] = glu_value(v0, v1, s.epilogue, s.cap); return; }
-        float v = epilogue_value(v0, s.epilogue, s.cap);
-        if (s.epilogue == HF2Q_EPI_ADD) v += s.residual[row];
-        s.y[row] = v;
-    });
+    if constexpr (PAIRS) {
+        stream.run<true>(chunk, xs, row1 - row0, per_row, [&](uint32_t r, float gate, float up) {
+            const uint32_t row = row0 + r;
+            if (s.bias) { gate += s.bias[row]; up += s.bias[row + 1]; }
+            s.y[row / 2] = glu_value(gate, up, s.epilogue, s.cap);
+        });
+    } else {
+        stream.run<false>(chunk, xs, row1 - row0, per_row, [&](uint32_t r, float v, float) {
+            const uint32_t row = row0 + r;
+            if (s.bias) v += s.bias[row];
+            v = epilogue_value(v, s.epilogue, s.cap);
+            if (s.epilogue == HF2Q_EPI_ADD) v += s.residual[row];
+            s.y[row] = v;
+        });
+    }
 }
 
 struct DenseArgs {
@@ -560,11 +567,15 @@ cudaError_t dense_any(const DenseArgs& a, int sms, uint32_t* status, cudaStream_
     return launch_pdl(dense_gemm_f32_kernel<X, Y, false>, dim3((a.n + FT - 1) / FT, (a.m + FT - 1) / FT), dim3(256), 0, st, a);
 }
 
+template <int PRO, bool PAIRS>
+cudaError_t launch_fused_as(const MatvecSegs& p, uint32_t blocks, size_t smem, uint32_t* status, cudaStream_t st) {
+    static PerDeviceFlag flag;
+    if (const cudaError_t e = ensure_max_dynamic_smem(dense_matvec_kernel<PRO, PAIRS>, MR_MAX_SMEM, flag); e != cudaSuccess) return e;
+    return launch_pdl(dense_matvec_kernel<PRO, PAIRS>, dim3(blocks), dim3(MR_THREADS), smem, st, p, status);
+}
 template <int PRO>
 cudaError_t launch_fused(const MatvecSegs& p, uint32_t blocks, size_t smem, uint32_t* status, cudaStream_t st) {
-    static PerDeviceFlag flag;
-    if (const cudaError_t e = ensure_max_dynamic_smem(dense_matvec_kernel<PRO>, MR_MAX_SMEM, flag); e != cudaSuccess) return e;
-    return launch_pdl(dense_matvec_kernel<PRO>, dim3(blocks), dim3(MR_THREADS), smem, st, p, status);
+    return epi_pairs(p.s[0].epilogue) ? launch_fused_as<PRO, true>(p, blocks, smem, status, st) : launch_fused_as<PRO, false>(p, blocks, smem, status, st);
 }
 
 }  // namespace
@@ -631,7 +642,7 @@ HF2Q_API int32_t hf2q_cuda_dense_matvec(hf2q_ctx* ctx, void* stream, uint32_t pr
             (prologue == HF2Q_PRO_NORM && (!s.pre.x || !s.pre.norm || s.pre.width > s.k || !pre_norm_aligned(s.pre) || (s.pre.a && (!s.pre.b || !s.pre.a_norm || !s.pre.b_norm)) || (s.pre.shift && (!s.pre.shift_state || !s.pre.pos)))) ||
             (prologue == HF2Q_PRO_GATED && (!gated_ok(s.gated) || s.gated.heads * s.gated.head_dim > s.k)) ||
             (prologue == HF2Q_PRO_HYPER && (!hyper_ok(s.hyper) || s.hyper.width > s.k || s.hyper.x_out == s.hyper.x)) || s.epilogue > HF2Q_EPI_CLAMP_GLU ||
-            (s.epilogue == HF2Q_EPI_ADD && !s.residual) || (epi_needs_cap(s.epilogue) && !(s.cap > 0.f)) || (epi_pairs(s.epilogue) && s.n % 2))
+            (s.epilogue == HF2Q_EPI_ADD && !s.residual) || (epi_needs_cap(s.epilogue) && !(s.cap > 0.f)) || (epi_pairs(s.epilogue) && s.n % 2) || epi_pairs(s.epilogue) != epi_pairs(segs[0].epilogue))
             return ctx_fail(ctx, HF2Q_ERR_INVALID_ARGUMENT, "dense_matvec: bad segment");
         p.s[i] = s;
         chunks[i] = static_cast<uint64_t>(s.n) * ((s.k + MV_CHUNK - 1) / MV_CHUNK);

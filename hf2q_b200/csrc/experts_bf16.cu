@@ -59,7 +59,7 @@ __global__ void __launch_bounds__(MR_THREADS) expert_glu_kernel(const __grid_con
     if (blockIdx.x == 0)
         for (uint32_t i = threadIdx.x; i < e.top; i += MR_THREADS) e.ids[i] = ids[i];
     __syncthreads();
-    stream.run(chunk, xs, row1 - row0, per_row, 2, [&](uint32_t r, float g, float u) {
+    stream.run<true>(chunk, xs, row1 - row0, per_row, [&](uint32_t r, float g, float u) {
         const uint32_t row = row0 + r;
         const float s = scores[row / (2 * e.ff)];
         e.act[row / 2] = siluf(s * g) * (s * u);
@@ -87,7 +87,7 @@ __global__ void __launch_bounds__(MR_THREADS) expert_down_kernel(const __grid_co
     float* xs = reinterpret_cast<float*>(mv_smem + MR_RING);
     for (uint32_t i = threadIdx.x; i < e.top * e.ff; i += MR_THREADS) xs[i] = e.act[i];
     __syncthreads();
-    stream.run(chunk, xs, row1 - row0, per_row, 1, [&](uint32_t r, float v, float) { e.y[row0 + r] = v; });
+    stream.run<false>(chunk, xs, row1 - row0, per_row, [&](uint32_t r, float v, float) { e.y[row0 + r] = v; });
 }
 
 constexpr uint32_t STEP_SMEM = 200 * 1024;                              // (the choice needs some static shared memory as well)

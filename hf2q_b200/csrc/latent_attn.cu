@@ -4,9 +4,11 @@
 //   append   prefill: latents and rotated key parts to the cache, rotated queries to a buffer; the caller expands the
 //            window's latents to keys and values with a product and runs the windowed prefill over them
 //   decode   three launches: the query moves into the latent space (q . uk c = (uk^T q) . c), attention over the cached
-//            rows with all heads sharing a tile of them, then the merge of the splits and the heads' value matrices
+//            rows with all heads sharing a tile of them (bf16: on the tensor cores; f32: in f32), then the merge of the
+//            splits and the heads' value matrices
 #include <math_constants.h>
 
+#include "mma_sync.cuh"
 #include "seq_common.cuh"
 
 namespace hf2q {
@@ -66,8 +68,14 @@ template <typename T>
 __global__ void __launch_bounds__(256) latent_query_kernel(const __grid_constant__ hf2q_latent_attn a, uint32_t slices, float* __restrict__ qa) {
     __shared__ __align__(16) float q[LD_DIM];
     pdl_trigger();
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    if (blockIdx.x < a.heads * slices) {                                    // weights: towards L2 before the wait
+        const uint32_t r0 = blockIdx.x % slices * LQ_ROWS, rows = min(LQ_ROWS, a.kv_rank - min(r0, a.kv_rank)), line = pad8(a.dim) * 2;
+        const char* w = static_cast<const char*>(a.uk_t) + (static_cast<size_t>(blockIdx.x / slices) * a.kv_rank + r0) * line;
+        for (uint32_t i = 128 * threadIdx.x; i < rows * line; i += 128 * 256) prefetch_l2(w + i);
+    }
     pdl_wait();
-    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, pos = *a.pos;
+    const uint32_t pos = *a.pos;
     if (blockIdx.x == a.heads * slices) {
         if (warp == 0) append_row<T>(a, a.proj + a.c_off, pos);
         return;
@@ -106,12 +114,12 @@ __host__ __device__ inline uint32_t part_elems(const hf2q_latent_attn& a) { retu
 // grid (groups of 8 NH heads, splits); a warp owns NH heads, a tile of 32 keys is shared by the CTA (lane = key for the
 // scores, lane = latent elements 2 lane + 64 c for the sums).  part [split][head][max, sum, 2 pad, acc]
 template <typename T, int NH, int NC>
-__global__ void __launch_bounds__(LD_WARPS * 32) latent_decode_kernel(const __grid_constant__ hf2q_latent_attn a, const float* __restrict__ qa,
-                                                                      float* __restrict__ part) {
+__global__ void __launch_bounds__(LD_WARPS * 32) latent_decode_kernel(const __grid_constant__ hf2q_latent_attn a, uint32_t bufs,
+                                                                      const float* __restrict__ qa, float* __restrict__ part) {
     extern __shared__ __align__(16) uint8_t lsm[];
     const uint32_t rp = pad8(a.kv_rank), row = row_elems(a), pitch = row + 16 / sizeof(T);
     float* qs = reinterpret_cast<float*>(lsm);                             // [8 NH][row]
-    T* tile = reinterpret_cast<T*>(qs + LD_WARPS * NH * row);              // [2][32][pitch]
+    T* tile = reinterpret_cast<T*>(qs + LD_WARPS * NH * row);              // [bufs][32][pitch]
     __shared__ float ps[LD_WARPS][NH][LD_KEYS];
     pdl_trigger();
     pdl_wait();
@@ -140,8 +148,9 @@ __global__ void __launch_bounds__(LD_WARPS * 32) latent_decode_kernel(const __gr
 #pragma unroll
         for (int c = 0; c < NC; ++c) acc[g][c][0] = acc[g][c][1] = 0.f;
     }
-    for (uint32_t p0 = lo, b = 0; p0 < hi; p0 += LD_KEYS, b ^= 1) {
-        if (p0 + LD_KEYS < hi) { stage(p0 + LD_KEYS, b ^ 1); cp_async_wait<1>(); }
+    for (uint32_t p0 = lo, b = 0; p0 < hi; p0 += LD_KEYS) {
+        const bool ahead = bufs == 2 && p0 + LD_KEYS < hi;
+        if (ahead) { stage(p0 + LD_KEYS, b ^ 1); cp_async_wait<1>(); }
         else cp_async_wait<0>();
         __syncthreads();
         const uint32_t cnt = min(LD_KEYS, hi - p0);
@@ -194,6 +203,8 @@ __global__ void __launch_bounds__(LD_WARPS * 32) latent_decode_kernel(const __gr
             }
         }
         __syncthreads();
+        if (bufs == 2) b ^= 1;
+        else if (p0 + LD_KEYS < hi) stage(p0 + LD_KEYS, 0);
     }
 #pragma unroll
     for (int g = 0; g < NH; ++g) {
@@ -208,6 +219,142 @@ __global__ void __launch_bounds__(LD_WARPS * 32) latent_decode_kernel(const __gr
     }
 }
 
+// bf16 cache: grid (groups of 16 MT heads, splits); tiles of 64 keys.  Scores: a warp takes 8 keys of the tile for all heads;
+// sums: a warp takes 8 NT latent elements for all heads.  kv_rank <= 64 NT.
+constexpr uint32_t LT_KEYS = 64, LT_SP = LT_KEYS + 4, LT_PP = LT_KEYS + 8;
+__host__ __device__ inline uint32_t tile_pitch(const hf2q_latent_attn& a) { return ((row_elems(a) + 31) & ~31u) + 8; }
+
+template <int MT, int NT>
+__global__ void __launch_bounds__(LD_WARPS * 32) latent_decode_mma_kernel(const __grid_constant__ hf2q_latent_attn a, const float* __restrict__ qa,
+                                                                          float* __restrict__ part) {
+    extern __shared__ __align__(16) uint8_t lsm[];
+    constexpr uint32_t HG = 16 * MT;
+    const uint32_t rp = pad8(a.kv_rank), row = row_elems(a), pitch = tile_pitch(a), ks = (pitch - 8) / 32;
+    __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(lsm);             // [HG][pitch]
+    __nv_bfloat16* tile = qs + HG * pitch;                                 // [2][64][pitch]
+    float* sc = reinterpret_cast<float*>(tile + 2 * LT_KEYS * pitch);      // [HG][LT_SP]
+    __nv_bfloat16* ps = reinterpret_cast<__nv_bfloat16*>(sc + HG * LT_SP); // [HG][LT_PP]
+    __shared__ float corr[HG];
+    pdl_trigger();
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, t4 = lane & 3, split = blockIdx.y, nsplit = gridDim.y;
+    const uint32_t h_cta = blockIdx.x * HG;
+    // keys never loaded and the padding behind a row must be finite
+    for (uint32_t i = threadIdx.x; i < 2 * LT_KEYS * pitch / 8; i += LD_WARPS * 32) reinterpret_cast<uint4*>(tile)[i] = make_uint4(0, 0, 0, 0);
+    __syncthreads();
+    pdl_wait();
+    const uint32_t pos = *a.pos, n = min(pos + 1, a.window), first = pos + 1 - n;
+    const uint32_t chunk = ((n + nsplit - 1) / nsplit + LT_KEYS - 1) / LT_KEYS * LT_KEYS;
+    const uint32_t lo = first + min(split * chunk, n), hi = first + min(split * chunk + chunk, n);
+    const __nv_bfloat16* cache = static_cast<const __nv_bfloat16*>(a.cache);
+    auto stage = [&](uint32_t p0, uint32_t b) {
+        const uint32_t per = row / 8, cnt = min(LT_KEYS, hi - p0);
+        for (uint32_t i = threadIdx.x; i < cnt * per; i += LD_WARPS * 32)
+            cp_async16(tile + (b * LT_KEYS + i / per) * pitch + i % per * 8, cache + static_cast<size_t>((p0 + i / per) % a.capacity) * row + i % per * 8);
+        cp_async_commit();
+    };
+    if (lo < hi) stage(lo, 0);
+    for (uint32_t i = threadIdx.x; i < HG * (pitch / 2); i += LD_WARPS * 32) {
+        const uint32_t g = i / (pitch / 2), c = 2 * (i % (pitch / 2)), h = h_cta + g;
+        const float2 v = h < a.heads && c < row ? *reinterpret_cast<const float2*>(qa + static_cast<size_t>(h) * row + c) : make_float2(0.f, 0.f);
+        reinterpret_cast<uint32_t*>(qs)[i] = pack_bf16(v.x, v.y);
+    }
+    constexpr int HW = HG / LD_WARPS;                                      // heads whose softmax this warp keeps
+    float mx[HW], l[HW], o[MT][NT][4];
+#pragma unroll
+    for (int g = 0; g < HW; ++g) { mx[g] = -CUDART_INF_F; l[g] = 0.f; }
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int c = 0; c < NT; ++c) o[m][c][0] = o[m][c][1] = o[m][c][2] = o[m][c][3] = 0.f;
+    const uint32_t col0 = warp * 8 * NT;
+    for (uint32_t p0 = lo, b = 0; p0 < hi; p0 += LT_KEYS, b ^= 1) {
+        if (p0 + LT_KEYS < hi) { stage(p0 + LT_KEYS, b ^ 1); cp_async_wait<1>(); }
+        else cp_async_wait<0>();
+        __syncthreads();
+        const uint32_t cnt = min(LT_KEYS, hi - p0), ts = smem_u32(tile + b * LT_KEYS * pitch);
+        float s[MT][4];
+#pragma unroll
+        for (int m = 0; m < MT; ++m) s[m][0] = s[m][1] = s[m][2] = s[m][3] = 0.f;
+        const uint32_t kaddr = ts + ((warp * 8 + (lane & 7)) * pitch + (lane >> 3) * 8) * 2;
+        const uint32_t qaddr = smem_u32(qs) + ((lane & 15) * pitch + (lane >> 4) * 8) * 2;
+#pragma unroll 3
+        for (uint32_t k = 0; k < ks; ++k) {                                // 32 elements of the rows per step
+            uint32_t f[4];
+            ldmatrix4(f, kaddr + 64 * k);
+#pragma unroll
+            for (int m = 0; m < MT; ++m) {
+                uint32_t q0[4], q1[4];
+                ldmatrix4(q0, qaddr + (16 * m * pitch) * 2 + 64 * k);
+                ldmatrix4(q1, qaddr + (16 * m * pitch) * 2 + 64 * k + 32);
+                mma_bf16(s[m], q0, f[0], f[1]);
+                mma_bf16(s[m], q1, f[2], f[3]);
+            }
+        }
+#pragma unroll
+        for (int m = 0; m < MT; ++m)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const uint32_t key = warp * 8 + 2 * t4 + (i & 1);
+                sc[(16 * m + gid + 8 * (i >> 1)) * LT_SP + key] = key < cnt ? s[m][i] * a.scale : -CUDART_INF_F;
+            }
+        __syncthreads();
+#pragma unroll
+        for (int g = 0; g < HW; ++g) {
+            const uint32_t h = warp * HW + g;
+            const float s0 = sc[h * LT_SP + lane], s1 = sc[h * LT_SP + 32 + lane];
+            float bm = fmaxf(s0, s1);
+#pragma unroll
+            for (int d = 16; d > 0; d >>= 1) bm = fmaxf(bm, __shfl_xor_sync(0xffffffffu, bm, d));
+            const float nm = fmaxf(mx[g], bm), c = expf(mx[g] - nm), e0 = expf(s0 - nm), e1 = expf(s1 - nm);      // (key p0 is always seen: nm is finite)
+            l[g] = l[g] * c + warp_sum(e0 + e1);
+            mx[g] = nm;
+            ps[h * LT_PP + lane] = __float2bfloat16_rn(e0);
+            ps[h * LT_PP + 32 + lane] = __float2bfloat16_rn(e1);
+            if (lane == 0) corr[h] = c;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int m = 0; m < MT; ++m) {
+            const float c0 = corr[16 * m + gid], c1 = corr[16 * m + gid + 8];
+#pragma unroll
+            for (int c = 0; c < NT; ++c) { o[m][c][0] *= c0; o[m][c][1] *= c0; o[m][c][2] *= c1; o[m][c][3] *= c1; }
+        }
+#pragma unroll
+        for (int k = 0; k < static_cast<int>(LT_KEYS) / 16; ++k) {
+            uint32_t pa[MT][4];
+#pragma unroll
+            for (int m = 0; m < MT; ++m) ldmatrix4(pa[m], smem_u32(ps) + ((16 * m + (lane & 15)) * LT_PP + 16 * k + (lane >> 4) * 8) * 2);
+#pragma unroll
+            for (int c = 0; c < NT; c += 2) {
+                if (col0 + 8 * c >= rp) continue;
+                uint32_t f[4];
+                ldmatrix4_trans(f, ts + ((16 * k + ((lane >> 3) & 1) * 8 + (lane & 7)) * pitch + col0 + 8 * c + (lane >> 4) * 8) * 2);
+#pragma unroll
+                for (int m = 0; m < MT; ++m) {
+                    mma_bf16(o[m][c], pa[m], f[0], f[1]);
+                    mma_bf16(o[m][c + 1], pa[m], f[2], f[3]);
+                }
+            }
+        }
+        __syncthreads();
+    }
+    float* dst = part + (static_cast<size_t>(split) * a.heads + h_cta) * part_elems(a);
+#pragma unroll
+    for (int g = 0; g < HW; ++g) {
+        const uint32_t h = warp * HW + g;
+        if (lane == 0 && h_cta + h < a.heads) { dst[h * part_elems(a)] = mx[g]; dst[h * part_elems(a) + 1] = l[g]; }
+    }
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int c = 0; c < NT; ++c)
+#pragma unroll
+            for (int u = 0; u < 2; ++u) {
+                const uint32_t h = 16 * m + gid + 8 * u, d = col0 + 8 * c + 2 * t4;
+                if (h_cta + h < a.heads && d < rp) *reinterpret_cast<float2*>(dst + h * part_elems(a) + 4 + d) = make_float2(o[m][c][2 * u], o[m][c][2 * u + 1]);
+            }
+}
+
 // grid (heads, slices of the value rows): merge of the splits, then the head's value matrix
 constexpr uint32_t LD_SPLITS = 64, LO_ROWS = 32, LD_RANK = 1024;
 __global__ void __launch_bounds__(256) latent_out_kernel(const __grid_constant__ hf2q_latent_attn a, uint32_t nsplit, const float* __restrict__ part,
@@ -215,6 +362,11 @@ __global__ void __launch_bounds__(256) latent_out_kernel(const __grid_constant__
     __shared__ __align__(16) float o[LD_RANK];
     __shared__ float w[LD_SPLITS];
     pdl_trigger();
+    {
+        const uint32_t v0 = min(blockIdx.y * LO_ROWS, a.vdim), bytes = min(LO_ROWS, a.vdim - v0) * pad8(a.kv_rank) * 2;
+        const char* u = static_cast<const char*>(a.uv) + (static_cast<size_t>(blockIdx.x) * a.vdim + v0) * pad8(a.kv_rank) * 2;
+        for (uint32_t i = 128 * threadIdx.x; i < bytes; i += 128 * 256) prefetch_l2(u + i);
+    }
     pdl_wait();
     const uint32_t h = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, rp = pad8(a.kv_rank);
     const size_t step = static_cast<size_t>(a.heads) * part_elems(a);
@@ -270,9 +422,17 @@ uint32_t elem_bytes(const hf2q_latent_attn& a) { return a.cache_dtype == HF2Q_DT
 uint32_t heads_per_warp(const hf2q_latent_attn& a) {
     return a.heads > 2 * LD_WARPS && a.kv_rank <= 512 && decode_smem(a, 4, elem_bytes(a)) <= LD_SMEM ? 4 : 1;
 }
-uint32_t head_groups(const hf2q_latent_attn& a) { const uint32_t per = LD_WARPS * heads_per_warp(a); return (a.heads + per - 1) / per; }
+size_t mma_smem(const hf2q_latent_attn& a, uint32_t mt) {
+    return 16ull * mt * (tile_pitch(a) * 2 + LT_SP * 4 + LT_PP * 2) + 2ull * LT_KEYS * tile_pitch(a) * 2;
+}
+uint32_t mma_mt(const hf2q_latent_attn& a) { return a.heads > 16 && mma_smem(a, 2) <= LD_SMEM ? 2 : 1; }
+bool on_tensor_cores(const hf2q_latent_attn& a) { return a.cache_dtype == HF2Q_DT_BF16 && a.kv_rank <= 512 && mma_smem(a, 1) <= LD_SMEM; }
+uint32_t head_groups(const hf2q_latent_attn& a) {
+    const uint32_t per = on_tensor_cores(a) ? 16 * mma_mt(a) : LD_WARPS * heads_per_warp(a);
+    return (a.heads + per - 1) / per;
+}
 uint32_t decode_splits(const hf2q_latent_attn& a, int sms) {
-    const uint32_t by_sm = static_cast<uint32_t>(sms) / head_groups(a), by_keys = (a.window + LD_KEYS - 1) / LD_KEYS;
+    const uint32_t keys = on_tensor_cores(a) ? LT_KEYS : LD_KEYS, by_sm = static_cast<uint32_t>(sms) / head_groups(a), by_keys = (a.window + keys - 1) / keys;
     const uint32_t s = by_sm < by_keys ? by_sm : by_keys;
     return s < 1 ? 1 : s > LD_SPLITS ? LD_SPLITS : s;
 }
@@ -282,11 +442,25 @@ template <typename T, int NH, int NC>
 cudaError_t launch_decode(const hf2q_latent_attn& a, const float* qa, float* part, uint32_t splits, cudaStream_t st) {
     static PerDeviceFlag flag;
     if (const cudaError_t e = ensure_max_dynamic_smem(latent_decode_kernel<T, NH, NC>, static_cast<int>(LD_SMEM), flag); e != cudaSuccess) return e;
-    return launch_pdl(latent_decode_kernel<T, NH, NC>, dim3(head_groups(a), splits), dim3(LD_WARPS * 32), decode_smem(a, NH, sizeof(T)), st, a, qa, part);
+    const uint32_t bufs = decode_smem(a, NH, sizeof(T)) <= LD_SMEM ? 2 : 1;
+    const size_t smem = decode_smem(a, NH, sizeof(T)) - (bufs == 1 ? static_cast<size_t>(LD_KEYS) * (row_elems(a) + 16 / sizeof(T)) * sizeof(T) : 0);
+    if (smem > LD_SMEM) return cudaErrorInvalidValue;
+    return launch_pdl(latent_decode_kernel<T, NH, NC>, dim3(head_groups(a), splits), dim3(LD_WARPS * 32), smem, st, a, bufs, qa, part);
+}
+template <int MT>
+cudaError_t launch_decode_mma(const hf2q_latent_attn& a, const float* qa, float* part, uint32_t splits, cudaStream_t st) {
+    auto launch = [&](auto kern, PerDeviceFlag& flag) {
+        if (const cudaError_t e = ensure_max_dynamic_smem(kern, static_cast<int>(LD_SMEM), flag); e != cudaSuccess) return e;
+        return launch_pdl(kern, dim3(head_groups(a), splits), dim3(LD_WARPS * 32), mma_smem(a, MT), st, a, qa, part);
+    };
+    static PerDeviceFlag f2, f4, f8;
+    if (a.kv_rank <= 128) return launch(latent_decode_mma_kernel<MT, 2>, f2);
+    if (a.kv_rank <= 256) return launch(latent_decode_mma_kernel<MT, 4>, f4);
+    return launch(latent_decode_mma_kernel<MT, 8>, f8);
 }
 template <typename T>
 cudaError_t launch_decode_any(const hf2q_latent_attn& a, const float* qa, float* part, uint32_t splits, cudaStream_t st) {
-    if (decode_smem(a, heads_per_warp(a), sizeof(T)) > LD_SMEM) return cudaErrorInvalidValue;
+    if (on_tensor_cores(a)) return mma_mt(a) == 2 ? launch_decode_mma<2>(a, qa, part, splits, st) : launch_decode_mma<1>(a, qa, part, splits, st);
     if (heads_per_warp(a) == 4) {
         if (a.kv_rank <= 128) return launch_decode<T, 4, 2>(a, qa, part, splits, st);
         return launch_decode<T, 4, 8>(a, qa, part, splits, st);

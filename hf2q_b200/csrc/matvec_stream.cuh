@@ -35,9 +35,10 @@ public:
             for (int i = 0; i < MR_STAGES; ++i) issue(i, chunk);
         }
     }
-    // rows of per_row chunks each, finished `unit` (1 or 2) at a time: finish(row, sum, sum of row + 1).  Every thread of
-    // the CTA calls it, after a barrier behind the last write of xs.
-    template <class F, class G> __device__ __forceinline__ void run(F chunk, const float* xs, uint32_t rows, uint32_t per_row, uint32_t unit, G finish) {
+    // rows of per_row chunks each, finished one (or with PAIRS two) at a time: finish(row, sum, sum of row + 1).  Every thread
+    // of the CTA calls it, after a barrier behind the last write of xs.
+    template <bool PAIRS, class F, class G> __device__ __forceinline__ void run(F chunk, const float* xs, uint32_t rows, uint32_t per_row, G finish) {
+        constexpr uint32_t unit = PAIRS ? 2 : 1;
         const uint32_t block_rows = max(unit, MR_PART / per_row / unit * unit);
         bool ok = true;
         uint32_t i = 0;                                                     // this warp's chunk counter
@@ -70,10 +71,11 @@ public:
             }
             __syncthreads();                                                // (the other half of `part` is free: its readers passed this barrier)
             for (uint32_t r = threadIdx.x * unit; r < nr; r += MR_THREADS * unit) {
-                float v[2] = {0.f, 0.f};
-                for (uint32_t u = 0; u < unit; ++u)
-                    for (uint32_t kc = 0; kc < per_row; ++kc) v[u] += sh_.part[pb][(r + u) * per_row + kc];
-                finish(r0 + r, v[0], v[1]);
+                float v = 0.f, w = 0.f;
+                for (uint32_t kc = 0; kc < per_row; ++kc) v += sh_.part[pb][r * per_row + kc];
+                if constexpr (PAIRS)
+                    for (uint32_t kc = 0; kc < per_row; ++kc) w += sh_.part[pb][(r + 1) * per_row + kc];
+                finish(r0 + r, v, w);
             }
         }
     }

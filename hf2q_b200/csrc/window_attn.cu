@@ -8,6 +8,7 @@
 //   decode    one launch: norm, append, window split over CTAs, merge by the CTA that arrives last
 #include <math_constants.h>
 
+#include "mma_sync.cuh"
 #include "seq_common.cuh"
 
 namespace hf2q {
@@ -23,28 +24,36 @@ __device__ __forceinline__ float score_of(float dot, float scale, float r1, floa
     return s;
 }
 
-// where a KV head's keys and values are: rings, or plain rows that start at position `first`
-template <typename T>
+// where a KV head's keys and values are: rings, or with PLAIN rows that start at position `first` and a shared key part
+template <typename T, bool PLAIN>
 struct KeyRows {
     const T *k, *v, *shared;
-    uint32_t k_row, v_row, first, capacity, s_row, s_capacity, dp, sp;      // sp: padded size of the shared part
-    bool linear;
+    uint32_t capacity, dp, sp, k_row, v_row, first, s_row, s_capacity;      // sp: padded size of the shared part
     __device__ __forceinline__ KeyRows(const hf2q_window_attn& a, uint32_t kvh, uint32_t pos0) {
         const uint32_t dvp = pad8(a.vdim);
         dp = pad8(a.dim);
-        sp = pad8(a.shared_dim);
-        linear = a.linear;
         capacity = a.capacity;
-        k_row = linear ? a.row_stride : dp;
-        v_row = linear ? a.row_stride : dvp;
-        first = linear && pos0 + 1 > a.window ? pos0 + 1 - a.window : 0u;
-        k = static_cast<const T*>(a.k_cache) + (linear ? static_cast<size_t>(kvh) * a.k_head_stride : static_cast<size_t>(kvh) * a.capacity * dp);
-        v = static_cast<const T*>(a.v_cache) + (linear ? static_cast<size_t>(kvh) * a.v_head_stride : static_cast<size_t>(kvh) * a.capacity * dvp);
-        shared = static_cast<const T*>(a.k_shared);
-        s_row = a.shared_stride;
-        s_capacity = a.shared_capacity;
+        if constexpr (PLAIN) {
+            sp = pad8(a.shared_dim);
+            k_row = v_row = a.row_stride;
+            first = pos0 + 1 > a.window ? pos0 + 1 - a.window : 0u;
+            k = static_cast<const T*>(a.k_cache) + static_cast<size_t>(kvh) * a.k_head_stride;
+            v = static_cast<const T*>(a.v_cache) + static_cast<size_t>(kvh) * a.v_head_stride;
+            shared = static_cast<const T*>(a.k_shared);
+            s_row = a.shared_stride;
+            s_capacity = a.shared_capacity;
+        } else {
+            sp = 0;
+            k_row = dp;
+            v_row = dvp;
+            k = static_cast<const T*>(a.k_cache) + static_cast<size_t>(kvh) * a.capacity * dp;
+            v = static_cast<const T*>(a.v_cache) + static_cast<size_t>(kvh) * a.capacity * dvp;
+        }
     }
-    __device__ __forceinline__ uint32_t slot(uint32_t p) const { return linear ? p - first : p % capacity; }
+    __device__ __forceinline__ uint32_t slot(uint32_t p) const {
+        if constexpr (PLAIN) return p - first;
+        else return p % capacity;
+    }
     __device__ __forceinline__ const T* key(uint32_t p) const { return k + static_cast<size_t>(slot(p)) * k_row; }
     __device__ __forceinline__ const T* value(uint32_t p) const { return v + static_cast<size_t>(slot(p)) * v_row; }
     __device__ __forceinline__ const T* shared_key(uint32_t p) const { return shared + static_cast<size_t>(p % s_capacity) * s_row; }
@@ -102,7 +111,7 @@ __global__ void __launch_bounds__(256) window_append_kernel(const __grid_constan
 
 // Online softmax of one warp for GR query heads against keys [lo, hi) of KV head g; qs: [GR][dp] f32 in shared
 // memory, ps: [GR][32] of this warp.  Lane = key for the scores, lane = value columns 2 lane + 64 c for the sums.
-template <typename T, int GR, int NC>
+template <typename T, int GR, int NC, bool PLAIN>
 struct WarpAttn {
     float mx[GR], l[GR], acc[GR][NC][2];
     __device__ __forceinline__ void init() {
@@ -114,29 +123,43 @@ struct WarpAttn {
             for (int c = 0; c < NC; ++c) acc[g][c][0] = acc[g][c][1] = 0.f;
         }
     }
-    __device__ __forceinline__ void keys(const hf2q_window_attn& a, const KeyRows<T>& kv, const float* qs, float* ps, const float (&r1)[GR],
+    __device__ __forceinline__ void keys(const hf2q_window_attn& a, const T* kc, const T* vc, const KeyRows<T, PLAIN>* kv, const float* qs, float* ps, const float (&r1)[GR],
                                          const float (&r2)[GR], uint32_t pos, uint32_t p0, uint32_t hi) {
-        const uint32_t lane = threadIdx.x & 31, dq = kv.dp + kv.sp, dvp = pad8(a.vdim);
+        const uint32_t lane = threadIdx.x & 31, dp = pad8(a.dim), dvp = pad8(a.vdim);
+        uint32_t dq = dp;
+        if constexpr (PLAIN) dq += kv->sp;
         const uint32_t p = p0 + lane;
         const bool live = p < hi;
         float s[GR];
 #pragma unroll
         for (int g = 0; g < GR; ++g) s[g] = 0.f;
         if (live) {
-            auto part = [&](const T* kr, uint32_t n, const float* q0) {
+            const T* kr;
+            if constexpr (PLAIN) kr = kv->key(p);
+            else kr = kc + static_cast<size_t>(p % a.capacity) * dp;
 #pragma unroll 4
-                for (uint32_t c = 0; c < n; c += 8) {
+            for (uint32_t c = 0; c < dp; c += 8) {
+                float k[8];
+                load8(kr + c, k);
+#pragma unroll
+                for (int g = 0; g < GR; ++g) {
+                    const float4 x = *reinterpret_cast<const float4*>(qs + g * dq + c), y = *reinterpret_cast<const float4*>(qs + g * dq + c + 4);
+                    s[g] += k[0] * x.x + k[1] * x.y + k[2] * x.z + k[3] * x.w + k[4] * y.x + k[5] * y.y + k[6] * y.z + k[7] * y.w;
+                }
+            }
+            if constexpr (PLAIN) {
+                kr = kv->shared_key(p) - dp;
+#pragma unroll 4
+                for (uint32_t c = dp; c < dq; c += 8) {
                     float k[8];
                     load8(kr + c, k);
 #pragma unroll
                     for (int g = 0; g < GR; ++g) {
-                        const float4 x = *reinterpret_cast<const float4*>(q0 + g * dq + c), y = *reinterpret_cast<const float4*>(q0 + g * dq + c + 4);
+                        const float4 x = *reinterpret_cast<const float4*>(qs + g * dq + c), y = *reinterpret_cast<const float4*>(qs + g * dq + c + 4);
                         s[g] += k[0] * x.x + k[1] * x.y + k[2] * x.z + k[3] * x.w + k[4] * y.x + k[5] * y.y + k[6] * y.z + k[7] * y.w;
                     }
                 }
-            };
-            part(kv.key(p), kv.dp, qs);
-            if (kv.sp) part(kv.shared_key(p), kv.sp, qs + kv.dp);
+            }
         }
 #pragma unroll
         for (int g = 0; g < GR; ++g) {
@@ -155,7 +178,9 @@ struct WarpAttn {
         const uint32_t cnt = min(32u, hi - p0);
 #pragma unroll 4
         for (uint32_t i = 0; i < cnt; ++i) {
-            const T* vr = kv.value(p0 + i);
+            const T* vr;
+            if constexpr (PLAIN) vr = kv->value(p0 + i);
+            else vr = vc + static_cast<size_t>((p0 + i) % a.capacity) * dvp;
 #pragma unroll
             for (int c = 0; c < NC; ++c) {
                 const uint32_t d = 2 * lane + 64 * c;
@@ -228,10 +253,9 @@ __global__ void __launch_bounds__(WD_WARPS * 32) window_decode_kernel(const __gr
         r2[g] = a.r1 ? a.r2[h0 + min(static_cast<uint32_t>(g), n_g - 1)] : 0.f;
     }
     __syncthreads();
-    const KeyRows<T> kv(a, kvh, pos);
-    WarpAttn<T, GR, NC> w;
+    WarpAttn<T, GR, NC, false> w;
     w.init();
-    for (uint32_t p0 = lo + warp * 32; p0 < hi; p0 += WD_WARPS * 32) w.keys(a, kv, qs, ps + warp * GR * 32, r1, r2, pos, p0, hi);
+    for (uint32_t p0 = lo + warp * 32; p0 < hi; p0 += WD_WARPS * 32) w.keys(a, kc, vc, nullptr, qs, ps + warp * GR * 32, r1, r2, pos, p0, hi);
 #pragma unroll
     for (int g = 0; g < GR; ++g) {
         if (lane == 0) { rm[warp * GR + g] = w.mx[g]; rl[warp * GR + g] = w.l[g]; }
@@ -288,7 +312,7 @@ __global__ void __launch_bounds__(WD_WARPS * 32) window_decode_kernel(const __gr
 constexpr uint32_t QK_MAX = 320;                        // dim and shared_dim together, padded
 
 // ---------------------------------------------------------------- prefill, f32: one warp per (query, head)
-template <typename T, typename OUT, int NC>
+template <typename T, typename OUT, int NC, bool PLAIN>
 __global__ void __launch_bounds__(256) window_prefill_f32_kernel(const __grid_constant__ hf2q_window_attn a, uint32_t m, const T* __restrict__ q,
                                                                  const float* __restrict__ gate, uint32_t ldg, OUT* __restrict__ out, uint32_t ldo) {
     __shared__ __align__(16) float qs[8][QK_MAX];
@@ -297,15 +321,15 @@ __global__ void __launch_bounds__(256) window_prefill_f32_kernel(const __grid_co
     pdl_wait();
     const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, h = blockIdx.y, t = blockIdx.x * 8 + warp;
     if (t >= m) return;
-    const KeyRows<T> kv(a, h / (a.heads / a.kv_heads), *a.pos);
+    const KeyRows<T, PLAIN> kv(a, h / (a.heads / a.kv_heads), *a.pos);
     const uint32_t dq = kv.dp + kv.sp;
     for (uint32_t i = lane; i < dq; i += 32) qs[warp][i] = to_f32(q[(static_cast<size_t>(t) * a.heads + h) * dq + i]);
     __syncwarp();
     const uint32_t pos = *a.pos + t, n = min(pos + 1, a.window), hi = pos + 1;
     const float r1[1] = {a.r1 ? a.r1[h] : 0.f}, r2[1] = {a.r1 ? a.r2[h] : 0.f};
-    WarpAttn<T, 1, NC> w;
+    WarpAttn<T, 1, NC, PLAIN> w;
     w.init();
-    for (uint32_t p0 = hi - n; p0 < hi; p0 += 32) w.keys(a, kv, qs[warp], ps[warp], r1, r2, pos, p0, hi);
+    for (uint32_t p0 = hi - n; p0 < hi; p0 += 32) w.keys(a, kv.k, kv.v, &kv, qs[warp], ps[warp], r1, r2, pos, p0, hi);
 #pragma unroll
     for (int c = 0; c < NC; ++c)
 #pragma unroll
@@ -324,25 +348,9 @@ __global__ void __launch_bounds__(256) window_prefill_f32_kernel(const __grid_co
 // ---------------------------------------------------------------- prefill, bf16 cache, tensor cores
 constexpr int WP_WARPS = 4, WP_Q = 16 * WP_WARPS, WP_K = 64;
 
-__device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ void ldmatrix4(uint32_t (&r)[4], uint32_t addr) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
-}
-__device__ __forceinline__ void ldmatrix4_trans(uint32_t (&r)[4], uint32_t addr) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
-}
-__device__ __forceinline__ uint32_t pack_bf16(float a, float b) {
-    const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
-    return *reinterpret_cast<const uint32_t*>(&h);
-}
-
 // grid (query tiles, heads); DK >= dim + shared_dim, DV >= vdim.  Keys are walked from the first one the tile's first
 // query sees.
-template <int DK, int DV, typename OUT>
+template <int DK, int DV, typename OUT, bool PLAIN>
 __global__ void __launch_bounds__(WP_WARPS * 32) window_prefill_mma_kernel(const __grid_constant__ hf2q_window_attn a, uint32_t m,
                                                                            const __nv_bfloat16* __restrict__ q, const float* __restrict__ gate, uint32_t ldg,
                                                                            OUT* __restrict__ out, uint32_t ldo) {
@@ -353,7 +361,7 @@ __global__ void __launch_bounds__(WP_WARPS * 32) window_prefill_mma_kernel(const
     const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, t4 = lane & 3;
     const uint32_t h = blockIdx.y, t0 = blockIdx.x * WP_Q;
     const uint32_t pos0 = *a.pos;
-    const KeyRows<__nv_bfloat16> rows(a, h / (a.heads / a.kv_heads), pos0);
+    const KeyRows<__nv_bfloat16, PLAIN> rows(a, h / (a.heads / a.kv_heads), pos0);
     const uint32_t dq = rows.dp + rows.sp, dvp = pad8(a.vdim), nk = (dq + 15) / 16, nv = (dvp + 15) / 16;
     const uint32_t q_lo = pos0 + t0, q_hi = pos0 + min(t0 + WP_Q, m) - 1;
     const uint32_t j0 = q_lo + 1 > a.window ? q_lo + 1 - a.window : 0u;
@@ -366,7 +374,7 @@ __global__ void __launch_bounds__(WP_WARPS * 32) window_prefill_mma_kernel(const
         const uint32_t ck = dq / 8, cv = dvp / 8, cd = rows.dp / 8;
         for (uint32_t i = threadIdx.x; i < WP_K * ck; i += WP_WARPS * 32) {
             const uint32_t r = i / ck, c = i % ck;
-            if (key0 + r <= q_hi) cp_async16(ks + r * KP + 8 * c, c < cd ? rows.key(key0 + r) + 8 * c : rows.shared_key(key0 + r) + 8 * (c - cd));
+            if (key0 + r <= q_hi) cp_async16(ks + r * KP + 8 * c, !PLAIN || c < cd ? rows.key(key0 + r) + 8 * c : rows.shared_key(key0 + r) + 8 * (c - cd));
         }
         for (uint32_t i = threadIdx.x; i < WP_K * cv; i += WP_WARPS * 32) {
             const uint32_t r = i / cv, c = i % cv;
@@ -501,7 +509,7 @@ bool window_ok(const hf2q_window_attn* a) {
 }
 // what the prefill takes beyond that: plain rows, a shared part of the keys
 bool window_rows_ok(const hf2q_window_attn* a) {
-    if (!a || (!a->linear && !a->shared_dim)) return window_ok(a);
+    if (!a || !a->linear) return window_ok(a);
     hf2q_window_attn b = *a;
     b.qkv = b.qkv ? b.qkv : static_cast<const float*>(a->k_cache);           // the queries come apart
     b.linear = b.shared_dim = 0;
@@ -545,31 +553,35 @@ cudaError_t launch_decode_gr(const hf2q_window_attn& a, float* out, uint8_t* scr
         default: return launch_decode_nc<T, 8>(a, out, scratch, sms, st);
     }
 }
-template <typename T, typename OUT>
+template <typename T, typename OUT, bool PLAIN>
 cudaError_t launch_prefill_f32(const hf2q_window_attn& a, uint32_t m, const void* q, const float* gate, uint32_t ldg, void* out, uint32_t ldo, cudaStream_t st) {
     const dim3 grid((m + 7) / 8, a.heads);
     const T* qt = static_cast<const T*>(q);
     OUT* o = static_cast<OUT*>(out);
-    if (a.vdim <= 64) return launch_pdl(window_prefill_f32_kernel<T, OUT, 1>, grid, dim3(256), 0, st, a, m, qt, gate, ldg, o, ldo);
-    if (a.vdim <= 128) return launch_pdl(window_prefill_f32_kernel<T, OUT, 2>, grid, dim3(256), 0, st, a, m, qt, gate, ldg, o, ldo);
-    return launch_pdl(window_prefill_f32_kernel<T, OUT, 4>, grid, dim3(256), 0, st, a, m, qt, gate, ldg, o, ldo);
+    if (a.vdim <= 64) return launch_pdl(window_prefill_f32_kernel<T, OUT, 1, PLAIN>, grid, dim3(256), 0, st, a, m, qt, gate, ldg, o, ldo);
+    if (a.vdim <= 128) return launch_pdl(window_prefill_f32_kernel<T, OUT, 2, PLAIN>, grid, dim3(256), 0, st, a, m, qt, gate, ldg, o, ldo);
+    return launch_pdl(window_prefill_f32_kernel<T, OUT, 4, PLAIN>, grid, dim3(256), 0, st, a, m, qt, gate, ldg, o, ldo);
 }
-template <int DK, int DV, typename OUT>
+template <int DK, int DV, typename OUT, bool PLAIN>
 cudaError_t launch_prefill_dm(const hf2q_window_attn& a, uint32_t m, const void* q, const float* gate, uint32_t ldg, void* out, uint32_t ldo, cudaStream_t st) {
     static PerDeviceFlag flag;
     const size_t smem = 2ull * WP_K * (DK + 8 + DV + 8) * 2;
-    if (const cudaError_t e = ensure_max_dynamic_smem(window_prefill_mma_kernel<DK, DV, OUT>, static_cast<int>(smem), flag); e != cudaSuccess) return e;
-    return launch_pdl(window_prefill_mma_kernel<DK, DV, OUT>, dim3((m + WP_Q - 1) / WP_Q, a.heads), dim3(WP_WARPS * 32), smem, st, a, m,
+    if (const cudaError_t e = ensure_max_dynamic_smem(window_prefill_mma_kernel<DK, DV, OUT, PLAIN>, static_cast<int>(smem), flag); e != cudaSuccess) return e;
+    return launch_pdl(window_prefill_mma_kernel<DK, DV, OUT, PLAIN>, dim3((m + WP_Q - 1) / WP_Q, a.heads), dim3(WP_WARPS * 32), smem, st, a, m,
                       static_cast<const __nv_bfloat16*>(q), gate, ldg, static_cast<OUT*>(out), ldo);
 }
 template <typename OUT>
 cudaError_t launch_prefill_mma(const hf2q_window_attn& a, uint32_t m, const void* q, const float* gate, uint32_t ldg, void* out, uint32_t ldo, cudaStream_t st) {
     const uint32_t k = pad8(a.dim) + pad8(a.shared_dim), v = a.vdim;
-    if (k <= 64 && v <= 64) return launch_prefill_dm<64, 64, OUT>(a, m, q, gate, ldg, out, ldo, st);
-    if (k <= 128 && v <= 128) return launch_prefill_dm<128, 128, OUT>(a, m, q, gate, ldg, out, ldo, st);
-    if (k <= 192 && v <= 128) return launch_prefill_dm<192, 128, OUT>(a, m, q, gate, ldg, out, ldo, st);
-    if (k <= 256) return launch_prefill_dm<256, 256, OUT>(a, m, q, gate, ldg, out, ldo, st);
-    return launch_prefill_dm<QK_MAX, 256, OUT>(a, m, q, gate, ldg, out, ldo, st);
+    if (a.linear) {
+        if (k <= 64 && v <= 64) return launch_prefill_dm<64, 64, OUT, true>(a, m, q, gate, ldg, out, ldo, st);
+        if (k <= 128 && v <= 128) return launch_prefill_dm<128, 128, OUT, true>(a, m, q, gate, ldg, out, ldo, st);
+        if (k <= 192 && v <= 128) return launch_prefill_dm<192, 128, OUT, true>(a, m, q, gate, ldg, out, ldo, st);
+        return launch_prefill_dm<QK_MAX, 256, OUT, true>(a, m, q, gate, ldg, out, ldo, st);
+    }
+    if (k <= 64 && v <= 64) return launch_prefill_dm<64, 64, OUT, false>(a, m, q, gate, ldg, out, ldo, st);
+    if (k <= 128 && v <= 128) return launch_prefill_dm<128, 128, OUT, false>(a, m, q, gate, ldg, out, ldo, st);
+    return launch_prefill_dm<256, 256, OUT, false>(a, m, q, gate, ldg, out, ldo, st);
 }
 
 }  // namespace
@@ -623,7 +635,8 @@ HF2Q_API int32_t hf2q_cuda_window_attn_prefill(hf2q_ctx* ctx, void* stream, cons
     const cudaStream_t st = static_cast<cudaStream_t>(stream);
     cudaError_t e = cudaErrorInvalidValue;
     if (a->cache_dtype == HF2Q_DT_F32) {
-        if (out_dtype == HF2Q_DT_F32) e = launch_prefill_f32<float, float>(*a, m, q, gate, ldg, out, ldo, st);
+        if (out_dtype == HF2Q_DT_F32)
+            e = a->linear ? launch_prefill_f32<float, float, true>(*a, m, q, gate, ldg, out, ldo, st) : launch_prefill_f32<float, float, false>(*a, m, q, gate, ldg, out, ldo, st);
     } else if (out_dtype == HF2Q_DT_BF16) {
         e = launch_prefill_mma<__nv_bfloat16>(*a, m, q, gate, ldg, out, ldo, st);
     } else if (out_dtype == HF2Q_DT_F32) {
