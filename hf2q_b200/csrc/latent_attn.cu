@@ -6,6 +6,7 @@
 //   decode   three launches: the query moves into the latent space (q . uk c = (uk^T q) . c), attention over the cached
 //            rows with all heads sharing a tile of them (bf16: on the tensor cores; f32: in f32), then the merge of the
 //            splits and the heads' value matrices
+#include <cooperative_groups.h>
 #include <math_constants.h>
 
 #include "mma_sync.cuh"
@@ -89,22 +90,28 @@ __global__ void __launch_bounds__(256) latent_query_kernel(const __grid_constant
     __syncthreads();
     // lanes in groups of eight share a row
     const uint32_t r_end = min((slice + 1) * LQ_ROWS, rp);
-    for (uint32_t r0 = slice * LQ_ROWS + warp * 4; r0 < r_end; r0 += 32) {
-        const uint32_t r = r0 + (lane >> 3);
-        float s = 0.f;
+    float s[LQ_ROWS / 32];
+#pragma unroll
+    for (uint32_t j = 0; j < LQ_ROWS / 32; ++j) {
+        const uint32_t r = slice * LQ_ROWS + 32 * j + warp * 4 + (lane >> 3);
+        s[j] = 0.f;
         if (r < a.kv_rank) {
             const __nv_bfloat16* w = static_cast<const __nv_bfloat16*>(a.uk_t) + (static_cast<size_t>(h) * a.kv_rank + r) * dp;
-#pragma unroll 4
+#pragma unroll 2
             for (uint32_t c = 8 * (lane & 7); c < dp; c += 64) {
                 float f[8];
                 load8(w + c, f);
 #pragma unroll
-                for (int i = 0; i < 8; ++i) s = fmaf(f[i], q[c + i], s);
+                for (int i = 0; i < 8; ++i) s[j] = fmaf(f[i], q[c + i], s[j]);
             }
         }
+    }
 #pragma unroll
-        for (int o = 4; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
-        if ((lane & 7) == 0 && r < r_end) dst[r] = s;
+    for (uint32_t j = 0; j < LQ_ROWS / 32; ++j) {
+        const uint32_t r = slice * LQ_ROWS + 32 * j + warp * 4 + (lane >> 3);
+#pragma unroll
+        for (int o = 4; o > 0; o >>= 1) s[j] += __shfl_xor_sync(0xffffffffu, s[j], o);
+        if ((lane & 7) == 0 && r < r_end) dst[r] = s[j];
     }
 }
 
@@ -220,27 +227,28 @@ __global__ void __launch_bounds__(LD_WARPS * 32) latent_decode_kernel(const __gr
 }
 
 // bf16 cache: grid (groups of 16 MT heads, splits); tiles of 64 keys.  Scores: a warp takes 8 keys of the tile for all heads;
-// sums: a warp takes 8 NT latent elements for all heads.  kv_rank <= 64 NT.
-constexpr uint32_t LT_KEYS = 64, LT_SP = LT_KEYS + 4, LT_PP = LT_KEYS + 8;
+// sums: a warp takes 8 NT latent elements for all heads.  kv_rank <= 64 NT.  The splits of a cluster merge theirs through
+// distributed shared memory: part [splits / cluster][head][...].
+constexpr uint32_t LT_CLUSTER = 8, LT_KEYS = 64, LT_SP = LT_KEYS + 4, LT_PP = LT_KEYS + 8;
 __host__ __device__ inline uint32_t tile_pitch(const hf2q_latent_attn& a) { return ((row_elems(a) + 31) & ~31u) + 8; }
 
 template <int MT, int NT>
-__global__ void __launch_bounds__(LD_WARPS * 32) latent_decode_mma_kernel(const __grid_constant__ hf2q_latent_attn a, const float* __restrict__ qa,
-                                                                          float* __restrict__ part) {
+__global__ void __launch_bounds__(LD_WARPS * 32) latent_decode_mma_kernel(const __grid_constant__ hf2q_latent_attn a, uint32_t bufs,
+                                                                          const float* __restrict__ qa, float* __restrict__ part) {
     extern __shared__ __align__(16) uint8_t lsm[];
     constexpr uint32_t HG = 16 * MT;
     const uint32_t rp = pad8(a.kv_rank), row = row_elems(a), pitch = tile_pitch(a), ks = (pitch - 8) / 32;
     __nv_bfloat16* qs = reinterpret_cast<__nv_bfloat16*>(lsm);             // [HG][pitch]
-    __nv_bfloat16* tile = qs + HG * pitch;                                 // [2][64][pitch]
-    float* sc = reinterpret_cast<float*>(tile + 2 * LT_KEYS * pitch);      // [HG][LT_SP]
+    __nv_bfloat16* tile = qs + HG * pitch;                                 // [bufs][64][pitch]
+    float* sc = reinterpret_cast<float*>(tile + bufs * LT_KEYS * pitch);   // [HG][LT_SP]
     __nv_bfloat16* ps = reinterpret_cast<__nv_bfloat16*>(sc + HG * LT_SP); // [HG][LT_PP]
-    __shared__ float corr[HG];
+    __shared__ float corr[HG], stats[HG][2], weight[LT_CLUSTER][HG];
     pdl_trigger();
     const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, t4 = lane & 3, split = blockIdx.y, nsplit = gridDim.y;
     const uint32_t h_cta = blockIdx.x * HG;
-    // keys never loaded and the padding behind a row must be finite
-    for (uint32_t i = threadIdx.x; i < 2 * LT_KEYS * pitch / 8; i += LD_WARPS * 32) reinterpret_cast<uint4*>(tile)[i] = make_uint4(0, 0, 0, 0);
-    __syncthreads();
+    // the padding behind a row must be finite
+    const uint32_t pad = (pitch - row) / 8;
+    for (uint32_t i = threadIdx.x; i < bufs * LT_KEYS * pad; i += LD_WARPS * 32) *reinterpret_cast<uint4*>(tile + i / pad * pitch + row + i % pad * 8) = make_uint4(0, 0, 0, 0);
     pdl_wait();
     const uint32_t pos = *a.pos, n = min(pos + 1, a.window), first = pos + 1 - n;
     const uint32_t chunk = ((n + nsplit - 1) / nsplit + LT_KEYS - 1) / LT_KEYS * LT_KEYS;
@@ -250,6 +258,8 @@ __global__ void __launch_bounds__(LD_WARPS * 32) latent_decode_mma_kernel(const 
         const uint32_t per = row / 8, cnt = min(LT_KEYS, hi - p0);
         for (uint32_t i = threadIdx.x; i < cnt * per; i += LD_WARPS * 32)
             cp_async16(tile + (b * LT_KEYS + i / per) * pitch + i % per * 8, cache + static_cast<size_t>((p0 + i / per) % a.capacity) * row + i % per * 8);
+        for (uint32_t i = cnt * per + threadIdx.x; i < LT_KEYS * per; i += LD_WARPS * 32)       // keys past the end: finite
+            *reinterpret_cast<uint4*>(tile + (b * LT_KEYS + i / per) * pitch + i % per * 8) = make_uint4(0, 0, 0, 0);
         cp_async_commit();
     };
     if (lo < hi) stage(lo, 0);
@@ -267,8 +277,8 @@ __global__ void __launch_bounds__(LD_WARPS * 32) latent_decode_mma_kernel(const 
 #pragma unroll
         for (int c = 0; c < NT; ++c) o[m][c][0] = o[m][c][1] = o[m][c][2] = o[m][c][3] = 0.f;
     const uint32_t col0 = warp * 8 * NT;
-    for (uint32_t p0 = lo, b = 0; p0 < hi; p0 += LT_KEYS, b ^= 1) {
-        if (p0 + LT_KEYS < hi) { stage(p0 + LT_KEYS, b ^ 1); cp_async_wait<1>(); }
+    for (uint32_t p0 = lo, b = 0; p0 < hi; p0 += LT_KEYS) {
+        if (bufs == 2 && p0 + LT_KEYS < hi) { stage(p0 + LT_KEYS, b ^ 1); cp_async_wait<1>(); }
         else cp_async_wait<0>();
         __syncthreads();
         const uint32_t cnt = min(LT_KEYS, hi - p0), ts = smem_u32(tile + b * LT_KEYS * pitch);
@@ -337,22 +347,54 @@ __global__ void __launch_bounds__(LD_WARPS * 32) latent_decode_mma_kernel(const 
             }
         }
         __syncthreads();
+        if (bufs == 2) b ^= 1;
+        else if (p0 + LT_KEYS < hi) stage(p0 + LT_KEYS, 0);
     }
-    float* dst = part + (static_cast<size_t>(split) * a.heads + h_cta) * part_elems(a);
+    // this split's sums and statistics to shared memory (over the tiles, which nobody reads any more)
+    float* sums = reinterpret_cast<float*>(tile);                          // [HG][rp]
 #pragma unroll
-    for (int g = 0; g < HW; ++g) {
-        const uint32_t h = warp * HW + g;
-        if (lane == 0 && h_cta + h < a.heads) { dst[h * part_elems(a)] = mx[g]; dst[h * part_elems(a) + 1] = l[g]; }
-    }
+    for (int g = 0; g < HW; ++g)
+        if (lane == 0) { stats[warp * HW + g][0] = mx[g]; stats[warp * HW + g][1] = l[g]; }
 #pragma unroll
     for (int m = 0; m < MT; ++m)
 #pragma unroll
         for (int c = 0; c < NT; ++c)
 #pragma unroll
             for (int u = 0; u < 2; ++u) {
-                const uint32_t h = 16 * m + gid + 8 * u, d = col0 + 8 * c + 2 * t4;
-                if (h_cta + h < a.heads && d < rp) *reinterpret_cast<float2*>(dst + h * part_elems(a) + 4 + d) = make_float2(o[m][c][2 * u], o[m][c][2 * u + 1]);
+                const uint32_t d = col0 + 8 * c + 2 * t4;
+                if (d < rp) *reinterpret_cast<float2*>(sums + (16 * m + gid + 8 * u) * rp + d) = make_float2(o[m][c][2 * u], o[m][c][2 * u + 1]);
             }
+    namespace cg = cooperative_groups;
+    const cg::cluster_group cl = cg::this_cluster();
+    const uint32_t rank = cl.block_rank(), size = cl.num_blocks();
+    cl.sync();
+    float* dst = part + (static_cast<size_t>(split / size) * a.heads + h_cta) * part_elems(a);
+    if (threadIdx.x < HG) {
+        const uint32_t h = threadIdx.x;
+        float m = -CUDART_INF_F, t = 0.f;
+        for (uint32_t r = 0; r < size; ++r) m = fmaxf(m, cl.map_shared_rank(&stats[0][0], r)[2 * h]);
+        for (uint32_t r = 0; r < size; ++r) {
+            const float* st = cl.map_shared_rank(&stats[0][0], r) + 2 * h;
+            const float c = st[0] == -CUDART_INF_F ? 0.f : expf(st[0] - m);
+            weight[r][h] = c;
+            t += st[1] * c;
+        }
+        if (rank == 0 && h_cta + h < a.heads) { dst[h * part_elems(a)] = m; dst[h * part_elems(a) + 1] = t; }
+    }
+    __syncthreads();
+    for (uint32_t i = rank * LD_WARPS * 32 + threadIdx.x; i < HG * (rp / 4); i += size * LD_WARPS * 32) {
+        const uint32_t h = i / (rp / 4), d = 4 * (i % (rp / 4));
+        if (h_cta + h >= a.heads) break;
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (uint32_t r = 0; r < LT_CLUSTER; ++r) {
+            if (r >= size) break;
+            const float4 x = *reinterpret_cast<const float4*>(cl.map_shared_rank(sums, r) + h * rp + d);
+            axpy(v, weight[r][h], x);
+        }
+        *reinterpret_cast<float4*>(dst + h * part_elems(a) + 4 + d) = v;
+    }
+    cl.sync();                                                             // nobody leaves while its sums are read
 }
 
 // grid (heads, slices of the value rows): merge of the splits, then the head's value matrix
@@ -422,52 +464,62 @@ uint32_t elem_bytes(const hf2q_latent_attn& a) { return a.cache_dtype == HF2Q_DT
 uint32_t heads_per_warp(const hf2q_latent_attn& a) {
     return a.heads > 2 * LD_WARPS && a.kv_rank <= 512 && decode_smem(a, 4, elem_bytes(a)) <= LD_SMEM ? 4 : 1;
 }
-size_t mma_smem(const hf2q_latent_attn& a, uint32_t mt) {
-    return 16ull * mt * (tile_pitch(a) * 2 + LT_SP * 4 + LT_PP * 2) + 2ull * LT_KEYS * tile_pitch(a) * 2;
+size_t mma_smem(const hf2q_latent_attn& a, uint32_t mt, uint32_t bufs) {
+    return 16ull * mt * (tile_pitch(a) * 2 + LT_SP * 4 + LT_PP * 2) + static_cast<size_t>(bufs) * LT_KEYS * tile_pitch(a) * 2;
 }
-uint32_t mma_mt(const hf2q_latent_attn& a) { return a.heads > 16 && mma_smem(a, 2) <= LD_SMEM ? 2 : 1; }
-bool on_tensor_cores(const hf2q_latent_attn& a) { return a.cache_dtype == HF2Q_DT_BF16 && a.kv_rank <= 512 && mma_smem(a, 1) <= LD_SMEM; }
-uint32_t head_groups(const hf2q_latent_attn& a) {
-    const uint32_t per = on_tensor_cores(a) ? 16 * mma_mt(a) : LD_WARPS * heads_per_warp(a);
+// 16 heads per CTA as long as the tiles of the window do not fill the GPU
+uint32_t mma_mt(const hf2q_latent_attn& a, int sms) {
+    const uint64_t ctas = static_cast<uint64_t>((a.heads + 15) / 16) * ((a.window + LT_KEYS - 1) / LT_KEYS);
+    return a.heads > 16 && ctas > static_cast<uint64_t>(sms) && mma_smem(a, 2, 1) <= LD_SMEM ? 2 : 1;
+}
+bool on_tensor_cores(const hf2q_latent_attn& a) { return a.cache_dtype == HF2Q_DT_BF16 && a.kv_rank <= 512 && mma_smem(a, 1, 1) <= LD_SMEM; }
+uint32_t head_groups(const hf2q_latent_attn& a, int sms) {
+    const uint32_t per = on_tensor_cores(a) ? 16 * mma_mt(a, sms) : LD_WARPS * heads_per_warp(a);
     return (a.heads + per - 1) / per;
 }
+uint32_t cluster_of(uint32_t splits) { return splits % 8 == 0 ? 8 : splits % 4 == 0 ? 4 : splits % 2 == 0 ? 2 : 1; }
 uint32_t decode_splits(const hf2q_latent_attn& a, int sms) {
-    const uint32_t keys = on_tensor_cores(a) ? LT_KEYS : LD_KEYS, by_sm = static_cast<uint32_t>(sms) / head_groups(a), by_keys = (a.window + keys - 1) / keys;
-    const uint32_t s = by_sm < by_keys ? by_sm : by_keys;
-    return s < 1 ? 1 : s > LD_SPLITS ? LD_SPLITS : s;
+    const bool tc = on_tensor_cores(a);
+    const uint32_t keys = tc ? LT_KEYS : LD_KEYS, by_sm = static_cast<uint32_t>(sms) / head_groups(a, sms), by_keys = (a.window + keys - 1) / keys;
+    uint32_t s = by_sm < by_keys ? by_sm : by_keys;
+    s = s < 1 ? 1 : s > LD_SPLITS ? LD_SPLITS : s;
+    return tc && s > 8 ? s / 8 * 8 : s;                                    // whole clusters
 }
 uint64_t query_floats(const hf2q_latent_attn& a) { return (static_cast<uint64_t>(a.heads) * row_elems(a) + 63) & ~63ull; }
 
 template <typename T, int NH, int NC>
-cudaError_t launch_decode(const hf2q_latent_attn& a, const float* qa, float* part, uint32_t splits, cudaStream_t st) {
+cudaError_t launch_decode(const hf2q_latent_attn& a, const float* qa, float* part, uint32_t splits, uint32_t groups, cudaStream_t st) {
     static PerDeviceFlag flag;
     if (const cudaError_t e = ensure_max_dynamic_smem(latent_decode_kernel<T, NH, NC>, static_cast<int>(LD_SMEM), flag); e != cudaSuccess) return e;
     const uint32_t bufs = decode_smem(a, NH, sizeof(T)) <= LD_SMEM ? 2 : 1;
     const size_t smem = decode_smem(a, NH, sizeof(T)) - (bufs == 1 ? static_cast<size_t>(LD_KEYS) * (row_elems(a) + 16 / sizeof(T)) * sizeof(T) : 0);
     if (smem > LD_SMEM) return cudaErrorInvalidValue;
-    return launch_pdl(latent_decode_kernel<T, NH, NC>, dim3(head_groups(a), splits), dim3(LD_WARPS * 32), smem, st, a, bufs, qa, part);
+    return launch_pdl(latent_decode_kernel<T, NH, NC>, dim3(groups, splits), dim3(LD_WARPS * 32), smem, st, a, bufs, qa, part);
+}
+template <int MT, int NT>
+cudaError_t launch_decode_nt(const hf2q_latent_attn& a, const float* qa, float* part, uint32_t splits, uint32_t groups, cudaStream_t st) {
+    static PerDeviceFlag flag;
+    if (const cudaError_t e = ensure_max_dynamic_smem(latent_decode_mma_kernel<MT, NT>, static_cast<int>(LD_SMEM), flag); e != cudaSuccess) return e;
+    const uint32_t tiles = (a.window + LT_KEYS - 1) / LT_KEYS, bufs = tiles > splits && mma_smem(a, MT, 2) <= LD_SMEM ? 2 : 1;
+    return launch_pdl_cluster(latent_decode_mma_kernel<MT, NT>, dim3(groups, splits), dim3(LD_WARPS * 32), dim3(1, cluster_of(splits)), mma_smem(a, MT, bufs), st, a, bufs,
+                              qa, part);
 }
 template <int MT>
-cudaError_t launch_decode_mma(const hf2q_latent_attn& a, const float* qa, float* part, uint32_t splits, cudaStream_t st) {
-    auto launch = [&](auto kern, PerDeviceFlag& flag) {
-        if (const cudaError_t e = ensure_max_dynamic_smem(kern, static_cast<int>(LD_SMEM), flag); e != cudaSuccess) return e;
-        return launch_pdl(kern, dim3(head_groups(a), splits), dim3(LD_WARPS * 32), mma_smem(a, MT), st, a, qa, part);
-    };
-    static PerDeviceFlag f2, f4, f8;
-    if (a.kv_rank <= 128) return launch(latent_decode_mma_kernel<MT, 2>, f2);
-    if (a.kv_rank <= 256) return launch(latent_decode_mma_kernel<MT, 4>, f4);
-    return launch(latent_decode_mma_kernel<MT, 8>, f8);
+cudaError_t launch_decode_mma(const hf2q_latent_attn& a, const float* qa, float* part, uint32_t splits, uint32_t groups, cudaStream_t st) {
+    if (a.kv_rank <= 128) return launch_decode_nt<MT, 2>(a, qa, part, splits, groups, st);
+    if (a.kv_rank <= 256) return launch_decode_nt<MT, 4>(a, qa, part, splits, groups, st);
+    return launch_decode_nt<MT, 8>(a, qa, part, splits, groups, st);
 }
 template <typename T>
-cudaError_t launch_decode_any(const hf2q_latent_attn& a, const float* qa, float* part, uint32_t splits, cudaStream_t st) {
-    if (on_tensor_cores(a)) return mma_mt(a) == 2 ? launch_decode_mma<2>(a, qa, part, splits, st) : launch_decode_mma<1>(a, qa, part, splits, st);
+cudaError_t launch_decode_any(const hf2q_latent_attn& a, const float* qa, float* part, uint32_t splits, uint32_t groups, int sms, cudaStream_t st) {
+    if (on_tensor_cores(a)) return mma_mt(a, sms) == 2 ? launch_decode_mma<2>(a, qa, part, splits, groups, st) : launch_decode_mma<1>(a, qa, part, splits, groups, st);
     if (heads_per_warp(a) == 4) {
-        if (a.kv_rank <= 128) return launch_decode<T, 4, 2>(a, qa, part, splits, st);
-        return launch_decode<T, 4, 8>(a, qa, part, splits, st);
+        if (a.kv_rank <= 128) return launch_decode<T, 4, 2>(a, qa, part, splits, groups, st);
+        return launch_decode<T, 4, 8>(a, qa, part, splits, groups, st);
     }
-    if (a.kv_rank <= 128) return launch_decode<T, 1, 2>(a, qa, part, splits, st);
-    if (a.kv_rank <= 512) return launch_decode<T, 1, 8>(a, qa, part, splits, st);
-    return launch_decode<T, 1, 16>(a, qa, part, splits, st);
+    if (a.kv_rank <= 128) return launch_decode<T, 1, 2>(a, qa, part, splits, groups, st);
+    if (a.kv_rank <= 512) return launch_decode<T, 1, 8>(a, qa, part, splits, groups, st);
+    return launch_decode<T, 1, 16>(a, qa, part, splits, groups, st);
 }
 
 }  // namespace
@@ -495,13 +547,14 @@ HF2Q_API int32_t hf2q_cuda_latent_decode(hf2q_ctx* ctx, void* stream, const hf2q
     const cudaStream_t st = static_cast<cudaStream_t>(stream);
     float* qa = static_cast<float*>(scratch);
     float* part = qa + query_floats(*a);
-    const uint32_t splits = decode_splits(*a, ctx_sm_count(ctx)), slices = (pad8(a->kv_rank) + LQ_ROWS - 1) / LQ_ROWS;
+    const int sms = ctx_sm_count(ctx);
+    const uint32_t splits = decode_splits(*a, sms), groups = head_groups(*a, sms), parts = on_tensor_cores(*a) ? splits / cluster_of(splits) : splits, slices = (pad8(a->kv_rank) + LQ_ROWS - 1) / LQ_ROWS;
     const dim3 grid_q(a->heads * slices + 1);
     const bool f32 = a->cache_dtype == HF2Q_DT_F32;
     cudaError_t e = f32 ? launch_pdl(latent_query_kernel<float>, grid_q, dim3(256), 0, st, *a, slices, qa)
                         : launch_pdl(latent_query_kernel<__nv_bfloat16>, grid_q, dim3(256), 0, st, *a, slices, qa);
-    if (e == cudaSuccess) e = f32 ? launch_decode_any<float>(*a, qa, part, splits, st) : launch_decode_any<__nv_bfloat16>(*a, qa, part, splits, st);
-    if (e == cudaSuccess) e = launch_pdl(latent_out_kernel, dim3(a->heads, (a->vdim + LO_ROWS - 1) / LO_ROWS), dim3(256), 0, st, *a, splits, part, out);
+    if (e == cudaSuccess) e = f32 ? launch_decode_any<float>(*a, qa, part, splits, groups, sms, st) : launch_decode_any<__nv_bfloat16>(*a, qa, part, splits, groups, sms, st);
+    if (e == cudaSuccess) e = launch_pdl(latent_out_kernel, dim3(a->heads, (a->vdim + LO_ROWS - 1) / LO_ROWS), dim3(256), 0, st, *a, parts, part, out);
     return ctx_cuda_result(ctx, e, "latent_decode", 3);
 }
 
