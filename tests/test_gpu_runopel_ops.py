@@ -242,8 +242,7 @@ def test_mamba2_whole_in_portions_and_token_by_token(sop, name, dt):
         assert rel(run_mixer(sop, m, pool, h, cuts, dt), want) < tol, cuts[:5]
 
 
-@pytest.mark.parametrize("dt", [torch.float32, torch.bfloat16])
-def test_mamba2_state_reaches_far_and_forgets_as_told(sop, dt):
+def test_mamba2_state_reaches_far_and_forgets_as_told(sop):
     """The first token's write alone, read a long way on, with slow decays; and heads whose decay is fast."""
     H, P, N, T = 3, 20, 24, 700
     rng = np.random.default_rng(0)
@@ -262,18 +261,13 @@ def test_mamba2_state_reaches_far_and_forgets_as_told(sop, dt):
                      heads=H, groups=1, state=N, vdim=P, taps=1, pos=pos)
         at = 0
         for c in cuts:
-            ssd_scan(sop, a, c, xbc[at:at + c], dd[at:at + c], la[at:at + c], y[at:at + c], dt)
+            sop.ssd_scan(a, c, xbc[at:at + c], dd[at:at + c], la[at:at + c], y[at:at + c])
             at += c
         got = y.cpu().double().numpy().reshape(T, H, P)
-        tol = 1e-4 if dt == torch.float32 else 1e-2
         for h in range(H):
             for lo, hi in ((0, 5), (90, 100), (600, 700)):
                 ref = want[lo:hi, h]
-                assert np.linalg.norm(got[lo:hi, h] - ref) <= tol * np.linalg.norm(ref) + 1e-7 * np.linalg.norm(want[:3, h]), (cuts[:3], h, lo)
-
-
-def ssd_scan(sop, a, m, xbc, dt, la, y, mode):
-    sop.ssd_scan(a, m, xbc, dt, la, y)
+                assert np.linalg.norm(got[lo:hi, h] - ref) <= 1e-4 * np.linalg.norm(ref) + 1e-7 * np.linalg.norm(want[:3, h]), (cuts[:3], h, lo)
 
 
 # ---- latent attention ---------------------------------------------------------------------------------------------
